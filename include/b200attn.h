@@ -128,6 +128,16 @@ int b200_paged_decode_attn_capped(void* out, const void* q, const void* k_cache,
                                   int32_t block_table_stride, float scale, float softcap, const float* sink,
                                   void* workspace, size_t workspace_bytes, int32_t num_ctas, int32_t dtype,
                                   b200_stream_t stream);
+/* The general form: keys of head_dim and values of value_dim (each 64 or 128; the workspace is sized by value_dim);
+ * window > 0: a row of n keys sees the last `window` of them and those below keep_first (window 0: all). */
+int b200_paged_decode_attn_windowed(void* out, const void* q, const void* k_cache, const void* v_cache,
+                                    const int32_t* block_tables, const int32_t* context_lens, int32_t batch,
+                                    int32_t num_heads, int32_t num_kv_heads, int32_t head_dim, int32_t value_dim,
+                                    int64_t q_stride, int64_t out_stride, int32_t num_blocks, int32_t block_size,
+                                    int32_t block_table_stride, float scale, float softcap, const float* sink,
+                                    int32_t window, int32_t keep_first, void* workspace, size_t workspace_bytes,
+                                    int32_t num_ctas, int32_t dtype, b200_stream_t stream);
+
 
 /* ---------------------------------------------------------------------------------
  * K1/K2 + K6 over an FP8 (e4m3) KV cache -- SURVEY.md 8f row f3. An EXTENSION of the path: the
@@ -210,10 +220,23 @@ int b200_prefill_varlen_attn_capped(void* out, const void* q, const void* k, con
                                     int32_t block_size, float scale, float softcap, const float* sink, int32_t dtype,
                                     void* workspace, int64_t workspace_bytes, b200_stream_t stream);
 
+/* The general form: keys of head_dim and values of value_dim (each 64 or 128; out [total_q, num_heads*value_dim], v rows and
+ * caches value_dim wide per head); window > 0: the query at position i sees keys j <= i with i - j < window or
+ * j < keep_first (window 0: every earlier key). Served by the tcgen05 kernel only, like the capped form. */
+int b200_prefill_varlen_attn_windowed(void* out, const void* q, const void* k, const void* v,
+                                      const int32_t* cu_seqlens_q, const int32_t* cu_seqlens_k, int32_t num_seqs,
+                                      int32_t total_q, int32_t total_k, int32_t max_seqlen_q, int32_t max_seqlen_k,
+                                      int32_t num_heads, int32_t num_kv_heads, int32_t head_dim, int32_t value_dim,
+                                      int64_t q_stride, int64_t k_stride, int64_t v_stride, int64_t out_stride,
+                                      const int32_t* block_tables, int32_t block_table_stride, int32_t num_blocks,
+                                      int32_t block_size, float scale, float softcap, const float* sink, int32_t window,
+                                      int32_t keep_first, int32_t dtype, void* workspace, int64_t workspace_bytes,
+                                      b200_stream_t stream);
+
 /* Bytes of split-KV workspace that let b200_prefill_varlen_attn use every SM for ANY launch it would
  * split (few query rows against many keys): the largest such launch has 148 CTAs x 256 rows of
  * un-normalised fp32 partials. A smaller (or NULL) workspace is legal: fewer (or no) key splits. */
-int64_t b200_prefill_workspace_size(int32_t head_dim);
+int64_t b200_prefill_workspace_size(int32_t head_dim);   /* head_dim: of the values */
 
 /* Tuning / test hook, process-wide: the tcgen05 prefill kernel has two CTA layouts -- 1 query tile of
  * 128 rows per CTA with two CTAs per SM, or 2 ping-pong tiles per CTA with one CTA per SM -- and picks
@@ -481,22 +504,25 @@ int b200_unitnorm_temp_cache(void* qkv, int64_t stride, const int64_t* positions
 
 /* out = gate-and-norm of y [rows, n] (fp32 when y_is_f32, else dtype) with gate [rows, n] (dtype, row
  * stride): RMS norm over each of `groups` equal parts times weight, the gate act(g) (0 sigmoid, 1 silu)
- * applied before the norm (gate_first) or after it; weight == NULL: the gate alone. */
+ * applied before the norm (gate_first) or after it; weight == NULL: the gate alone. The result times out_scale is rounded
+ * and written with row stride out_stride (a slice of a wider row). */
 int b200_gated_norm(void* out, const void* y, int32_t y_is_f32, const void* gate, int64_t gate_stride,
                     const float* weight, float eps, int32_t rows, int32_t n, int32_t groups,
-                    int32_t gate_first, int32_t gate_act, int32_t dtype, b200_stream_t stream);
+                    int32_t gate_first, int32_t gate_act, int64_t out_stride, float out_scale, int32_t dtype,
+                    b200_stream_t stream);
 
-/* out[i] = act(x[i]); act: 0 silu, 1 relu, 2 gelu (tanh form), 3 squared relu. */
+/* out[i] = act(x[i]); act: 0 silu, 1 relu, 2 gelu (tanh form), 3 squared relu, 4 tanh. */
 int b200_act_only(void* out, const void* x, int64_t total, int32_t act, int32_t dtype, b200_stream_t stream);
 
 /* A norm on a sublayer's OUTPUT, then the fp32 residual: u = y[iy] (+ y2[iy2]); n = norm(u) -- kind 0: layer norm
  * (u - mean) / sqrt(var + eps) * w + b (b may be NULL), kind 1: u / sqrt(mean u^2 + eps) * (offset + w); residual
- * <- accumulate ? residual + n : n; h (may be NULL) <- residual in `dtype`. iy = y_index ? clamp(y_index[r], y_rows)
+ * <- n (accumulate 0), residual + n (1); accumulate 2: u also has carry * residual, residual <- n (a norm after the sum).
+ * h (may be NULL) <- residual in `dtype`. iy = y_index ? clamp(y_index[r], y_rows)
  * : r, likewise iy2: rows gathered by token id / position (embedding + learned position + norm in one launch). */
 int b200_norm_residual(void* h, float* residual, const void* y, const int64_t* y_index, int64_t y_rows,
                        const void* y2, const int64_t* y2_index, int64_t y2_rows, const float* w, const float* b,
-                       float eps, float offset, int32_t kind, int32_t accumulate, int32_t rows, int32_t hidden,
-                       int32_t dtype, b200_stream_t stream);
+                       float eps, float offset, int32_t kind, int32_t accumulate, float carry, int32_t rows,
+                       int32_t hidden, int32_t dtype, b200_stream_t stream);
 
 /* In place on x [T, nq | nk | nv] (row stride `stride`): q and k are divided by the root mean square of ALL their
  * columns (every head at once) and multiplied by the plain weights wq [nq], wk [nk]; k and v rows are stored at
@@ -549,7 +575,7 @@ int b200_act_and_mul(void* out, const void* x, int32_t rows, int32_t inter, int3
 /* Causal softmax attention for any key size `dim` and value size `vdim` (<= 512), packed keys
  * (block_tables == NULL: k, v are this step's rows in the order of cu_k) or paged caches
  * [nb, bs, G*dim] / [nb, bs, G*vdim]. q [T, H, dim] -> out [T, H*vdim]. fp32 scores and accumulation.
- * window > 0: the query at position i sees keys j with 0 <= i - j < window. v == NULL: the values are the
+ * window > 0: the query at position i sees keys j <= i with i - j < window or j < keep_first. v == NULL: the values are the
  * first vdim columns of the key rows (one cached latent row serves as key and as value; vdim <= dim).
  * softcap > 0: scores become softcap * tanh(score / softcap). sink (fp32 [H] or NULL): exp(sink[h]) joins the softmax
  * denominator without a value. gate ([T, gate_stride] of dtype, or NULL): head h of token t is multiplied by
@@ -558,7 +584,7 @@ int b200_attn_generic(void* out, const void* q, int64_t q_stride, const void* k,
                       const void* v, int64_t v_stride, const int32_t* block_tables, int32_t bt_stride,
                       int32_t block_size, const int32_t* cu_q, const int32_t* cu_k, const int32_t* ctx_lens,
                       int32_t num_seqs, int32_t max_q, int32_t num_heads, int32_t num_kv_heads, int32_t dim,
-                      int32_t vdim, float scale, int32_t window, float softcap, const float* sink, const void* gate,
+                      int32_t vdim, float scale, int32_t window, int32_t keep_first, float softcap, const float* sink, const void* gate,
                       int64_t gate_stride, int32_t dtype, b200_stream_t stream);
 
 /* Per head S_t = a_t S_(t-1) + k_t (b_t v_t)^T, o_t = S_t^T q_t; S fp32 [kdim, vdim] in state
@@ -606,20 +632,29 @@ int b200_rotary_heads(void* out, int64_t out_stride, int32_t out_head, int32_t o
 
 /* Inputs of b200_delta_rule from projected activations: qk [T, 2*groups*dim] fp32 = q and k heads of qk_in
  * divided by sqrt(sum x^2 + unit_eps), q also times q_scale; decay [T, H*dim] fp32 =
- * exp(-exp(a_log[h]) softplus(a[t, h*dim + i] + dt_bias[h*dim + i])); beta [T, H] = sigmoid(b[t, h]). */
+ * exp(-exp(a_log[h]) softplus(a[t, h*dim + i] + dt_bias[h*dim + i])); beta [T, H] = sigmoid(b[t, h]). per_head: one decay
+ * per head, a [T, H], dt_bias [H], decay [T, H]. */
 int b200_delta_prep(float* qk, float* decay, float* beta, const void* qk_in, int64_t qk_stride, const void* a,
                     int64_t a_stride, const void* b, int64_t b_stride, const float* dt_bias, const float* a_log,
                     int32_t tokens, int32_t num_heads, int32_t groups, int32_t dim, float unit_eps,
-                    float q_scale, int32_t dtype, b200_stream_t stream);
+                    float q_scale, int32_t per_head, int32_t dtype, b200_stream_t stream);
 
 /* Gated delta rule per head: S <- diag(g_t) S; w = beta_t (v_t - S^T k_t); S <- S + k_t w^T; o_t = S^T q_t,
  * S fp32 [kdim, vdim] in state [slots, H, kdim, vdim]. q, k fp32 [T, groups*kdim] (row strides given),
- * g fp32 [T, H*kdim], beta fp32 [T, H], v [T, H*vdim] in dtype; out fp32 [T, H*vdim]. kdim <= 256. */
+ * g fp32 [T, H*kdim] (mode 0), beta fp32 [T, H], v [T, H*vdim] in dtype; out fp32 [T, H*vdim]. kdim <= 256. mode 1: one
+ * decay per head, g fp32 [T, H]. mode 2 (wkv): o_t = S^T q_t + beta_t v_t; S <- diag(g_t) S + k_t v_t^T, the read-out
+ * before the write. */
 int b200_delta_rule(float* out, const float* q, int64_t q_stride, const float* k, int64_t k_stride,
                     const void* v, int64_t v_stride, const float* g, const float* beta, float* state,
                     const int32_t* state_slots, const int32_t* cu_q, const int32_t* cu_k,
                     const int32_t* ctx_lens, int32_t num_seqs, int32_t num_heads, int32_t groups, int32_t kdim,
-                    int32_t vdim, int32_t dtype, b200_stream_t stream);
+                    int32_t vdim, int32_t mode, int32_t dtype, b200_stream_t stream);
+
+/* Inputs of the wkv mode from projected activations r, k [T, H*dim] (row strides) and z fp32 [T, H*dim]: r and k in fp32,
+ * decay = exp(-exp(z + w0)), bonus [T, H] = sum_i r_i u_i k_i per head; w0, u fp32 [H*dim]. */
+int b200_wkv_prep(float* r_out, float* k_out, float* decay, float* bonus, const void* r, int64_t r_stride,
+                  const void* k, int64_t k_stride, const float* z, const float* w0, const float* u, int32_t tokens,
+                  int32_t num_heads, int32_t dim, int32_t dtype, b200_stream_t stream);
 
 /* Latent attention, per token: cq [T, q_rank] = rms(dq) * wq; row = [rms(dkv[:rank]) * wc | rotary(dkv[rank:])]
  * (rot columns, the first `dims` rotated) written to kc [T, rank + rot] (optional) and to the paged cache
@@ -703,6 +738,22 @@ int b200_rope_mix_cache(void* qkv, int64_t stride, const float* table, int32_t d
                         const int32_t* slots, int32_t slot_pairs, int32_t block_size, int32_t num_tokens,
                         int32_t num_heads, int32_t num_kv_heads, int32_t dim, int32_t vdim, int32_t dtype,
                         b200_stream_t stream);
+
+/* In place on qkv [T, H*dim | G*dim | G*vdim] (row stride in elements): every q (k) head divided by its root mean square
+ * (eps inside the root) times wq (wk) fp32 [dim], then its first `dims` columns rotated by table [T, dims/2, 2] in pairs
+ * (2i, 2i+1) (interleaved) or (i, i + dims/2), rounded once; k and v rows are stored at `slots` (flat, or (block, offset)
+ * pairs; negative: not stored) of the paged caches [nb, bs, G*dim] / [nb, bs, G*vdim] when given. */
+int b200_norm_rope_cache(void* qkv, int64_t stride, const float* wq, const float* wk, float eps, const float* table,
+                         int32_t dims, int32_t interleaved, void* k_cache, void* v_cache, const int32_t* slots,
+                         int32_t slot_pairs, int32_t block_size, int32_t num_tokens, int32_t num_heads,
+                         int32_t num_kv_heads, int32_t dim, int32_t vdim, int32_t dtype, b200_stream_t stream);
+
+/* out[m * mix_stride + t * width + c] = h_t + (h_(t-1) - h_t) * mu[m, c] for m < mixes (mu fp32 [mixes, width]); h_(-1) is
+ * zero at a sequence's start, else state[slot] ([slots, width], dtype), which then receives the span's last row. */
+int b200_token_shift(void* out, int64_t mix_stride, const void* h, int64_t h_stride, const float* mu, int32_t mixes,
+                     void* state, const int32_t* state_slots, const int32_t* cu_q, const int32_t* cu_k,
+                     const int32_t* ctx_lens, int32_t num_seqs, int32_t max_q, int32_t width, int32_t dtype,
+                     b200_stream_t stream);
 
 /* out[t, h, :] = x[t, h, :] * sigmoid(gate[t * gate_stride + h]); x, out [rows, num_heads * vdim] contiguous. */
 int b200_head_gate(void* out, const void* x, const void* gate, int64_t gate_stride, int32_t rows, int32_t num_heads,

@@ -21,6 +21,8 @@
 //    heads) is the M dimension of mma.sync m16n8k16 (rows 8-15 are structurally zero), i.e.
 //    the whole group shares a single read of the KV bytes. fp32 online softmax in the exp2
 //    domain; running max/sum per thread, reduced with warp shuffles.
+//  * Optional sliding window with kept first tokens: the work list of a row holds only the tiles that have a visible key
+//    (tile_list), borders are masked element by element. Keys and values may have different head sizes (DK, DV).
 //  Algorithmic bytes per launch: sum_b ctx_b * 2 * Hkv * D * 2 B (+ q, out: negligible).
 #include "decode_common.cuh"
 
@@ -31,24 +33,24 @@ namespace b200 {
 
 constexpr int kStages = 3;
 
-template <typename T, int D, int HKV_CTA>
+template <typename T, int DK, int DV, int HKV_CTA>
 __global__ void __launch_bounds__(kDecodeThreads, 1)
 paged_decode_kernel(const __grid_constant__ CUtensorMap tmK,
                     const __grid_constant__ CUtensorMap tmV, const DecodeParams p) {
   constexpr int UNITS = 8 / HKV_CTA;          // 16-token units per tile (per head)
   constexpr int TILE_TOKENS = 16 * UNITS;
-  constexpr int CH = D / 64;                  // 128-byte chunks per head row
-  constexpr int TILE_BYTES = 16 * 8 * D * 2;  // bytes of K (or V) per tile, all variants
-  constexpr int KSTEPS = D / 16;
-  constexpr int NT = D / 8;                   // 8-wide output column tiles
-  constexpr int MERGE_FLOATS = 8 * D + 16;    // one warp's (O rows, m, l)
+  constexpr int CHK = DK / 64, CHV = DV / 64; // 128-byte chunks per key / value head row
+  constexpr int K_BYTES = 16 * 8 * DK * 2, V_BYTES = 16 * 8 * DV * 2;  // bytes of K / V per tile, all variants
+  constexpr int KSTEPS = DK / 16;
+  constexpr int NT = DV / 8;                  // 8-wide output column tiles
+  constexpr int MERGE_FLOATS = 8 * DV + 16;   // one warp's (O rows, m, l)
 
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
                                              ~uintptr_t(1023));
-  uint8_t* kbuf = smem;                                  // [kStages][TILE_BYTES]
-  uint8_t* vbuf = smem + kStages * TILE_BYTES;           // [kStages][TILE_BYTES]
-  float* merge = reinterpret_cast<float*>(smem + 2 * kStages * TILE_BYTES);  // [4][MERGE_FLOATS]
+  uint8_t* kbuf = smem;                                  // [kStages][K_BYTES]
+  uint8_t* vbuf = smem + kStages * K_BYTES;              // [kStages][V_BYTES]
+  float* merge = reinterpret_cast<float*>(smem + kStages * (K_BYTES + V_BYTES));  // [4][MERGE_FLOATS]
   int* prefix = reinterpret_cast<int*>(merge + (UNITS > 1 ? 4 * MERGE_FLOATS : 0));
   const int items = p.batch * p.hg_count;
   uint64_t* bars = reinterpret_cast<uint64_t*>(
@@ -62,8 +64,7 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK,
 
   // ---- tiles per item -> exclusive prefix sum in shared memory
   for (int i = threadIdx.x; i < items; i += blockDim.x) {
-    const int len = p.context_lens[i / p.hg_count];
-    prefix[i + 1] = len > 0 ? (len + TILE_TOKENS - 1) / TILE_TOKENS : 0;
+    prefix[i + 1] = tile_list<TILE_TOKENS>(p.context_lens[i / p.hg_count], p.window, p.keep_first).count;
   }
   if (threadIdx.x == 0) {
     prefix[0] = 0;
@@ -100,7 +101,7 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK,
   }
 
   const int OPS = TILE_TOKENS / p.rows_box;  // TMA ops per full tile (K or V)
-  const int op_bytes = p.rows_box * HKV_CTA * D * 2;
+  const int k_op_bytes = p.rows_box * HKV_CTA * DK * 2, v_op_bytes = p.rows_box * HKV_CTA * DV * 2;
 
   if (warp == kConsumerWarps) {
     // =========================== TMA producer ===========================
@@ -112,7 +113,7 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK,
     int stage = 0, phase = 0;
     for (int t0 = lo; t0 < hi; t0 += 32) {
       const int tt = t0 + lane;
-      int nops = 0, chunk0 = 0;
+      int nops = 0, hg0 = 0;
       int rows[UNITS];
 #pragma unroll
       for (int o = 0; o < UNITS; ++o) rows[o] = -1;
@@ -121,9 +122,9 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK,
         const int j = tt - prefix[it];
         const int b = it / p.hg_count, hg = it - b * p.hg_count;
         const int len = p.context_lens[b];
-        const int tok0 = j * TILE_TOKENS;
+        const int tok0 = tile_list<TILE_TOKENS>(len, p.window, p.keep_first).tile(j) * TILE_TOKENS;
         nops = min(OPS, (len - tok0 + p.rows_box - 1) / p.rows_box);
-        chunk0 = hg * HKV_CTA * CH;
+        hg0 = hg * HKV_CTA;
 #pragma unroll
         for (int o = 0; o < UNITS; ++o) {
           if (o < nops) {
@@ -137,24 +138,24 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK,
       const int n = min(32, hi - t0);
       for (int i = 0; i < n; ++i) {
         const int my_nops = __shfl_sync(0xffffffffu, nops, i);
-        const int my_chunk0 = __shfl_sync(0xffffffffu, chunk0, i);
+        const int my_hg0 = __shfl_sync(0xffffffffu, hg0, i);
         int my_rows[UNITS];
 #pragma unroll
         for (int o = 0; o < UNITS; ++o) my_rows[o] = __shfl_sync(0xffffffffu, rows[o], i);
         if (lane == 0) {
           mbar_wait(&empty[stage], phase ^ 1);
-          mbar_expect_tx(&full_k[stage], my_nops * op_bytes);
+          mbar_expect_tx(&full_k[stage], my_nops * k_op_bytes);
 #pragma unroll
           for (int o = 0; o < UNITS; ++o)
             if (o < my_nops)
-              tma_load_3d(kbuf + stage * TILE_BYTES + o * op_bytes, &tmK, &full_k[stage], 0,
-                          my_rows[o], my_chunk0, policy);
-          mbar_expect_tx(&full_v[stage], my_nops * op_bytes);
+              tma_load_3d(kbuf + stage * K_BYTES + o * k_op_bytes, &tmK, &full_k[stage], 0,
+                          my_rows[o], my_hg0 * CHK, policy);
+          mbar_expect_tx(&full_v[stage], my_nops * v_op_bytes);
 #pragma unroll
           for (int o = 0; o < UNITS; ++o)
             if (o < my_nops)
-              tma_load_3d(vbuf + stage * TILE_BYTES + o * op_bytes, &tmV, &full_v[stage], 0,
-                          my_rows[o], my_chunk0, policy);
+              tma_load_3d(vbuf + stage * V_BYTES + o * v_op_bytes, &tmV, &full_v[stage], 0,
+                          my_rows[o], my_hg0 * CHV, policy);
         }
         if (++stage == kStages) stage = 0, phase ^= 1;
       }
@@ -176,7 +177,7 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK,
   for (int it = blockIdx.x; it < items; it += gridDim.x) {
     if (prefix[it + 1] == prefix[it]) {
       const int b = it / p.hg_count, hg = it - b * p.hg_count;
-      const int n = HKV_CTA * G * D;  // contiguous elements of this head group
+      const int n = HKV_CTA * G * DV;  // contiguous elements of this head group
       T* dst = obase + (int64_t)b * p.out_stride + (int64_t)hg * n;
       for (int e = threadIdx.x * 2; e < n; e += kConsumerWarps * 64)
         *reinterpret_cast<uint32_t*>(dst + e) = 0u;
@@ -188,7 +189,8 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK,
   const int op_idx = tok_off / p.rows_box;
   const int r0 = tok_off - op_idx * p.rows_box;
   const int panel_bytes = p.rows_box * 128;
-  const int unit_base = op_idx * op_bytes + (head_local * CH) * panel_bytes + r0 * 128;
+  const int k_unit = op_idx * k_op_bytes + (head_local * CHK) * panel_bytes + r0 * 128;
+  const int v_unit = op_idx * v_op_bytes + (head_local * CHV) * panel_bytes + r0 * 128;
   // K (non-transposed ldmatrix): matrices (tok0-7,lo16B) (tok0-7,hi16B) (tok8-15,lo) (tok8-15,hi)
   const int k_tok = ((lane >> 4) << 3) + (lane & 7);
   const int k_half = (lane >> 3) & 1;
@@ -207,12 +209,14 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK,
     const int j1 = min(ntiles, j0 + (hi - t));
     const int b = it / p.hg_count, hg = it - b * p.hg_count;
     const int len = p.context_lens[b];
+    const TileList list = tile_list<TILE_TOKENS>(len, p.window, p.keep_first);
+    const int hidden_hi = p.window > 0 ? len - p.window : 0;   // keys [keep_first, hidden_hi) are hidden
     const int kv_head = hg * HKV_CTA + head_local;
 
     // ---- Q fragments for this (sequence, kv head): rows = query heads of the GQA group
     uint32_t qa[KSTEPS][2];
     {
-      const T* qrow = qbase + (int64_t)b * p.q_stride + (int64_t)(kv_head * G + g) * D;
+      const T* qrow = qbase + (int64_t)b * p.q_stride + (int64_t)(kv_head * G + g) * DK;
 #pragma unroll
       for (int ks = 0; ks < KSTEPS; ++ks) {
         qa[ks][0] = g < G ? *reinterpret_cast<const uint32_t*>(qrow + ks * 16 + 2 * t4) : 0u;
@@ -225,11 +229,11 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK,
     float m_run = -INFINITY, l_run = 0.f;
 
     for (int j = j0; j < j1; ++j) {
-      const int tok0 = j * TILE_TOKENS + tok_off;  // first token of this warp's unit
-      const bool active = tok0 < len;
+      const int tok0 = list.tile(j) * TILE_TOKENS + tok_off;  // first token of this warp's unit
+      const bool active = tok0 < len && (tok0 + 16 > hidden_hi || tok0 < p.keep_first);   // some key is visible
       mbar_wait(&full_k[stage], phase);
       if (active) {
-        const uint32_t kb = smem_u32(kbuf + stage * TILE_BYTES) + unit_base;
+        const uint32_t kb = smem_u32(kbuf + stage * K_BYTES) + k_unit;
         float s[2][4];
 #pragma unroll
         for (int n = 0; n < 2; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
@@ -258,6 +262,15 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK,
             for (int e = 0; e < 2; ++e)
               if (n * 8 + 2 * t4 + e >= valid) s[n][e] = -INFINITY;
         }
+        if (tok0 < hidden_hi && tok0 + 16 > p.keep_first) {     // the unit holds keys outside the window
+#pragma unroll
+          for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+              const int key = tok0 + n * 8 + 2 * t4 + e;
+              if (key < hidden_hi && key >= p.keep_first) s[n][e] = -INFINITY;
+            }
+        }
         // online softmax for row g (rows 8..15 are padding)
         float mx = fmaxf(fmaxf(s[0][0], s[0][1]), fmaxf(s[1][0], s[1][1]));
         mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
@@ -278,14 +291,14 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK,
         const uint32_t pa0 = pack2<T>(p00, p01), pa2 = pack2<T>(p10, p11);
 
         mbar_wait(&full_v[stage], phase);
-        uint8_t* vstage = vbuf + stage * TILE_BYTES + unit_base;
+        uint8_t* vstage = vbuf + stage * V_BYTES + v_unit;
         if (valid < 16) {
           // rows past the context hold stale cache bytes (possibly NaN patterns): zero them so
           // that 0 * garbage cannot poison the accumulator.
-          const int nz = (16 - valid) * CH * 8;
+          const int nz = (16 - valid) * CHV * 8;
           for (int idx = lane; idx < nz; idx += 32) {
-            const int row = valid + idx / (CH * 8);
-            const int rem = idx % (CH * 8);
+            const int row = valid + idx / (CHV * 8);
+            const int rem = idx % (CHV * 8);
             *reinterpret_cast<uint4*>(vstage + (rem >> 3) * panel_bytes + row * 128 +
                                       ((rem & 7) << 4)) = make_uint4(0, 0, 0, 0);
           }
@@ -321,19 +334,19 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK,
         if (unit >= stride && unit < 2 * stride) {
 #pragma unroll
           for (int n = 0; n < NT; ++n)
-            *reinterpret_cast<float2*>(slot + g * D + n * 8 + 2 * t4) =
+            *reinterpret_cast<float2*>(slot + g * DV + n * 8 + 2 * t4) =
                 make_float2(o_acc[n][0], o_acc[n][1]);
-          if (t4 == 0) slot[8 * D + g] = m_run, slot[8 * D + 8 + g] = l_run;
+          if (t4 == 0) slot[8 * DV + g] = m_run, slot[8 * DV + 8 + g] = l_run;
         }
         named_bar_sync(1, kConsumerWarps * 32);
         if (unit < stride) {
-          const float m_o = slot[8 * D + g], l_o = slot[8 * D + 8 + g];
+          const float m_o = slot[8 * DV + g], l_o = slot[8 * DV + 8 + g];
           const float m_new = fmaxf(m_run, m_o);
           const float a = m_new == -INFINITY ? 0.f : ex2_approx((m_run - m_new) * sl2);
           const float bsc = m_new == -INFINITY ? 0.f : ex2_approx((m_o - m_new) * sl2);
 #pragma unroll
           for (int n = 0; n < NT; ++n) {
-            const float2 o2 = *reinterpret_cast<const float2*>(slot + g * D + n * 8 + 2 * t4);
+            const float2 o2 = *reinterpret_cast<const float2*>(slot + g * DV + n * 8 + 2 * t4);
             o_acc[n][0] = o_acc[n][0] * a + o2.x * bsc;
             o_acc[n][1] = o_acc[n][1] * a + o2.y * bsc;
           }
@@ -348,7 +361,7 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK,
       if (whole) {
         if (p.sink != nullptr) l_run += ex2_approx(p.sink[kv_head * G + g] * kLog2e - m_run * sl2);
         const float inv = 1.f / l_run;
-        T* orow = obase + (int64_t)b * p.out_stride + (int64_t)(kv_head * G + g) * D;
+        T* orow = obase + (int64_t)b * p.out_stride + (int64_t)(kv_head * G + g) * DV;
 #pragma unroll
         for (int n = 0; n < NT; ++n)
           *reinterpret_cast<uint32_t*>(orow + n * 8 + 2 * t4) =
@@ -357,7 +370,7 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK,
         const int slot = blockIdx.x * 2 + (seg_index == 0 ? 0 : 1);
         const int rows = HKV_CTA * G;
         const int r = head_local * G + g;
-        float* po = p.part_o + ((int64_t)slot * rows + r) * D;
+        float* po = p.part_o + ((int64_t)slot * rows + r) * DV;
 #pragma unroll
         for (int n = 0; n < NT; ++n)
           *reinterpret_cast<float2*>(po + n * 8 + 2 * t4) = make_float2(o_acc[n][0], o_acc[n][1]);
@@ -449,15 +462,14 @@ int get_panel_map(const void* cache, int64_t rows, int64_t row_bytes, int chunks
   return B200_OK;
 }
 
-template <typename T, int D, int HKV_CTA>
+template <typename T, int DK, int DV, int HKV_CTA>
 static int decode_launch_t(const CUtensorMap& mk, const CUtensorMap& mv, const DecodeParams& p,
                            int grid, cudaStream_t stream) {
   constexpr int UNITS = 8 / HKV_CTA;
-  constexpr int TILE_BYTES = 16 * 8 * D * 2;
   const int items = p.batch * p.hg_count;
-  size_t smem = 1024 + 2 * kStages * TILE_BYTES + (UNITS > 1 ? 4 * (8 * D + 16) * 4 : 0) +
+  size_t smem = 1024 + kStages * 16 * 8 * (DK + DV) * 2 + (UNITS > 1 ? 4 * (8 * DV + 16) * 4 : 0) +
                 (items + 1) * 4 + 8 + 3 * kStages * 8;
-  auto kern = paged_decode_kernel<T, D, HKV_CTA>;
+  auto kern = paged_decode_kernel<T, DK, DV, HKV_CTA>;
   static bool attr_set = false;
   if (!attr_set) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -471,19 +483,19 @@ static int decode_launch_t(const CUtensorMap& mk, const CUtensorMap& mv, const D
     // small batches: one item may span every CTA -> one block per (boundary, row)
     const int rows = HKV_CTA * p.G;
     const dim3 cgrid(grid - 1, items >= 64 ? 1 : rows);
-    launch_pdl(decode_combine_kernel<T, D>, cgrid, dim3(256), 0, stream, p, rows);
+    launch_pdl(decode_combine_kernel<T, DV>, cgrid, dim3(256), 0, stream, p, rows);
   }
   return finish_launch(grid > 1 ? 2 : 1);
 }
 
-template <typename T, int D>
+template <typename T, int DK, int DV>
 static int decode_launch_d(int hkv_cta, const CUtensorMap& mk, const CUtensorMap& mv,
                            const DecodeParams& p, int grid, cudaStream_t stream) {
   switch (hkv_cta) {
-    case 8: return decode_launch_t<T, D, 8>(mk, mv, p, grid, stream);
-    case 4: return decode_launch_t<T, D, 4>(mk, mv, p, grid, stream);
-    case 2: return decode_launch_t<T, D, 2>(mk, mv, p, grid, stream);
-    case 1: return decode_launch_t<T, D, 1>(mk, mv, p, grid, stream);
+    case 8: return decode_launch_t<T, DK, DV, 8>(mk, mv, p, grid, stream);
+    case 4: return decode_launch_t<T, DK, DV, 4>(mk, mv, p, grid, stream);
+    case 2: return decode_launch_t<T, DK, DV, 2>(mk, mv, p, grid, stream);
+    case 1: return decode_launch_t<T, DK, DV, 1>(mk, mv, p, grid, stream);
   }
   return B200_ERR_UNSUPPORTED;
 }
@@ -528,6 +540,20 @@ extern "C" int b200_paged_decode_attn_capped(void* out, const void* q, const voi
                                              float softcap, const float* sink, void* workspace,
                                              size_t workspace_bytes, int32_t num_ctas, int32_t dtype,
                                              b200_stream_t stream_) {
+  return b200_paged_decode_attn_windowed(out, q, k_cache, v_cache, block_tables, context_lens, batch, num_heads,
+                                         num_kv_heads, head_dim, head_dim, q_stride, out_stride, num_blocks, block_size,
+                                         block_table_stride, scale, softcap, sink, 0, 0, workspace, workspace_bytes,
+                                         num_ctas, dtype, stream_);
+}
+
+extern "C" int b200_paged_decode_attn_windowed(void* out, const void* q, const void* k_cache, const void* v_cache,
+                                               const int32_t* block_tables, const int32_t* context_lens, int32_t batch,
+                                               int32_t num_heads, int32_t num_kv_heads, int32_t head_dim,
+                                               int32_t value_dim, int64_t q_stride, int64_t out_stride,
+                                               int32_t num_blocks, int32_t block_size, int32_t block_table_stride,
+                                               float scale, float softcap, const float* sink, int32_t window,
+                                               int32_t keep_first, void* workspace, size_t workspace_bytes,
+                                               int32_t num_ctas, int32_t dtype, b200_stream_t stream_) {
   cudaStream_t stream = (cudaStream_t)stream_;
   B200_RETURN_IF(dtype != B200_DTYPE_BF16 && dtype != B200_DTYPE_F16, B200_ERR_BAD_DTYPE);
   B200_RETURN_IF(batch < 0 || num_heads <= 0 || num_kv_heads <= 0 || num_blocks <= 0 ||
@@ -538,7 +564,8 @@ extern "C" int b200_paged_decode_attn_capped(void* out, const void* q, const voi
   B200_RETURN_IF(!out || !q || !k_cache || !v_cache || !block_tables || !context_lens ||
                      !workspace,
                  B200_ERR_NULL_POINTER);
-  B200_RETURN_IF(head_dim != 64 && head_dim != 128, B200_ERR_UNSUPPORTED);
+  B200_RETURN_IF((head_dim != 64 && head_dim != 128) || (value_dim != 64 && value_dim != 128), B200_ERR_UNSUPPORTED);
+  B200_RETURN_IF(window < 0 || keep_first < 0, B200_ERR_BAD_SHAPE);
   const int G = num_heads / num_kv_heads;
   const int hkv_cta = hkv_cta_of(num_kv_heads);
   B200_RETURN_IF(G > 8 || hkv_cta == 0, B200_ERR_UNSUPPORTED);
@@ -549,7 +576,7 @@ extern "C" int b200_paged_decode_attn_capped(void* out, const void* q, const voi
   const int hg_count = num_kv_heads / hkv_cta;
   B200_RETURN_IF((int64_t)batch * hg_count > kMaxItems, B200_ERR_UNSUPPORTED);
   B200_RETURN_IF(q_stride < (int64_t)num_heads * head_dim ||
-                     out_stride < (int64_t)num_heads * head_dim,
+                     out_stride < (int64_t)num_heads * value_dim,
                  B200_ERR_BAD_SHAPE);
   B200_RETURN_IF(q_stride % 2 != 0 || out_stride % 2 != 0 ||
                      (reinterpret_cast<uintptr_t>(q) & 3) || (reinterpret_cast<uintptr_t>(out) & 3),
@@ -557,7 +584,7 @@ extern "C" int b200_paged_decode_attn_capped(void* out, const void* q, const voi
   B200_RETURN_IF(!aligned16(k_cache) || !aligned16(v_cache) || !aligned16(workspace),
                  B200_ERR_MISALIGNED);
   B200_RETURN_IF(workspace_bytes <
-                     b200_paged_decode_attn_workspace_size(batch, num_heads, num_kv_heads, head_dim),
+                     b200_paged_decode_attn_workspace_size(batch, num_heads, num_kv_heads, value_dim),
                  B200_ERR_WORKSPACE);
 
   DecodeParams p;
@@ -573,7 +600,7 @@ extern "C" int b200_paged_decode_attn_capped(void* out, const void* q, const voi
   p.owner = reinterpret_cast<int32_t*>(ws);
   ws += align_up((size_t)kMaxCtas * 4, 256);
   p.part_o = reinterpret_cast<float*>(ws);
-  ws += align_up((size_t)kMaxCtas * 2 * rows * head_dim * 4, 256);
+  ws += align_up((size_t)kMaxCtas * 2 * rows * value_dim * 4, 256);
   p.part_ml = reinterpret_cast<float*>(ws);
   p.q_stride = q_stride;
   p.out_stride = out_stride;
@@ -588,24 +615,24 @@ extern "C" int b200_paged_decode_attn_capped(void* out, const void* q, const voi
   p.scale_log2 = scale * 1.4426950408889634f;
   if (softcap > 0.f) p.cap = softcap, p.cap_pre = scale / softcap;
   p.sink = sink;
+  p.window = window, p.keep_first = window > 0 ? keep_first : 0;
 
-  const int chunks = num_kv_heads * head_dim / 64;
-  const int chunks_box = hkv_cta * head_dim / 64;
+  const int k_chunks = num_kv_heads * head_dim / 64, v_chunks = num_kv_heads * value_dim / 64;
   CUtensorMap mk, mv;
-  int rc = get_panel_map(k_cache, (int64_t)num_blocks * block_size, (int64_t)chunks * 128, chunks,
-                         p.rows_box, chunks_box, dtype, &mk);
+  int rc = get_panel_map(k_cache, (int64_t)num_blocks * block_size, (int64_t)k_chunks * 128, k_chunks,
+                         p.rows_box, hkv_cta * head_dim / 64, dtype, &mk);
   if (rc != B200_OK) return rc;
-  rc = get_panel_map(v_cache, (int64_t)num_blocks * block_size, (int64_t)chunks * 128, chunks,
-                     p.rows_box, chunks_box, dtype, &mv);
+  rc = get_panel_map(v_cache, (int64_t)num_blocks * block_size, (int64_t)v_chunks * 128, v_chunks,
+                     p.rows_box, hkv_cta * value_dim / 64, dtype, &mv);
   if (rc != B200_OK) return rc;
 
   int grid = num_ctas > 0 ? num_ctas : num_sms();
   if (grid > kMaxCtas) grid = kMaxCtas;
-  if (dtype == B200_DTYPE_BF16) {
-    return head_dim == 128
-               ? decode_launch_d<__nv_bfloat16, 128>(hkv_cta, mk, mv, p, grid, stream)
-               : decode_launch_d<__nv_bfloat16, 64>(hkv_cta, mk, mv, p, grid, stream);
-  }
-  return head_dim == 128 ? decode_launch_d<__half, 128>(hkv_cta, mk, mv, p, grid, stream)
-                         : decode_launch_d<__half, 64>(hkv_cta, mk, mv, p, grid, stream);
+#define B200_DECODE_DISPATCH(T)                                                              \
+  (head_dim == 128 ? (value_dim == 128 ? decode_launch_d<T, 128, 128>(hkv_cta, mk, mv, p, grid, stream)  \
+                                       : decode_launch_d<T, 128, 64>(hkv_cta, mk, mv, p, grid, stream))  \
+                   : (value_dim == 128 ? decode_launch_d<T, 64, 128>(hkv_cta, mk, mv, p, grid, stream)   \
+                                       : decode_launch_d<T, 64, 64>(hkv_cta, mk, mv, p, grid, stream)))
+  return dtype == B200_DTYPE_BF16 ? B200_DECODE_DISPATCH(__nv_bfloat16) : B200_DECODE_DISPATCH(__half);
+#undef B200_DECODE_DISPATCH
 }

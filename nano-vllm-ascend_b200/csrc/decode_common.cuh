@@ -29,7 +29,24 @@ struct DecodeParams {
   // query head (fp32 [H], natural-log units) that joins the softmax denominator without a value
   float cap = 0.f, cap_pre = 0.f;
   const float* sink = nullptr;
+  int window = 0, keep_first = 0;   // window > 0: only the last `window` keys and those below keep_first are visible
 };
+
+// The key tiles (of TT tokens) that a row of `len` keys visits: tile j of the row's list is tile j of its keys for j < kept,
+// tile j + skip past them.
+struct TileList {
+  int kept, skip, count;
+  __device__ __forceinline__ int tile(int j) const { return j < kept ? j : j + skip; }
+};
+template <int TT>
+__device__ __forceinline__ TileList tile_list(int len, int window, int keep_first) {
+  TileList r;
+  const int all = len > 0 ? (len + TT - 1) / TT : 0;
+  r.kept = window > 0 ? (min(keep_first, max(len, 0)) + TT - 1) / TT : 0;
+  r.skip = window > 0 ? max(0, max(0, len - window) / TT - r.kept) : 0;
+  r.count = all - r.skip;
+  return r;
+}
 
 // first idx in [1, items] with prefix[idx] > t, minus one
 __device__ __forceinline__ int find_item(const int* prefix, int items, int t) {

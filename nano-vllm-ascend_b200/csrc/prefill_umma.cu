@@ -32,6 +32,11 @@
 // issuing thread and execute in issue order; softmax(j+1) of tile t starts only after S[t](j+1) has
 // completed, hence after PV[t](j) has.
 //
+// Sliding window with kept first tokens (window > 0): position i sees j <= i with i - j < window or j < keep_first. A CTA
+// visits the tiles of the kept keys, then those from its first row's window on; the tiles between are skipped by
+// index (p.keep_tiles, `skip`), the borders are masked element by element.
+// Keys and values may have different head sizes (DK, DV in {64, 128}); D below stands for the one that applies.
+//
 // Split-KV (few, long rows: the prefix-cache-hit form q_len << k_len): when the grid
 // would leave most SMs idle, `kv_splits` CTAs share one (sequence, head, 256 rows), each takes a
 // contiguous range of key tiles and writes un-normalised (O, m, l) partials to a caller-provided
@@ -49,7 +54,7 @@ struct PrefillUmmaParams {
   int64_t out_stride;
   int H, G, block_size, bt_stride;
   int kv_rows_box;   // rows per K/V TMA op (128 packed; min(block_size, 128) paged)
-  int kv_split;      // 1: each TMA op carries a single 64-wide chunk (paged, rows_box < 128)
+  int k_split, v_split;   // 1: each TMA op carries a single 64-wide chunk (paged, rows_box < 128)
   int kv_splits;     // CTAs sharing one (sequence, head, 256 rows) along the keys; 1 = no split
   float* part_o;     // kv_splits > 1: [total_q][H][kv_splits][D] un-normalised O
   float* part_ml;    // kv_splits > 1: [total_q][H][kv_splits][2]  (row max in the exp2 domain, row sum)
@@ -58,6 +63,7 @@ struct PrefillUmmaParams {
   // query head (fp32 [H], natural-log units) that joins the softmax denominator without a value
   float cap = 0.f, cap_pre = 0.f;
   const float* sink = nullptr;
+  int window = 0, keep_first = 0;   // window 0: every earlier key
 };
 
 constexpr int kUBM = 128, kUBN = 128;
@@ -68,7 +74,7 @@ constexpr int kUBM = 128, kUBN = 128;
 // shared memory, 256 TMEM columns, 192 threads -> TWO CTAs per SM: the two chains sharing the tensor pipe
 // are independent CTAs, so one CTA's prologue (barrier init, TMEM alloc, Q load) and epilogue run under
 // the other's main loop and the hardware balances 128-row items.
-template <typename T, int D, int QT>
+template <typename T, int DK, int DV, int QT>
 __global__ void __launch_bounds__((4 * QT + 2) * 32, 3 - QT)
 prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                      const __grid_constant__ CUtensorMap tmV, const PrefillUmmaParams p) {
@@ -76,18 +82,19 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   constexpr int kTmaWarp = 4 * QT, kMmaWarp = 4 * QT + 1;
   constexpr uint32_t kTmemCols = QT * 256;      // O[t] at 128 t, S[t] at QT * 128 + 128 t
   constexpr uint32_t kSBase = QT * 128;
-  constexpr int CH = D / 64;                    // 128-byte chunks per head row
+  constexpr int CHK = DK / 64, CHV = DV / 64;   // 128-byte chunks per key / value head row
   constexpr int QPANEL = kUBM * 128;            // bytes of one Q panel (128 rows)
   constexpr int KPANEL = kUBN * 128;            // bytes of one K / V panel (128 rows)
-  constexpr int QTILE = CH * QPANEL;
-  constexpr int KTILE = CH * KPANEL;
+  constexpr int QTILE = CHK * QPANEL;
+  constexpr int KTILE = CHK * KPANEL;
+  constexpr int VTILE = CHV * KPANEL;
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
                                              ~uintptr_t(1023));
   uint8_t* sQ = smem;                            // [QT][QTILE]
   uint8_t* sK = sQ + QT * QTILE;                  // [kUStages][KTILE]
-  uint8_t* sV = sK + kUStages * KTILE;           // [kUStages][KTILE]
-  uint64_t* bars = reinterpret_cast<uint64_t*>(sV + kUStages * KTILE);
+  uint8_t* sV = sK + kUStages * KTILE;           // [kUStages][VTILE]
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sV + kUStages * VTILE);
   uint64_t* q_full = bars;                       // [1]
   uint64_t* k_full = bars + 1;                   // [kUStages]
   uint64_t* v_full = k_full + kUStages;          // [kUStages]
@@ -109,20 +116,28 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   const int kvh = head / p.G;
   const int off = Lk - Lq;
   int n_tiles[2] = {0, 0};
+  // tiles [0, kept) hold the kept first keys; the next `skip` tiles end before the window of this CTA's first row
+  const int kept = p.window > 0 ? (min(p.keep_first, Lk) + kUBN - 1) / kUBN : 0;
+  const int skip = p.window > 0 ? max(0, max(0, m0 + off - p.window + 1) / kUBN - kept) : 0;
 #pragma unroll
   for (int t = 0; t < QT; ++t) {
     const int r0 = m0 + t * kUBM;
     const int n_end = r0 < Lq ? min(Lk, r0 + kUBM + off) : 0;
-    n_tiles[t] = n_end > 0 ? (n_end + kUBN - 1) / kUBN : 0;
+    n_tiles[t] = n_end > 0 ? (n_end + kUBN - 1) / kUBN - skip : 0;
   }
   const int ntq = (QT == 2 && m0 + kUBM < Lq) ? 2 : 1;
   // this CTA's share of the key tiles: [j_lo, j_hi) of the tiles the later query tile needs
   const int nt_all = max(n_tiles[0], n_tiles[1]);
   const int j_lo = (int)((long long)nt_all * split / p.kv_splits);
   const int j_hi = (int)((long long)nt_all * (split + 1) / p.kv_splits);
-  const int NT = j_hi - j_lo;                 // loop trip count; tile index = j_lo + j
+  const int NT = j_hi - j_lo;                 // loop trip count; tile index = j_lo + j, past the kept tiles + skip
+  auto first_key = [&](int j) { return (j_lo + j + (j_lo + j >= kept ? skip : 0)) * kUBN; };
+  bool ends_here[2] = {false, false};         // this split holds the last key tile of query tile t
 #pragma unroll
-  for (int t = 0; t < QT; ++t) n_tiles[t] = max(0, min(n_tiles[t], j_hi) - j_lo);
+  for (int t = 0; t < QT; ++t) {
+    ends_here[t] = n_tiles[t] > j_lo && n_tiles[t] <= j_hi;
+    n_tiles[t] = max(0, min(n_tiles[t], j_hi) - j_lo);
+  }
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
@@ -160,26 +175,28 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         const uint64_t pol_stream = l2_policy_evict_first();
         mbar_expect_tx(q_full, ntq * QTILE);
         for (int t = 0; t < ntq; ++t)
-          tma_load_3d(sQ + t * QTILE, &tmQ, q_full, 0, q0 + m0 + t * kUBM, head * CH, pol_stream);
+          tma_load_3d(sQ + t * QTILE, &tmQ, q_full, 0, q0 + m0 + t * kUBM, head * CHK, pol_stream);
       }
       uint8_t* ring = is_k ? sK : sV;
       uint64_t* full = is_k ? k_full : v_full;
       uint64_t* empty = is_k ? k_empty : v_empty;
+      const int CH = is_k ? CHK : CHV, TILE = is_k ? KTILE : VTILE;
+      const int split_boxes = is_k ? p.k_split : p.v_split;
       for (int j = 0; j < NT; ++j) {
         const int s = j % kUStages;
         mbar_wait(&empty[s], ((j / kUStages) & 1) ^ 1);
-        const int n0 = (j_lo + j) * kUBN;
+        const int n0 = first_key(j);
         if (p.block_tables == nullptr) {
-          mbar_expect_tx(&full[s], KTILE);
-          tma_load_3d(ring + s * KTILE, tm, &full[s], 0, k0 + n0, kvh * CH, pol_keep);
+          mbar_expect_tx(&full[s], TILE);
+          tma_load_3d(ring + s * TILE, tm, &full[s], 0, k0 + n0, kvh * CH, pol_keep);
         } else {
           // Every op of the tile is issued: boxes past the end of the sequence use an out-of-range
           // row, which TMA zero-fills without touching memory -- P is exactly 0 there, but 0 x (stale
           // shared memory that happens to hold an Inf/NaN pattern) would poison O.
           const int rb = p.kv_rows_box;
           const int nops = kUBN / rb;
-          const int per_op = p.kv_split ? CH : 1;
-          const int op_bytes = rb * 128 * (p.kv_split ? 1 : CH);
+          const int per_op = split_boxes ? CH : 1;
+          const int op_bytes = rb * 128 * (split_boxes ? 1 : CH);
           mbar_expect_tx(&full[s], nops * per_op * op_bytes);
           for (int o = 0; o < nops; ++o) {
             const int tok = n0 + o * rb;
@@ -187,8 +204,8 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
             const int blk = tok < Lk ? p.block_tables[(int64_t)seq * p.bt_stride + entry] : -1;
             const int row = blk < 0 ? -(1 << 30) : blk * p.block_size + (tok - entry * p.block_size);
             for (int c = 0; c < per_op; ++c) {
-              const int dst = (p.kv_split ? c * KPANEL : 0) + o * rb * 128;
-              tma_load_3d(ring + s * KTILE + dst, tm, &full[s], 0, row, kvh * CH + c, pol_keep);
+              const int dst = (split_boxes ? c * KPANEL : 0) + o * rb * 128;
+              tma_load_3d(ring + s * TILE + dst, tm, &full[s], 0, row, kvh * CH + c, pol_keep);
             }
           }
         }
@@ -199,7 +216,7 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     // Warp-uniform control flow, loop-invariant descriptor bases + compile-time offsets, one elected
     // lane issues.
     const uint32_t idesc_s = umma::make_idesc<T>(kUBM, kUBN, 0, 0);   // S = Q K^T, both K-major
-    const uint32_t idesc_o = umma::make_idesc<T>(kUBM, D, 0, 1);      // O = P V, P from TMEM, V MN-major
+    const uint32_t idesc_o = umma::make_idesc<T>(kUBM, DV, 0, 1);      // O = P V, P from TMEM, V MN-major
     const uint64_t qd0 = umma::desc_kmajor(smem_u32(sQ));
     const uint64_t kd0 = umma::desc_kmajor(smem_u32(sK));
     const uint64_t vd0 = umma::desc_mnmajor(smem_u32(sV), KPANEL);
@@ -210,7 +227,7 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         const uint64_t kd = umma::desc_advance(kd0, (j % kUStages) * KTILE);
         const uint32_t d = tb + kSBase + t * 128;
 #pragma unroll
-        for (int ks = 0; ks < D / 16; ++ks) {
+        for (int ks = 0; ks < DK / 16; ++ks) {
           const uint64_t ad = umma::desc_advance(qd0, t * QTILE + (ks >> 2) * QPANEL + (ks & 3) * 32);
           const uint64_t bd = umma::desc_advance(kd, (ks >> 2) * KPANEL + (ks & 3) * 32);
           umma::mma_ss(d, ad, bd, idesc_s, ks > 0);
@@ -235,7 +252,7 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       const bool more = j + 1 < NT;
       bool k_ready = false;
       umma::fence_after_sync();
-      const uint64_t vd = umma::desc_advance(vd0, s * KTILE);
+      const uint64_t vd = umma::desc_advance(vd0, s * VTILE);
 #pragma unroll
       for (int t = 0; t < QT; ++t) {
         if (j < n_tiles[t]) {
@@ -293,7 +310,7 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         for (int c = 0; c < 128; ++c)
           sr[c >> 5][c & 31] = __float_as_uint(p.cap * tanh_ex2(__uint_as_float(sr[c >> 5][c & 31]) * p.cap_pre));
       }
-      const int n0 = (j_lo + j) * kUBN;
+      const int n0 = first_key(j);
       // mask (warp-uniform test: does this tile touch the diagonal or the end of the keys?)
       const int warp_row0 = m0 + t * kUBM + (warp & 3) * 32;
       if (n0 + kUBN > Lk || n0 + kUBN - 1 > warp_row0 + off) {
@@ -301,6 +318,12 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
 #pragma unroll
         for (int c = 0; c < 128; ++c)
           if (c > limit) sr[c >> 5][c & 31] = 0xff800000u;   // -inf
+      }
+      if (p.window > 0 && n0 + kUBN > p.keep_first && n0 <= warp_row0 + 31 + off - p.window) {
+        const int low = qrow + off - p.window - n0, keep = p.keep_first - n0;   // hidden: keep <= c <= low
+#pragma unroll
+        for (int c = 0; c < 128; ++c)
+          if (c <= low && c >= keep) sr[c >> 5][c & 31] = 0xff800000u;
       }
       float mx = __uint_as_float(sr[0][0]);
 #pragma unroll
@@ -313,7 +336,7 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
           mbar_wait(&o_full[t], (j - 1) & 1);             // PV[t](j-1) landed
           umma::fence_after_sync();
 #pragma unroll
-          for (int c0 = 0; c0 < D; c0 += 16) {     // 16 columns at a time: the S row stays in registers
+          for (int c0 = 0; c0 < DV; c0 += 16) {    // 16 columns at a time: the S row stays in registers
             uint32_t orr[16];
             umma::ld16(o_addr + c0, orr);
             umma::wait_ld();
@@ -348,14 +371,17 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       }
       l_run += sum;
     }
-    // the sink joins the denominator once: in the split that holds the first keys
-    if (p.sink != nullptr && split == 0 && nt > 0 && m_ref != -INFINITY)
-      l_run += ex2_approx(p.sink[head] * kLog2e - m_ref * sl2);
+    // the sink joins the denominator once: in the split that holds the query tile's last keys (never an empty one)
+    if (p.sink != nullptr && ends_here[t]) {
+      const float sink2 = p.sink[head] * kLog2e;
+      if (m_ref == -INFINITY) m_ref = sink2 / sl2, l_run = 1.f;      // no key of this split is visible to the row
+      else l_run += ex2_approx(sink2 - m_ref * sl2);
+    }
     // ---- epilogue: O / l -> global, or (split-KV) the un-normalised partial -> workspace
     if (m0 + t * kUBM < Lq) {
-      T* orow = reinterpret_cast<T*>(p.out) + (int64_t)(q0 + qrow) * p.out_stride + (int64_t)head * D;
+      T* orow = reinterpret_cast<T*>(p.out) + (int64_t)(q0 + qrow) * p.out_stride + (int64_t)head * DV;
       const int64_t pidx = ((int64_t)(q0 + qrow) * p.H + head) * p.kv_splits + split;
-      float* prow = p.part_o + pidx * D;
+      float* prow = p.part_o + pidx * DV;
       const bool split_out = p.kv_splits > 1;
       if (split_out && qrow < Lq) {
         p.part_ml[pidx * 2] = (nt > 0 && m_ref != -INFINITY) ? m_ref * sl2 : -INFINITY;
@@ -366,7 +392,7 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         umma::fence_after_sync();
         const float inv = split_out ? 1.f : (l_run > 0.f ? 1.f / l_run : 0.f);
 #pragma unroll
-        for (int c0 = 0; c0 < D; c0 += 32) {
+        for (int c0 = 0; c0 < DV; c0 += 32) {
           uint32_t orr[32];
           umma::ld32(o_addr + c0, orr);
           umma::wait_ld();
@@ -390,9 +416,9 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         }
       } else if (qrow < Lq) {
         if (split_out) {
-          for (int c = 0; c < D; c += 4) *reinterpret_cast<uint4*>(prow + c) = make_uint4(0, 0, 0, 0);
+          for (int c = 0; c < DV; c += 4) *reinterpret_cast<uint4*>(prow + c) = make_uint4(0, 0, 0, 0);
         } else {
-          for (int c = 0; c < D; c += 8) *reinterpret_cast<uint4*>(orow + c) = make_uint4(0, 0, 0, 0);
+          for (int c = 0; c < DV; c += 8) *reinterpret_cast<uint4*>(orow + c) = make_uint4(0, 0, 0, 0);
         }
       }
     }
@@ -436,13 +462,13 @@ prefill_combine_kernel(T* __restrict__ out, int64_t out_stride, const float* __r
   for (int i = 0; i < V; i += 2) *reinterpret_cast<uint32_t*>(orow + i) = pack2<T>(acc[i] * inv, acc[i + 1] * inv);
 }
 
-template <typename T, int D, int QT>
+template <typename T, int DK, int DV, int QT>
 static int prefill_umma_launch_t(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv,
                                  const PrefillUmmaParams& p, int num_seqs, int max_seqlen_q, int total_q,
                                  cudaStream_t stream) {
-  constexpr int CH = D / 64;
-  constexpr size_t smem = 1024 + QT * CH * kUBM * 128 + 2 * QT * CH * kUBN * 128 + 32 * 8 + 16;
-  auto kern = prefill_umma_kernel<T, D, QT>;
+  constexpr int CHK = DK / 64, CHV = DV / 64;
+  constexpr size_t smem = 1024 + QT * CHK * kUBM * 128 + QT * (CHK + CHV) * kUBN * 128 + 32 * 8 + 16;
+  auto kern = prefill_umma_kernel<T, DK, DV, QT>;
   static bool attr_set = false;
   if (!attr_set) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -454,7 +480,7 @@ static int prefill_umma_launch_t(const CUtensorMap& mq, const CUtensorMap& mk, c
   launch_pdl(kern, grid, dim3((4 * QT + 2) * 32), smem, stream, mq, mk, mv, p);
   if (p.kv_splits > 1) {
     const int64_t items = (int64_t)total_q * p.H;
-    launch_pdl(prefill_combine_kernel<T, D>, dim3((unsigned)((items + 7) / 8)), dim3(256), 0, stream,
+    launch_pdl(prefill_combine_kernel<T, DV>, dim3((unsigned)((items + 7) / 8)), dim3(256), 0, stream,
                reinterpret_cast<T*>(p.out), p.out_stride, (const float*)p.part_o, (const float*)p.part_ml,
                items, p.H, p.kv_splits);
   }
@@ -486,27 +512,27 @@ int prefill_kv_splits(int num_seqs, int H, int max_seqlen_q, int max_seqlen_k, i
 static int g_forced_query_tiles = 0;
 void prefill_force_query_tiles(int qt) { g_forced_query_tiles = qt; }
 
-int prefill_query_tiles(int num_seqs, int H, int max_seqlen_q, int D) {
+int prefill_query_tiles(int num_seqs, int H, int max_seqlen_q, int D, int span) {
   if (g_forced_query_tiles) return g_forced_query_tiles;
   const int64_t ctas2 = (int64_t)((max_seqlen_q + 2 * kUBM - 1) / (2 * kUBM)) * H * num_seqs;
   if (ctas2 * 2 <= 148) return 2;                 // key-split territory (prefill_kv_splits)
-  return (D == 128 && max_seqlen_q >= 2048) ? 2 : 1;
+  return (D == 128 && max_seqlen_q >= 2048 && span >= 2048) ? 2 : 1;   // span: tokens along the keys a row walks over
 }
 
 // Entry used by b200_prefill_varlen_attn (prefill_attn.cu). Returns B200_ERR_UNSUPPORTED when the
 // strides cannot be described by a TMA map (caller falls back to the mma.sync kernel).
 int prefill_umma_launch(void* out, const void* q, const void* k, const void* v,
                          const int32_t* cu_q, const int32_t* cu_k, int num_seqs, int total_q,
-                         int total_k, int max_seqlen_q, int H, int Hkv, int D, int64_t q_stride,
+                         int total_k, int max_seqlen_q, int H, int Hkv, int DK, int DV, int64_t q_stride,
                          int64_t k_stride, int64_t v_stride, int64_t out_stride,
                         const int32_t* block_tables, int bt_stride, int num_blocks, int block_size,
                         float scale, int dtype, void* workspace, int64_t workspace_bytes, int max_seqlen_k,
-                        cudaStream_t stream, float softcap, const float* sink) {
+                        cudaStream_t stream, float softcap, const float* sink, int window, int keep_first) {
   if (q_stride % 8 != 0 || out_stride % 8 != 0 || !aligned16(out)) return B200_ERR_UNSUPPORTED;
   if (total_q <= 0) return B200_ERR_UNSUPPORTED;
-  const int CH = D / 64;
+  const int CHK = DK / 64, CHV = DV / 64;
   CUtensorMap mq, mk, mv;
-  int rc = get_panel_map(q, total_q, q_stride * 2, H * CH, kUBM, CH, dtype, &mq);
+  int rc = get_panel_map(q, total_q, q_stride * 2, H * CHK, kUBM, CHK, dtype, &mq);
   if (rc != B200_OK) return rc;
   PrefillUmmaParams p;
   p.cu_q = cu_q, p.cu_k = cu_k, p.block_tables = block_tables;
@@ -515,39 +541,43 @@ int prefill_umma_launch(void* out, const void* q, const void* k, const void* v,
   p.scale_log2 = scale * 1.4426950408889634f;
   if (softcap > 0.f) p.cap = softcap, p.cap_pre = scale / softcap;
   p.sink = sink;
-  const int qt = prefill_query_tiles(num_seqs, H, max_seqlen_q, D);
+  p.window = window, p.keep_first = window > 0 ? keep_first : 0;
+  // keys that a 128-row query tile can see at most: what the choice of layout and of key splits is made on
+  if (window > 0 && max_seqlen_k > window + p.keep_first + 3 * kUBM) max_seqlen_k = window + p.keep_first + 3 * kUBM;
+  const int qt = prefill_query_tiles(num_seqs, H, max_seqlen_q, DV, window > 0 ? max_seqlen_k : max_seqlen_q);
   p.kv_splits = (workspace != nullptr && (reinterpret_cast<uintptr_t>(workspace) & 15) == 0)
-                    ? prefill_kv_splits(num_seqs, H, max_seqlen_q, max_seqlen_k, total_q, D, workspace_bytes, qt)
+                    ? prefill_kv_splits(num_seqs, H, max_seqlen_q, max_seqlen_k, total_q, DV, workspace_bytes, qt)
                     : 1;
   p.part_o = reinterpret_cast<float*>(workspace);
-  p.part_ml = p.part_o + (int64_t)total_q * H * p.kv_splits * D;
+  p.part_ml = p.part_o + (int64_t)total_q * H * p.kv_splits * DV;
   if (block_tables == nullptr) {
     if (k_stride % 8 != 0 || v_stride % 8 != 0 || total_k <= 0) return B200_ERR_UNSUPPORTED;
-    p.kv_rows_box = kUBN, p.kv_split = 0;
-    rc = get_panel_map(k, total_k, k_stride * 2, Hkv * CH, kUBN, CH, dtype, &mk);
+    p.kv_rows_box = kUBN, p.k_split = p.v_split = 0;
+    rc = get_panel_map(k, total_k, k_stride * 2, Hkv * CHK, kUBN, CHK, dtype, &mk);
     if (rc != B200_OK) return rc;
-    rc = get_panel_map(v, total_k, v_stride * 2, Hkv * CH, kUBN, CH, dtype, &mv);
+    rc = get_panel_map(v, total_k, v_stride * 2, Hkv * CHV, kUBN, CHV, dtype, &mv);
     if (rc != B200_OK) return rc;
   } else {
     if (block_size % 16 != 0 || (block_size < kUBN && kUBN % block_size != 0) ||
         (block_size > kUBN && block_size % kUBN != 0))
       return B200_ERR_UNSUPPORTED;
     p.kv_rows_box = block_size < kUBN ? block_size : kUBN;
-    p.kv_split = p.kv_rows_box < kUBN ? 1 : 0;
+    p.k_split = p.v_split = p.kv_rows_box < kUBN ? 1 : 0;
     const int64_t rows = (int64_t)num_blocks * block_size;
-    const int cbox = p.kv_split ? 1 : CH;
-    rc = get_panel_map(k, rows, (int64_t)Hkv * D * 2, Hkv * CH, p.kv_rows_box, cbox, dtype, &mk);
+    rc = get_panel_map(k, rows, (int64_t)Hkv * DK * 2, Hkv * CHK, p.kv_rows_box, p.k_split ? 1 : CHK, dtype, &mk);
     if (rc != B200_OK) return rc;
-    rc = get_panel_map(v, rows, (int64_t)Hkv * D * 2, Hkv * CH, p.kv_rows_box, cbox, dtype, &mv);
+    rc = get_panel_map(v, rows, (int64_t)Hkv * DV * 2, Hkv * CHV, p.kv_rows_box, p.v_split ? 1 : CHV, dtype, &mv);
     if (rc != B200_OK) return rc;
   }
-#define B200_PREFILL_DISPATCH(T, DD)                                                                   \
-  (qt == 2 ? prefill_umma_launch_t<T, DD, 2>(mq, mk, mv, p, num_seqs, max_seqlen_q, total_q, stream) \
-           : prefill_umma_launch_t<T, DD, 1>(mq, mk, mv, p, num_seqs, max_seqlen_q, total_q, stream))
-  if (dtype == B200_DTYPE_BF16)
-    return D == 128 ? B200_PREFILL_DISPATCH(__nv_bfloat16, 128) : B200_PREFILL_DISPATCH(__nv_bfloat16, 64);
-  return D == 128 ? B200_PREFILL_DISPATCH(__half, 128) : B200_PREFILL_DISPATCH(__half, 64);
+#define B200_PREFILL_QT(T, K, V)                                                                          \
+  (qt == 2 ? prefill_umma_launch_t<T, K, V, 2>(mq, mk, mv, p, num_seqs, max_seqlen_q, total_q, stream) \
+           : prefill_umma_launch_t<T, K, V, 1>(mq, mk, mv, p, num_seqs, max_seqlen_q, total_q, stream))
+#define B200_PREFILL_DISPATCH(T)                                                      \
+  (DK == 128 ? (DV == 128 ? B200_PREFILL_QT(T, 128, 128) : B200_PREFILL_QT(T, 128, 64)) \
+             : (DV == 128 ? B200_PREFILL_QT(T, 64, 128) : B200_PREFILL_QT(T, 64, 64)))
+  return dtype == B200_DTYPE_BF16 ? B200_PREFILL_DISPATCH(__nv_bfloat16) : B200_PREFILL_DISPATCH(__half);
 #undef B200_PREFILL_DISPATCH
+#undef B200_PREFILL_QT
 }
 
 }  // namespace b200

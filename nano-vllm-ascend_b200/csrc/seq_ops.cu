@@ -6,10 +6,10 @@
 //   unitnorm_temp_cache  per-head unit RMS of q and k, position-dependent query temperature, K/V scatter
 //   gated_norm           (grouped) RMS norm and an output gate, in either order
 //   act_and_mul          act(gate) * up for the gated feed-forward
-//   act_only             act(x) for a feed-forward without a gate (silu, relu, gelu, squared relu)
-//   norm_residual        r (+)= norm(y [+ y2]); h = r in the element type: a norm on the sublayer's OUTPUT (layer norm
-//                        with weight and bias, or RMS norm), the rows of y / y2 optionally gathered by index
-//                        (token embedding + learned position + norm in one launch)
+//   act_only             act(x) for a feed-forward without a gate (silu, relu, gelu, squared relu) or a low-rank path (tanh)
+//   norm_residual        r (+)= norm(y [+ y2]), or r = norm(carry r + y [+ y2]); h = r in the element type: a norm on the
+//                        sublayer's OUTPUT or on the SUM (layer norm with weight and bias, or RMS norm), the rows of y / y2
+//                        optionally gathered by index (token embedding + learned position + norm in one launch)
 //   rownorm_cache        RMS norm of q and of k over the WHOLE projection (all heads at once), K/V scatter
 //   gate_prep            what a gated linear recurrence with tied input reads: silu(q) and the lower-bounded forget
 //                        gate l + (1 - l) sigmoid(f + bias), both fp32
@@ -20,7 +20,10 @@
 //   rotary_table         cos / sin of position * frequency for a table of frequencies (fp64 angles), times a magnitude
 //   rope_mix_cache       rotation of part of every q and k head by that table, values blended with another layer's
 //                        values of the same token, K/V scatter
+//   norm_rope_cache      per-head RMS norm of q and k with a weight shared by the heads, rotation of part of every head by
+//                        that table, K/V scatter
 //   head_gate            every head of a row times sigmoid of one logit per (token, head)
+//   token_shift          several mixes of a row with the row of the token before, the last row of a sequence carried in a slot
 //
 // All are bound by HBM traffic; arithmetic is fp32 whatever the element type. Shapes are free: no
 // multiple-of-8 rule, so that small and odd models run (a 16-byte path is taken where rows allow it).
@@ -383,26 +386,27 @@ unitnorm_temp_cache_vec_kernel(T* __restrict__ qkv, int64_t stride, const int64_
 // y: [rows, n] fp32 or T; gate: [rows, n] T with a row stride. One CTA per (row, group of n / groups):
 //   gate_first: out = norm_group(y * act(gate)) * w          (gate, then norm)
 //   else      : out = norm_group(y) * w * act(gate)          (norm, then gate)
-// w == nullptr: no norm at all, out = y * act(gate). gate_act: 0 sigmoid, 1 silu, 2 no gate (gate may be null).
+// w == nullptr: no norm at all, out = y * act(gate). gate_act: 0 sigmoid, 1 silu, 2 no gate (gate may be null). The result
+// is multiplied by out_scale before it is rounded, and written with its own row stride (a slice of a wider row).
 template <typename T, typename Y>
 __global__ void __launch_bounds__(256)
 gated_norm_kernel(T* __restrict__ out, const Y* __restrict__ y, const T* __restrict__ gate,
                   int64_t gate_stride, const float* __restrict__ w, float eps, int n, int groups,
-                  int gate_first, int gate_act) {
+                  int gate_first, int gate_act, int64_t out_stride, float out_scale) {
   __shared__ float red[32];
   pdl_wait();
   const int64_t r = blockIdx.x;
   const int len = n / groups, lo = blockIdx.y * len;
   const Y* yr = y + r * n + lo;
   const T* gr = gate + r * gate_stride + lo;
-  T* o = out + r * n + lo;
+  T* o = out + r * out_stride + lo;
   auto gate_at = [&](int i) -> float {
     if (gate_act == 2) return 1.f;
     const float g = to_f32<T>(gr[i]);
     return gate_act == 1 ? silu_f(g) : sigmoid_f(g);
   };
   if (w == nullptr) {
-    for (int i = threadIdx.x; i < len; i += blockDim.x) o[i] = from_f32<T>(to_f32<Y>(yr[i]) * gate_at(i));
+    for (int i = threadIdx.x; i < len; i += blockDim.x) o[i] = from_f32<T>(to_f32<Y>(yr[i]) * gate_at(i) * out_scale);
     return;
   }
   float ss = 0.f;
@@ -416,7 +420,7 @@ gated_norm_kernel(T* __restrict__ out, const Y* __restrict__ y, const T* __restr
     float v = to_f32<Y>(yr[i]);
     if (gate_first) v = v * gate_at(i) * rstd * w[lo + i];
     else v = v * rstd * w[lo + i] * gate_at(i);
-    o[i] = from_f32<T>(v);
+    o[i] = from_f32<T>(v * out_scale);
   }
 }
 
@@ -461,14 +465,14 @@ template <typename T, typename Y>
 __global__ void __launch_bounds__(256)
 gated_norm_vec_kernel(T* __restrict__ out, const Y* __restrict__ y, const T* __restrict__ gate,
                       int64_t gate_stride, const float* __restrict__ w, float eps, int n, int groups,
-                      int gate_first, int gate_act) {
+                      int gate_first, int gate_act, int64_t out_stride, float out_scale) {
   __shared__ float red[32];
   pdl_wait();
   const int64_t r = blockIdx.x;
   const int len = n / groups, lo = blockIdx.y * len;
   const Y* yr = y + r * n + lo;
   const T* gr = gate + r * gate_stride + lo;
-  T* o = out + r * n + lo;
+  T* o = out + r * out_stride + lo;
   constexpr int kV = 2;                               // up to 256 * 2 * 8 = 4096 elements per group in registers
   float val[kV][8], gv[kV][8];
   float ss = 0.f;
@@ -502,6 +506,8 @@ gated_norm_vec_kernel(T* __restrict__ out, const Y* __restrict__ y, const T* __r
 #pragma unroll
         for (int e = 0; e < 8; ++e) ov[e] = val[m][e];
       }
+#pragma unroll
+      for (int e = 0; e < 8; ++e) ov[e] *= out_scale;
       store8<T>(o + vi * 8, ov);
     }
   }
@@ -514,7 +520,7 @@ template <typename T, typename Y>
 __global__ void __launch_bounds__(256)
 gated_norm_warp_kernel(T* __restrict__ out, const Y* __restrict__ y, const T* __restrict__ gate,
                        int64_t gate_stride, const float* __restrict__ w, float eps, int64_t rows, int n, int groups,
-                       int gate_first, int gate_act, int gl) {
+                       int gate_first, int gate_act, int gl, int64_t out_stride, float out_scale) {
   pdl_wait();
   const int lane = threadIdx.x & 31, sub = lane % gl;
   const int64_t warp = (int64_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -524,7 +530,7 @@ gated_norm_warp_kernel(T* __restrict__ out, const Y* __restrict__ y, const T* __
   const int len = n / groups, lo = live ? (int)(unit % groups) * len : 0;
   const Y* yr = y + r * n + lo;
   const T* gr = gate + r * gate_stride + lo;
-  T* o = out + r * n + lo;
+  T* o = out + r * out_stride + lo;
   constexpr int kV = 2;
   float val[kV][8], gv[kV][8];
   float ss = 0.f;
@@ -551,14 +557,15 @@ gated_norm_warp_kernel(T* __restrict__ out, const Y* __restrict__ y, const T* __
       float ov[8], wv[8];
       load8<float>(w + lo + vi * 8, wv);
 #pragma unroll
-      for (int e = 0; e < 8; ++e) ov[e] = gate_first ? val[m][e] * rstd * wv[e] : val[m][e] * rstd * wv[e] * gv[m][e];
+      for (int e = 0; e < 8; ++e)
+        ov[e] = out_scale * (gate_first ? val[m][e] * rstd * wv[e] : val[m][e] * rstd * wv[e] * gv[m][e]);
       store8<T>(o + vi * 8, ov);
     }
   }
 }
 
 // ------------------------------------------------------------------ act(x) without a gate
-// act: 0 silu, 1 relu, 2 gelu (tanh form), 3 squared relu.
+// act: 0 silu, 1 relu, 2 gelu (tanh form), 3 squared relu, 4 tanh.
 __device__ __forceinline__ float act_f(float x, int act) {
   if (act == 1) return fmaxf(x, 0.f);
   if (act == 2) return gelu_tanh_f(x);
@@ -566,6 +573,7 @@ __device__ __forceinline__ float act_f(float x, int act) {
     const float r = fmaxf(x, 0.f);
     return r * r;
   }
+  if (act == 4) return tanhf(x);
   return silu_f(x);
 }
 
@@ -592,14 +600,16 @@ act_only_vec_kernel(T* __restrict__ out, const T* __restrict__ x, int64_t total8
 
 // ------------------------------------------------------------------ a norm on the sublayer's output, then the residual
 // u = y[iy] (+ y2[iy2]) in fp32; n = norm(u): kind 0 (u - mean) / sqrt(var + eps) * w + b, kind 1 u / sqrt(mean u^2 + eps)
-// * (offset + w); r <- accumulate ? r + n : n; h <- r in the element type (h may be null). iy / iy2: row r itself, or
-// index[r] clamped to the table's rows (a token id, a position). Dynamic smem: hidden floats.
+// * (offset + w); accumulate 0: r <- n; 1: r <- r + n; 2 (a norm after the sum): u also has carry * r, r <- n. h <- r in
+// the element type (h may be null). iy / iy2: row r itself, or index[r] clamped to the table's rows (a token id, a
+// position). Dynamic smem: hidden floats.
 template <typename T>
 __global__ void __launch_bounds__(256)
 norm_residual_kernel(T* __restrict__ h, float* __restrict__ res, const T* __restrict__ y,
                      const int64_t* __restrict__ y_index, int64_t y_rows, const T* __restrict__ y2,
                      const int64_t* __restrict__ y2_index, int64_t y2_rows, const float* __restrict__ w,
-                     const float* __restrict__ b, float eps, float offset, int kind, int accumulate, int hidden) {
+                     const float* __restrict__ b, float eps, float offset, int kind, int accumulate, float carry,
+                     int hidden) {
   extern __shared__ float row[];
   __shared__ float red[32];
   pdl_wait();
@@ -613,10 +623,12 @@ norm_residual_kernel(T* __restrict__ h, float* __restrict__ res, const T* __rest
     if (y2_index != nullptr) i2 = i2 < 0 ? 0 : (i2 >= y2_rows ? y2_rows - 1 : i2);
     y2r = y2 + i2 * hidden;
   }
+  float* rr = res + r * hidden;
   float s1 = 0.f;
   for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
     float v = to_f32<T>(yr[i]);
     if (y2r != nullptr) v += to_f32<T>(y2r[i]);
+    if (accumulate == 2) v += carry * rr[i];
     row[i] = v;
     s1 += kind == 0 ? v : v * v;
   }
@@ -633,11 +645,10 @@ norm_residual_kernel(T* __restrict__ h, float* __restrict__ res, const T* __rest
   } else {
     rstd = 1.0f / sqrtf(s1 + eps);
   }
-  float* rr = res + r * hidden;
   T* hr = h != nullptr ? h + r * hidden : nullptr;
   for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
     float n = kind == 0 ? (row[i] - mean) * rstd * w[i] + (b != nullptr ? b[i] : 0.f) : row[i] * rstd * (offset + w[i]);
-    if (accumulate) n += rr[i];
+    if (accumulate == 1) n += rr[i];
     rr[i] = n;
     if (hr != nullptr) hr[i] = from_f32<T>(n);
   }
@@ -650,7 +661,8 @@ __global__ void __launch_bounds__(256)
 norm_residual_vec_kernel(T* __restrict__ h, float* __restrict__ res, const T* __restrict__ y,
                          const int64_t* __restrict__ y_index, int64_t y_rows, const T* __restrict__ y2,
                          const int64_t* __restrict__ y2_index, int64_t y2_rows, const float* __restrict__ w,
-                         const float* __restrict__ b, float eps, float offset, int kind, int accumulate, int hidden) {
+                         const float* __restrict__ b, float eps, float offset, int kind, int accumulate, float carry,
+                         int hidden) {
   __shared__ float red[32];
   pdl_wait();
   const int nvec = hidden / 8;
@@ -664,6 +676,7 @@ norm_residual_vec_kernel(T* __restrict__ h, float* __restrict__ res, const T* __
     if (y2_index != nullptr) i2 = i2 < 0 ? 0 : (i2 >= y2_rows ? y2_rows - 1 : i2);
     y2r = y2 + i2 * hidden;
   }
+  float* rr = res + r * hidden;
   float val[kResVecs][8];
   float s1 = 0.f;
 #pragma unroll
@@ -676,6 +689,12 @@ norm_residual_vec_kernel(T* __restrict__ h, float* __restrict__ res, const T* __
         load8<T>(y2r + vi * 8, t);
 #pragma unroll
         for (int e = 0; e < 8; ++e) val[n][e] += t[e];
+      }
+      if (accumulate == 2) {
+        float t[8];
+        load8<float>(rr + vi * 8, t);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) val[n][e] += carry * t[e];
       }
 #pragma unroll
       for (int e = 0; e < 8; ++e) s1 += kind == 0 ? val[n][e] : val[n][e] * val[n][e];
@@ -701,7 +720,6 @@ norm_residual_vec_kernel(T* __restrict__ h, float* __restrict__ res, const T* __
   } else {
     rstd = 1.0f / sqrtf(s1 + eps);
   }
-  float* rr = res + r * hidden;
   T* hr = h != nullptr ? h + r * hidden : nullptr;
 #pragma unroll
   for (int n = 0; n < kResVecs; ++n) {
@@ -710,12 +728,12 @@ norm_residual_vec_kernel(T* __restrict__ h, float* __restrict__ res, const T* __
       float wv[8], bv[8], ov[8];
       load8<float>(w + vi * 8, wv);
       if (kind == 0 && b != nullptr) load8<float>(b + vi * 8, bv);
-      if (accumulate) load8<float>(rr + vi * 8, ov);
+      if (accumulate == 1) load8<float>(rr + vi * 8, ov);
 #pragma unroll
       for (int e = 0; e < 8; ++e) {
         const float nrm = kind == 0 ? (val[n][e] - mean) * rstd * wv[e] + (b != nullptr ? bv[e] : 0.f)
                                     : val[n][e] * rstd * (offset + wv[e]);
-        ov[e] = accumulate ? ov[e] + nrm : nrm;
+        ov[e] = accumulate == 1 ? ov[e] + nrm : nrm;
       }
       store8<float>(rr + vi * 8, ov);
       if (hr != nullptr) store8<T>(hr + vi * 8, ov);
@@ -1094,6 +1112,173 @@ rope_mix_cache_vec_kernel(T* __restrict__ qkv, int64_t stride, const float2* __r
   if (slot >= 0 && c >= nq) store8<T>(k_cache + slot * (int64_t)nk + (c - nq), f);
 }
 
+// qkv: [T, H*dim | G*dim | G*vdim] (row stride given). Every q and k head: divided by its root mean square (eps inside the
+// root), times a weight [dim] shared by the q (or k) heads; then its first `dims` columns are rotated by the table, in pairs
+// (2i, 2i+1) or (i, i + dims/2), and the result is rounded once, in place. k and v rows are also stored at their cache
+// slot when caches are bound. One warp per (token, head of q | k | v); fp32 arithmetic.
+template <typename T>
+__global__ void __launch_bounds__(256)
+norm_rope_cache_kernel(T* __restrict__ qkv, int64_t stride, const float* __restrict__ wq, const float* __restrict__ wk,
+                       float eps, const float2* __restrict__ table, int dims, int interleaved, T* __restrict__ k_cache,
+                       T* __restrict__ v_cache, const int* __restrict__ slots, int slot_pairs, int block_size,
+                       int num_tokens, int H, int G, int dim, int vdim) {
+  pdl_wait();
+  const int lane = threadIdx.x & 31;
+  const int64_t unit = (int64_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  const int per_tok = H + 2 * G;
+  if (unit >= (int64_t)num_tokens * per_tok) return;
+  const int t = (int)(unit / per_tok), u = (int)(unit % per_tok);
+  int64_t slot = -1;
+  if (k_cache != nullptr && u >= H)
+    slot = slot_pairs ? (int64_t)slots[2 * t] * block_size + slots[2 * t + 1] : (int64_t)slots[t];
+  T* row = qkv + (int64_t)t * stride;
+  if (u >= H + G) {                                  // a value head: copy only
+    if (slot < 0) return;
+    const int g = u - H - G;
+    const T* src = row + (int64_t)(H + G) * dim + (int64_t)g * vdim;
+    T* dst = v_cache + slot * ((int64_t)G * vdim) + (int64_t)g * vdim;
+    for (int i = lane; i < vdim; i += 32) dst[i] = src[i];
+    return;
+  }
+  T* x = row + (int64_t)u * dim;                     // q heads then k heads, both `dim` wide
+  const float* w = u < H ? wq : wk;
+  float ss = 0.f;
+  for (int i = lane; i < dim; i += 32) {
+    const float v = to_f32<T>(x[i]);
+    ss += v * v;
+  }
+  const float rstd = 1.0f / sqrtf(warp_sum(ss) / (float)dim + eps);
+  T* dst = (u >= H && slot >= 0) ? k_cache + slot * ((int64_t)G * dim) + (int64_t)(u - H) * dim : nullptr;
+  const int half = dims / 2;
+  const float2* cs = table + (int64_t)t * half;
+  for (int i = lane; i < half; i += 32) {
+    const int a = interleaved ? 2 * i : i, b = interleaved ? 2 * i + 1 : i + half;
+    const float2 r = cs[i];
+    const float p = to_f32<T>(x[a]) * rstd * w[a], q = to_f32<T>(x[b]) * rstd * w[b];
+    const T ra = from_f32<T>(p * r.x - q * r.y), rb = from_f32<T>(q * r.x + p * r.y);
+    x[a] = ra, x[b] = rb;
+    if (dst != nullptr) dst[a] = ra, dst[b] = rb;
+  }
+  for (int i = dims + lane; i < dim; i += 32) {
+    const T v = from_f32<T>(to_f32<T>(x[i]) * rstd * w[i]);
+    x[i] = v;
+    if (dst != nullptr) dst[i] = v;
+  }
+}
+
+// 16-byte form (neighbouring pairs; dim = 8 * GL with GL a power of two up to 32; dims, vdim multiples of 8; 16-byte
+// aligned rows): GL adjacent lanes share one head, 32 / GL heads per warp
+template <typename T, int GL>
+__global__ void __launch_bounds__(256)
+norm_rope_cache_vec_kernel(T* __restrict__ qkv, int64_t stride, const float* __restrict__ wq,
+                           const float* __restrict__ wk, float eps, const float2* __restrict__ table, int dims,
+                           T* __restrict__ k_cache, T* __restrict__ v_cache, const int* __restrict__ slots,
+                           int slot_pairs, int block_size, int num_tokens, int H, int G, int vdim) {
+  pdl_wait();
+  constexpr int dim = GL * 8, UPW = 32 / GL;
+  const int lane = threadIdx.x & 31, gl = lane % GL;
+  const int64_t unit = ((int64_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5)) * UPW + lane / GL;
+  const int per_tok = H + 2 * G;
+  const bool live = unit < (int64_t)num_tokens * per_tok;
+  const int t = live ? (int)(unit / per_tok) : 0, u = live ? (int)(unit % per_tok) : 0;
+  int64_t slot = -1;
+  if (live && k_cache != nullptr && u >= H)
+    slot = slot_pairs ? (int64_t)slots[2 * t] * block_size + slots[2 * t + 1] : (int64_t)slots[t];
+  T* row = qkv + (int64_t)t * stride;
+  const bool is_v = u >= H + G;
+  if (live && is_v && slot >= 0) {
+    const T* src = row + (int64_t)(H + G) * dim + (int64_t)(u - H - G) * vdim;
+    T* dst = v_cache + slot * ((int64_t)G * vdim) + (int64_t)(u - H - G) * vdim;
+    for (int vi = gl; vi * 8 < vdim; vi += GL) {
+      float tmp[8];
+      load8<T>(src + vi * 8, tmp);
+      store8<T>(dst + vi * 8, tmp);
+    }
+  }
+  const bool normed = live && !is_v;
+  T* x = row + (int64_t)u * dim + gl * 8;
+  float f[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+  if (normed) load8<T>(x, f);
+  float ss = 0.f;
+#pragma unroll
+  for (int e = 0; e < 8; ++e) ss += f[e] * f[e];
+#pragma unroll
+  for (int off = GL / 2; off > 0; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
+  if (!normed) return;
+  const float rstd = 1.0f / sqrtf(ss / (float)dim + eps);
+  float wv[8];
+  load8<float>((u < H ? wq : wk) + gl * 8, wv);
+#pragma unroll
+  for (int e = 0; e < 8; ++e) f[e] *= rstd * wv[e];
+  if (gl * 8 < dims) {
+    const float4* cs = reinterpret_cast<const float4*>(table + (int64_t)t * (dims / 2) + gl * 4);
+    const float4 a = cs[0], b = cs[1];               // (cos, sin) of four neighbouring pairs
+    const float co[4] = {a.x, a.z, b.x, b.z}, si[4] = {a.y, a.w, b.y, b.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float p = f[2 * i], q = f[2 * i + 1];
+      f[2 * i] = p * co[i] - q * si[i];
+      f[2 * i + 1] = q * co[i] + p * si[i];
+    }
+  }
+  store8<T>(x, f);
+  if (u >= H && slot >= 0) store8<T>(k_cache + slot * ((int64_t)G * dim) + (int64_t)(u - H) * dim + gl * 8, f);
+}
+
+// ------------------------------------------------------------------ mixes of a row with the row of the token before
+// out[m][t] = h_t + (h_(t-1) - h_t) * mu[m], m < M; h_(-1) is zero at a sequence's start, else the row that the step
+// before left in state[slot] ([W], element type). A thread owns one channel (VEC: 8) of kShiftSeg consecutive tokens of
+// one sequence; the thread of a sequence's first segment reads the carried row and then writes the new one, so no other
+// thread can see a half-updated row.
+constexpr int kShiftSeg = 8;
+
+template <typename T, int V>
+__global__ void __launch_bounds__(128)
+token_shift_kernel(T* __restrict__ out, int64_t mix_stride, const T* __restrict__ h, int64_t h_stride,
+                   const float* __restrict__ mu, int M, T* __restrict__ state, const int* __restrict__ state_slots,
+                   const int* __restrict__ cu_q, const int* __restrict__ cu_k, const int* __restrict__ ctx_lens, int W) {
+  pdl_wait();
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * V;
+  const int s = blockIdx.z;
+  const SeqSpan sp = seq_span(cu_q, cu_k, ctx_lens, s);
+  const int t0 = blockIdx.y * kShiftSeg;
+  if (c >= W || t0 >= sp.q_len) return;
+  auto load = [&](const T* p, float (&f)[V]) {
+    if constexpr (V == 8) load8<T>(p, f);
+    else f[0] = to_f32<T>(*p);
+  };
+  auto store = [&](T* p, const float (&f)[V]) {
+    if constexpr (V == 8) store8<T>(p, f);
+    else *p = from_f32<T>(f[0]);
+  };
+  T* carried = state != nullptr ? state + (int64_t)state_slots[s] * W + c : nullptr;
+  const T* hs = h + (int64_t)sp.q_start * h_stride + c;
+  float prev[V], cur[V], next[V];
+#pragma unroll
+  for (int e = 0; e < V; ++e) prev[e] = 0.f;
+  if (t0 > 0) load(hs + (int64_t)(t0 - 1) * h_stride, prev);
+  else if (carried != nullptr && sp.first_pos() > 0) load(carried, prev);
+  if (t0 == 0 && carried != nullptr) {
+    load(hs + (int64_t)(sp.q_len - 1) * h_stride, next);
+    store(carried, next);
+  }
+  const int t1 = min(t0 + kShiftSeg, sp.q_len);
+  for (int t = t0; t < t1; ++t) {
+    load(hs + (int64_t)t * h_stride, cur);
+    T* o = out + (int64_t)(sp.q_start + t) * W + c;
+    for (int m = 0; m < M; ++m) {
+      float w[V], y[V];
+      if constexpr (V == 8) load8<float>(mu + (int64_t)m * W + c, w);
+      else w[0] = mu[(int64_t)m * W + c];
+#pragma unroll
+      for (int e = 0; e < V; ++e) y[e] = cur[e] + (prev[e] - cur[e]) * w[e];
+      store(o + m * mix_stride, y);
+    }
+#pragma unroll
+    for (int e = 0; e < V; ++e) prev[e] = cur[e];
+  }
+}
+
 // out[t, h, :] = x[t, h, :] * sigmoid(gate[t, h]): one logit per (token, head). In place when out == x.
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -1233,17 +1418,17 @@ extern "C" int b200_unitnorm_temp_cache(void* qkv, int64_t stride, const int64_t
 
 extern "C" int b200_gated_norm(void* out, const void* y, int32_t y_is_f32, const void* gate,
                                int64_t gate_stride, const float* weight, float eps, int32_t rows, int32_t n,
-                               int32_t groups, int32_t gate_first, int32_t gate_act, int32_t dtype,
-                               b200_stream_t stream) {
+                               int32_t groups, int32_t gate_first, int32_t gate_act, int64_t out_stride,
+                               float out_scale, int32_t dtype, b200_stream_t stream) {
   B200_RETURN_IF(rows < 0 || n <= 0 || groups <= 0 || n % groups != 0, B200_ERR_BAD_SHAPE);
   if (rows == 0) return B200_OK;
-  B200_RETURN_IF(gate_act < 0 || gate_act > 2, B200_ERR_BAD_SHAPE);
+  B200_RETURN_IF(gate_act < 0 || gate_act > 2 || out_stride < n, B200_ERR_BAD_SHAPE);
   B200_RETURN_IF(!out || !y || (!gate && gate_act != 2), B200_ERR_NULL_POINTER);
   const dim3 grid(rows, weight ? groups : 1);
   const int g = weight ? groups : 1;
   const int len = n / g;
-  if (len % 8 == 0 && len <= 4096 && n % 8 == 0 && gate_stride % 8 == 0 && aligned16(out) && aligned16(y) &&
-      (!gate || aligned16(gate)) && (!weight || aligned16(weight))) {
+  if (len % 8 == 0 && len <= 4096 && n % 8 == 0 && gate_stride % 8 == 0 && out_stride % 8 == 0 && aligned16(out) &&
+      aligned16(y) && (!gate || aligned16(gate)) && (!weight || aligned16(weight))) {
     if (weight && g > 1 && len <= 512) {               // a norm per head: warps, not CTAs, per group
       int gl = 1;
       while (gl * 8 < len && gl < 32) gl <<= 1;
@@ -1252,10 +1437,12 @@ extern "C" int b200_gated_norm(void* out, const void* y, int32_t y_is_f32, const
       B200_DISPATCH_3(dtype, T, {
         if (y_is_f32)
           launch_pdl(gated_norm_warp_kernel<T, float>, wgrid, dim3(256), 0, (cudaStream_t)stream, (T*)out,
-                     (const float*)y, (const T*)gate, gate_stride, weight, eps, (int64_t)rows, n, g, gate_first, gate_act, gl);
+                     (const float*)y, (const T*)gate, gate_stride, weight, eps, (int64_t)rows, n, g, gate_first, gate_act, gl,
+                     out_stride, out_scale);
         else
           launch_pdl(gated_norm_warp_kernel<T, T>, wgrid, dim3(256), 0, (cudaStream_t)stream, (T*)out, (const T*)y,
-                     (const T*)gate, gate_stride, weight, eps, (int64_t)rows, n, g, gate_first, gate_act, gl);
+                     (const T*)gate, gate_stride, weight, eps, (int64_t)rows, n, g, gate_first, gate_act, gl,
+                     out_stride, out_scale);
       });
       return finish_launch();
     }
@@ -1263,20 +1450,24 @@ extern "C" int b200_gated_norm(void* out, const void* y, int32_t y_is_f32, const
     B200_DISPATCH_3(dtype, T, {
       if (y_is_f32)
         launch_pdl(gated_norm_vec_kernel<T, float>, grid, dim3(threads), 0, (cudaStream_t)stream, (T*)out,
-                   (const float*)y, (const T*)gate, gate_stride, weight, eps, n, g, gate_first, gate_act);
+                   (const float*)y, (const T*)gate, gate_stride, weight, eps, n, g, gate_first, gate_act, out_stride,
+                   out_scale);
       else
         launch_pdl(gated_norm_vec_kernel<T, T>, grid, dim3(threads), 0, (cudaStream_t)stream, (T*)out, (const T*)y,
-                   (const T*)gate, gate_stride, weight, eps, n, g, gate_first, gate_act);
+                   (const T*)gate, gate_stride, weight, eps, n, g, gate_first, gate_act, out_stride,
+                   out_scale);
     });
     return finish_launch();
   }
   B200_DISPATCH_3(dtype, T, {
     if (y_is_f32)
       launch_pdl(gated_norm_kernel<T, float>, grid, dim3(256), 0, (cudaStream_t)stream, (T*)out,
-                 (const float*)y, (const T*)gate, gate_stride, weight, eps, n, g, gate_first, gate_act);
+                 (const float*)y, (const T*)gate, gate_stride, weight, eps, n, g, gate_first, gate_act, out_stride,
+                   out_scale);
     else
       launch_pdl(gated_norm_kernel<T, T>, grid, dim3(256), 0, (cudaStream_t)stream, (T*)out, (const T*)y,
-                 (const T*)gate, gate_stride, weight, eps, n, g, gate_first, gate_act);
+                 (const T*)gate, gate_stride, weight, eps, n, g, gate_first, gate_act, out_stride,
+                   out_scale);
   });
   return finish_launch();
 }
@@ -1304,7 +1495,7 @@ extern "C" int b200_act_and_mul(void* out, const void* x, int32_t rows, int32_t 
 
 extern "C" int b200_act_only(void* out, const void* x, int64_t total, int32_t act, int32_t dtype,
                              b200_stream_t stream) {
-  B200_RETURN_IF(total < 0 || act < 0 || act > 3, B200_ERR_BAD_SHAPE);
+  B200_RETURN_IF(total < 0 || act < 0 || act > 4, B200_ERR_BAD_SHAPE);
   if (total == 0) return B200_OK;
   B200_RETURN_IF(!out || !x, B200_ERR_NULL_POINTER);
   if (total % 8 == 0 && aligned16(out) && aligned16(x)) {
@@ -1323,9 +1514,9 @@ extern "C" int b200_act_only(void* out, const void* x, int64_t total, int32_t ac
 
 extern "C" int b200_norm_residual(void* h, float* residual, const void* y, const int64_t* y_index, int64_t y_rows,
                                   const void* y2, const int64_t* y2_index, int64_t y2_rows, const float* w,
-                                  const float* b, float eps, float offset, int32_t kind, int32_t accumulate,
+                                  const float* b, float eps, float offset, int32_t kind, int32_t accumulate, float carry,
                                   int32_t rows, int32_t hidden, int32_t dtype, b200_stream_t stream) {
-  B200_RETURN_IF(rows < 0 || hidden <= 0 || (kind != 0 && kind != 1), B200_ERR_BAD_SHAPE);
+  B200_RETURN_IF(rows < 0 || hidden <= 0 || (kind != 0 && kind != 1) || accumulate < 0 || accumulate > 2, B200_ERR_BAD_SHAPE);
   if (rows == 0) return B200_OK;
   B200_RETURN_IF(!residual || !y || !w, B200_ERR_NULL_POINTER);
   B200_RETURN_IF((y_index && y_rows <= 0) || (y2 && y2_index && y2_rows <= 0), B200_ERR_BAD_SHAPE);
@@ -1336,7 +1527,8 @@ extern "C" int b200_norm_residual(void* h, float* residual, const void* y, const
     const int threads = hidden / 8 >= 256 ? 256 : ((hidden / 8 + 31) / 32) * 32;
     B200_DISPATCH_3(dtype, T, launch_pdl(norm_residual_vec_kernel<T>, dim3(rows), dim3(threads), 0,
                                          (cudaStream_t)stream, (T*)h, residual, (const T*)y, y_index, y_rows,
-                                         (const T*)y2, y2_index, y2_rows, w, b, eps, offset, kind, accumulate, hidden));
+                                         (const T*)y2, y2_index, y2_rows, w, b, eps, offset, kind, accumulate, carry,
+                                         hidden));
     return finish_launch();
   }
   B200_DISPATCH_3(dtype, T, {
@@ -1344,7 +1536,7 @@ extern "C" int b200_norm_residual(void* h, float* residual, const void* y, const
       cudaFuncSetAttribute(norm_residual_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     launch_pdl(norm_residual_kernel<T>, dim3(rows), dim3(256), smem, (cudaStream_t)stream, (T*)h, residual,
                (const T*)y, y_index, y_rows, (const T*)y2, y2_index, y2_rows, w, b, eps, offset, kind, accumulate,
-               hidden);
+               carry, hidden);
   });
   return finish_launch();
 }
@@ -1474,6 +1666,72 @@ extern "C" int b200_rope_mix_cache(void* qkv, int64_t stride, const float* table
                                        stride, (const float2*)table, dims, interleaved, (const T*)v_other,
                                        v_other_stride, lambda, (T*)k_cache, (T*)v_cache, slots, slot_pairs, block_size,
                                        num_tokens, num_heads, num_kv_heads, dim, vdim));
+  return finish_launch();
+}
+
+extern "C" int b200_norm_rope_cache(void* qkv, int64_t stride, const float* wq, const float* wk, float eps,
+                                    const float* table, int32_t dims, int32_t interleaved, void* k_cache, void* v_cache,
+                                    const int32_t* slots, int32_t slot_pairs, int32_t block_size, int32_t num_tokens,
+                                    int32_t num_heads, int32_t num_kv_heads, int32_t dim, int32_t vdim, int32_t dtype,
+                                    b200_stream_t stream) {
+  B200_RETURN_IF(num_tokens < 0 || num_heads <= 0 || num_kv_heads <= 0 || dim <= 0 || vdim <= 0 || dims < 0 ||
+                     dims > dim || dims % 2 != 0,
+                 B200_ERR_BAD_SHAPE);
+  if (num_tokens == 0) return B200_OK;
+  B200_RETURN_IF(!qkv || !wq || !wk || (dims > 0 && !table) || (k_cache == nullptr) != (v_cache == nullptr) ||
+                     (k_cache && !slots),
+                 B200_ERR_NULL_POINTER);
+  const int64_t units = (int64_t)num_tokens * (num_heads + 2 * num_kv_heads);
+  const int gl = dim / 8;
+  if (interleaved && dim % 8 == 0 && (gl & (gl - 1)) == 0 && gl <= 32 && vdim % 8 == 0 && dims % 8 == 0 &&
+      stride % 8 == 0 && aligned16(qkv) && aligned16(wq) && aligned16(wk) && (dims == 0 || aligned16(table)) &&
+      (!k_cache || (aligned16(k_cache) && aligned16(v_cache)))) {
+    const int upw = 32 / gl;
+    const dim3 vgrid((unsigned)((units + 8 * upw - 1) / (8 * upw)));
+#define B200_NORM_ROPE_VEC(GLV)                                                                                       \
+  B200_DISPATCH_3(dtype, T, launch_pdl(norm_rope_cache_vec_kernel<T, GLV>, vgrid, dim3(256), 0, (cudaStream_t)stream, \
+                                       (T*)qkv, stride, wq, wk, eps, (const float2*)table, dims, (T*)k_cache,         \
+                                       (T*)v_cache, slots, slot_pairs, block_size, num_tokens, num_heads,             \
+                                       num_kv_heads, vdim))
+    switch (gl) {
+      case 1: B200_NORM_ROPE_VEC(1); break;
+      case 2: B200_NORM_ROPE_VEC(2); break;
+      case 4: B200_NORM_ROPE_VEC(4); break;
+      case 8: B200_NORM_ROPE_VEC(8); break;
+      case 16: B200_NORM_ROPE_VEC(16); break;
+      default: B200_NORM_ROPE_VEC(32); break;
+    }
+#undef B200_NORM_ROPE_VEC
+    return finish_launch();
+  }
+  B200_DISPATCH_3(dtype, T, launch_pdl(norm_rope_cache_kernel<T>, dim3((unsigned)((units + 7) / 8)), dim3(256), 0,
+                                       (cudaStream_t)stream, (T*)qkv, stride, wq, wk, eps, (const float2*)table, dims,
+                                       interleaved, (T*)k_cache, (T*)v_cache, slots, slot_pairs, block_size, num_tokens,
+                                       num_heads, num_kv_heads, dim, vdim));
+  return finish_launch();
+}
+
+extern "C" int b200_token_shift(void* out, int64_t mix_stride, const void* h, int64_t h_stride, const float* mu,
+                                int32_t mixes, void* state, const int32_t* state_slots, const int32_t* cu_q,
+                                const int32_t* cu_k, const int32_t* ctx_lens, int32_t num_seqs, int32_t max_q,
+                                int32_t width, int32_t dtype, b200_stream_t stream) {
+  B200_RETURN_IF(num_seqs < 0 || max_q < 0 || width <= 0 || mixes <= 0, B200_ERR_BAD_SHAPE);
+  if (num_seqs == 0 || max_q == 0) return B200_OK;
+  B200_RETURN_IF(!out || !h || !mu || (cu_q == nullptr) == (ctx_lens == nullptr) || (cu_q && !cu_k) ||
+                     (state && !state_slots), B200_ERR_NULL_POINTER);
+  B200_RETURN_IF(out == h, B200_ERR_UNSUPPORTED);
+  const bool vec = width % 8 == 0 && h_stride % 8 == 0 && mix_stride % 8 == 0 && aligned16(out) && aligned16(h) &&
+                   aligned16(mu) && (!state || aligned16(state));
+  const int lanes = vec ? width / 8 : width;
+  const dim3 grid((lanes + 127) / 128, (max_q + kShiftSeg - 1) / kShiftSeg, num_seqs);
+  B200_DISPATCH_3(dtype, T, {
+    if (vec)
+      launch_pdl(token_shift_kernel<T, 8>, grid, dim3(128), 0, (cudaStream_t)stream, (T*)out, mix_stride, (const T*)h,
+                 h_stride, mu, mixes, (T*)state, state_slots, cu_q, cu_k, ctx_lens, width);
+    else
+      launch_pdl(token_shift_kernel<T, 1>, grid, dim3(128), 0, (cudaStream_t)stream, (T*)out, mix_stride, (const T*)h,
+                 h_stride, mu, mixes, (T*)state, state_slots, cu_q, cu_k, ctx_lens, width);
+  });
   return finish_launch();
 }
 

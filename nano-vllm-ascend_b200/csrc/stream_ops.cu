@@ -7,8 +7,10 @@
 //   rotary_heads        rotary positions on the first `dims` columns of every head (pairs (2i, 2i+1) or
 //                       (i, i + dims/2)), a scale per head range, output in fp32 or the element type, with free
 //                       input/output head strides (so that a rotated part can be written into a wider head).
-//   delta_prep          what a gated delta rule reads besides v: q and k as fp32 unit vectors (q scaled), the
-//                       per-channel decay exp(-exp(A) softplus(a + bias)) and beta = sigmoid(b), all fp32.
+//   delta_prep          what a gated delta rule reads besides v: q and k as fp32 unit vectors (q scaled), the decay
+//                       exp(-exp(A) softplus(a + bias)) per key channel or per head, and beta = sigmoid(b), all fp32.
+//   wkv_prep            what a wkv recurrence reads besides v: the receptance and k in fp32, the decay exp(-exp(z + w0))
+//                       and the coefficient sum_i r_i u_i k_i with which the current token counts, all fp32.
 //   latent_kv_prep      RMS norm of the query latent; RMS norm of the key/value latent and rotation of the shared
 //                       rotated key, written as one cache row [latent | rotated key] (packed and/or paged).
 //   glu_clamped         min(g, L) sigmoid(alpha min(g, L)) (clamp(u, -L, L) + 1) for a gated feed-forward.
@@ -246,17 +248,18 @@ rotary_heads_kernel(const RotaryParams P) {
 
 // ------------------------------------------------------------------ inputs of a gated delta rule
 // One warp per (token, unit): units 0 .. 2G-1 are the q and k heads (unit vectors), units 2G .. 2G+H-1 the decay
-// rows of the heads (and beta).
+// rows of the heads (and beta). One decay per head (per_head): unit 2G holds all of them, a lane per head.
 template <typename T>
 __global__ void __launch_bounds__(256)
 delta_prep_kernel(float* __restrict__ qk, float* __restrict__ decay, float* __restrict__ beta,
                   const T* __restrict__ qk_in, int64_t qk_stride, const T* __restrict__ a, int64_t a_stride,
                   const T* __restrict__ b, int64_t b_stride, const float* __restrict__ dt_bias,
-                  const float* __restrict__ a_log, int tokens, int H, int G, int dim, float unit_eps, float q_scale) {
+                  const float* __restrict__ a_log, int tokens, int H, int G, int dim, float unit_eps, float q_scale,
+                  int per_head) {
   pdl_wait();
   const int lane = threadIdx.x & 31;
   const int64_t unit = (int64_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-  const int per_tok = 2 * G + H;
+  const int per_tok = 2 * G + (per_head ? 1 : H);
   if (unit >= (int64_t)tokens * per_tok) return;
   const int t = (int)(unit / per_tok), u = (int)(unit % per_tok);
   if (u < 2 * G) {
@@ -271,6 +274,13 @@ delta_prep_kernel(float* __restrict__ qk, float* __restrict__ decay, float* __re
     for (int i = lane; i < dim; i += 32) o[i] = to_f32<T>(x[i]) * mul;
     return;
   }
+  if (per_head) {
+    for (int h = lane; h < H; h += 32) {
+      decay[(int64_t)t * H + h] = expf(-expf(a_log[h]) * softplus_f(to_f32<T>(a[(int64_t)t * a_stride + h]) + dt_bias[h]));
+      beta[(int64_t)t * H + h] = sigmoid_f(to_f32<T>(b[(int64_t)t * b_stride + h]));
+    }
+    return;
+  }
   const int h = u - 2 * G;
   const float rate = expf(a_log[h]);
   const T* ar = a + (int64_t)t * a_stride + (int64_t)h * dim;
@@ -278,6 +288,61 @@ delta_prep_kernel(float* __restrict__ qk, float* __restrict__ decay, float* __re
   for (int i = lane; i < dim; i += 32)
     o[i] = expf(-rate * softplus_f(to_f32<T>(ar[i]) + dt_bias[(int64_t)h * dim + i]));
   if (lane == 0) beta[(int64_t)t * H + h] = sigmoid_f(to_f32<T>(b[(int64_t)t * b_stride + h]));
+}
+
+// ------------------------------------------------------------------ inputs of a wkv recurrence
+// Per (token, head): r and k to fp32, decay = exp(-exp(z + w0)) per key channel, bonus = sum_i r_i u_i k_i. gl = 1 .. 32
+// adjacent lanes per head (the smallest power of two that covers it with 8 elements per lane, VEC; a full warp element by
+// element otherwise); sums by xor shuffles inside the lane group.
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256)
+wkv_prep_kernel(float* __restrict__ r_out, float* __restrict__ k_out, float* __restrict__ decay,
+                float* __restrict__ bonus, const T* __restrict__ r, int64_t r_stride, const T* __restrict__ k,
+                int64_t k_stride, const float* __restrict__ z, const float* __restrict__ w0, const float* __restrict__ u,
+                int64_t tokens, int H, int dim, int gl) {
+  pdl_wait();
+  const int lane = threadIdx.x & 31, sub = lane % gl;
+  const int64_t warp = (int64_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  const int64_t unit = warp * (32 / gl) + lane / gl;
+  const bool live = unit < tokens * H;
+  const int64_t t = live ? unit / H : 0;
+  const int h = live ? (int)(unit % H) : 0;
+  const T* rr = r + t * r_stride + (int64_t)h * dim;
+  const T* kr = k + t * k_stride + (int64_t)h * dim;
+  const int64_t o = t * ((int64_t)H * dim) + (int64_t)h * dim;
+  const float* w0h = w0 + (int64_t)h * dim;
+  const float* uh = u + (int64_t)h * dim;
+  float acc = 0.f;
+  if (live) {
+    if constexpr (VEC) {
+      for (int i = sub * 8; i < dim; i += gl * 8) {
+        float a[8], b[8], c[8], d[8], e[8];
+        load8<T>(rr + i, a);
+        load8<T>(kr + i, b);
+        load8<float>(z + o + i, c);
+        load8<float>(w0h + i, d);
+        load8<float>(uh + i, e);
+#pragma unroll
+        for (int n = 0; n < 8; ++n) {
+          acc += a[n] * e[n] * b[n];
+          c[n] = expf(-expf(c[n] + d[n]));
+        }
+        store8<float>(r_out + o + i, a);
+        store8<float>(k_out + o + i, b);
+        store8<float>(decay + o + i, c);
+      }
+    } else {
+      for (int i = sub; i < dim; i += gl) {
+        const float a = to_f32<T>(rr[i]), b = to_f32<T>(kr[i]);
+        acc += a * uh[i] * b;
+        r_out[o + i] = a;
+        k_out[o + i] = b;
+        decay[o + i] = expf(-expf(z[o + i] + w0h[i]));
+      }
+    }
+  }
+  for (int off = gl >> 1; off > 0; off >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, off);
+  if (live && sub == 0) bonus[unit] = acc;
 }
 
 // ------------------------------------------------------------------ latents of a latent attention
@@ -638,16 +703,39 @@ extern "C" int b200_rotary_heads(void* out, int64_t out_stride, int32_t out_head
 extern "C" int b200_delta_prep(float* qk, float* decay, float* beta, const void* qk_in, int64_t qk_stride,
                                const void* a, int64_t a_stride, const void* b, int64_t b_stride,
                                const float* dt_bias, const float* a_log, int32_t tokens, int32_t num_heads,
-                               int32_t groups, int32_t dim, float unit_eps, float q_scale, int32_t dtype,
-                               b200_stream_t stream) {
+                               int32_t groups, int32_t dim, float unit_eps, float q_scale, int32_t per_head,
+                               int32_t dtype, b200_stream_t stream) {
   B200_RETURN_IF(tokens < 0 || num_heads <= 0 || groups <= 0 || dim <= 0, B200_ERR_BAD_SHAPE);
   if (tokens == 0) return B200_OK;
   B200_RETURN_IF(!qk || !decay || !beta || !qk_in || !a || !b || !dt_bias || !a_log, B200_ERR_NULL_POINTER);
-  const int64_t units = (int64_t)tokens * (2 * groups + num_heads);
+  const int64_t units = (int64_t)tokens * (2 * groups + (per_head ? 1 : num_heads));
   const dim3 grid((unsigned)((units + 7) / 8));
   B200_DISPATCH_3(dtype, T, launch_pdl(delta_prep_kernel<T>, grid, dim3(256), 0, (cudaStream_t)stream, qk, decay, beta,
                                        (const T*)qk_in, qk_stride, (const T*)a, a_stride, (const T*)b, b_stride,
-                                       dt_bias, a_log, tokens, num_heads, groups, dim, unit_eps, q_scale));
+                                       dt_bias, a_log, tokens, num_heads, groups, dim, unit_eps, q_scale, per_head));
+  return finish_launch();
+}
+
+extern "C" int b200_wkv_prep(float* r_out, float* k_out, float* decay, float* bonus, const void* r, int64_t r_stride,
+                             const void* k, int64_t k_stride, const float* z, const float* w0, const float* u,
+                             int32_t tokens, int32_t num_heads, int32_t dim, int32_t dtype, b200_stream_t stream) {
+  B200_RETURN_IF(tokens < 0 || num_heads <= 0 || dim <= 0, B200_ERR_BAD_SHAPE);
+  if (tokens == 0) return B200_OK;
+  B200_RETURN_IF(!r_out || !k_out || !decay || !bonus || !r || !k || !z || !w0 || !u, B200_ERR_NULL_POINTER);
+  const bool vec = dim % 8 == 0 && r_stride % 8 == 0 && k_stride % 8 == 0 && aligned16(r_out) && aligned16(k_out) &&
+                   aligned16(decay) && aligned16(r) && aligned16(k) && aligned16(z) && aligned16(w0) && aligned16(u);
+  int gl = vec ? 1 : 32;
+  while (vec && gl * 8 < dim && gl < 32) gl <<= 1;
+  const int64_t warps = ((int64_t)tokens * num_heads + 32 / gl - 1) / (32 / gl);
+  const dim3 grid((unsigned)((warps + 7) / 8));
+  B200_DISPATCH_3(dtype, T, {
+    if (vec)
+      launch_pdl(wkv_prep_kernel<T, true>, grid, dim3(256), 0, (cudaStream_t)stream, r_out, k_out, decay, bonus,
+                 (const T*)r, r_stride, (const T*)k, k_stride, z, w0, u, (int64_t)tokens, num_heads, dim, gl);
+    else
+      launch_pdl(wkv_prep_kernel<T, false>, grid, dim3(256), 0, (cudaStream_t)stream, r_out, k_out, decay, bonus,
+                 (const T*)r, r_stride, (const T*)k, k_stride, z, w0, u, (int64_t)tokens, num_heads, dim, gl);
+  });
   return finish_launch();
 }
 

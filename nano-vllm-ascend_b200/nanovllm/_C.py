@@ -55,6 +55,15 @@ PROTOTYPES = {
                                                   c_int32, c_int32, c_int32, c_int64, c_int64, c_int64, c_int64,
                                                   c_void_p, c_int32, c_int32, c_int32, c_float, c_float, c_void_p,
                                                   c_int32, c_void_p, c_int64, c_void_p]),
+    "b200_prefill_varlen_attn_windowed": (c_int32, [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int32,
+                                                    c_int32, c_int32, c_int32, c_int32, c_int32, c_int32, c_int32,
+                                                    c_int32, c_int64, c_int64, c_int64, c_int64, c_void_p, c_int32,
+                                                    c_int32, c_int32, c_float, c_float, c_void_p, c_int32, c_int32,
+                                                    c_int32, c_void_p, c_int64, c_void_p]),
+    "b200_paged_decode_attn_windowed": (c_int32, [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int32,
+                                                  c_int32, c_int32, c_int32, c_int32, c_int64, c_int64, c_int32,
+                                                  c_int32, c_int32, c_float, c_float, c_void_p, c_int32, c_int32,
+                                                  c_void_p, c_size_t, c_int32, c_int32, c_void_p]),
     "b200_prefill_workspace_size": (c_int64, [c_int32]),
     "b200_prefill_set_query_tiles": (c_int32, [c_int32]),
     "b200_gather_dequant_fp8": (c_int32, [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int32,
@@ -125,12 +134,12 @@ PROTOTYPES = {
                                            c_void_p, c_void_p, c_int32, c_int32, c_int32, c_int32, c_int32,
                                            c_int32, c_int32, c_int32, c_void_p]),
     "b200_gated_norm": (c_int32, [c_void_p, c_void_p, c_int32, c_void_p, c_int64, c_void_p, c_float, c_int32,
-                                  c_int32, c_int32, c_int32, c_int32, c_int32, c_void_p]),
+                                  c_int32, c_int32, c_int32, c_int32, c_int64, c_float, c_int32, c_void_p]),
     "b200_act_and_mul": (c_int32, [c_void_p, c_void_p, c_int32, c_int32, c_int32, c_int32, c_void_p]),
     "b200_attn_generic": (c_int32, [c_void_p, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_void_p,
                                     c_int32, c_int32, c_void_p, c_void_p, c_void_p, c_int32, c_int32, c_int32,
-                                    c_int32, c_int32, c_int32, c_float, c_int32, c_float, c_void_p, c_void_p, c_int64,
-                                    c_int32, c_void_p]),
+                                    c_int32, c_int32, c_int32, c_float, c_int32, c_int32, c_float, c_void_p, c_void_p,
+                                    c_int64, c_int32, c_void_p]),
     "b200_linear_recurrence": (c_int32, [c_void_p, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64,
                                          c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int32, c_int32, c_int32,
                                          c_int32, c_int32, c_int32, c_int32, c_int32, c_void_p, c_void_p,
@@ -144,10 +153,12 @@ PROTOTYPES = {
                                     c_float, c_int32, c_void_p]),
     "b200_delta_prep": (c_int32, [c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_int64, c_void_p,
                                   c_int64, c_void_p, c_void_p, c_int32, c_int32, c_int32, c_int32, c_float,
-                                  c_float, c_int32, c_void_p]),
+                                  c_float, c_int32, c_int32, c_void_p]),
+    "b200_wkv_prep": (c_int32, [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_int64, c_void_p,
+                                c_void_p, c_void_p, c_int32, c_int32, c_int32, c_int32, c_void_p]),
     "b200_delta_rule": (c_int32, [c_void_p, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_void_p,
                                   c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int32, c_int32,
-                                  c_int32, c_int32, c_int32, c_int32, c_void_p]),
+                                  c_int32, c_int32, c_int32, c_int32, c_int32, c_void_p]),
     "b200_latent_kv_prep": (c_int32, [c_void_p, c_void_p, c_void_p, c_void_p, c_int32, c_int32, c_void_p, c_int64,
                                       c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int32, c_int32, c_int32,
                                       c_int32, c_int32, c_double, c_int32, c_float, c_int32, c_void_p]),
@@ -160,8 +171,8 @@ PROTOTYPES = {
                                       c_void_p]),
     "b200_act_only": (c_int32, [c_void_p, c_void_p, c_int64, c_int32, c_int32, c_void_p]),
     "b200_norm_residual": (c_int32, [c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_int64,
-                                     c_void_p, c_void_p, c_float, c_float, c_int32, c_int32, c_int32, c_int32, c_int32,
-                                     c_void_p]),
+                                     c_void_p, c_void_p, c_float, c_float, c_int32, c_int32, c_float, c_int32, c_int32,
+                                     c_int32, c_void_p]),
     "b200_rownorm_cache": (c_int32, [c_void_p, c_int64, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p,
                                      c_int32, c_int32, c_int32, c_int32, c_int32, c_int32, c_int32, c_void_p]),
     "b200_gate_prep": (c_int32, [c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_int32,
@@ -186,6 +197,11 @@ PROTOTYPES = {
     "b200_rope_mix_cache": (c_int32, [c_void_p, c_int64, c_void_p, c_int32, c_int32, c_void_p, c_int64, c_void_p,
                                       c_void_p, c_void_p, c_void_p, c_int32, c_int32, c_int32, c_int32, c_int32,
                                       c_int32, c_int32, c_int32, c_void_p]),
+    "b200_norm_rope_cache": (c_int32, [c_void_p, c_int64, c_void_p, c_void_p, c_float, c_void_p, c_int32, c_int32,
+                                       c_void_p, c_void_p, c_void_p, c_int32, c_int32, c_int32, c_int32, c_int32,
+                                       c_int32, c_int32, c_int32, c_void_p]),
+    "b200_token_shift": (c_int32, [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int32, c_void_p, c_void_p, c_void_p,
+                                   c_void_p, c_void_p, c_int32, c_int32, c_int32, c_int32, c_void_p]),
     "b200_head_gate": (c_int32, [c_void_p, c_void_p, c_void_p, c_int64, c_int32, c_int32, c_int32, c_int32,
                                  c_void_p]),
     "b200_moe_combine_weighted": (c_int32, [c_void_p, c_void_p, c_void_p, c_void_p, c_int32, c_int32, c_int32,

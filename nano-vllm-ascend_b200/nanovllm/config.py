@@ -139,6 +139,28 @@ def nurilorn_preset(width: int, pattern: str, repeats: int, vocab: int = 32768, 
             "layers": [{"type": "attention", "mixer": dict(mixer), "mlp": mlp[ch]} for ch in pattern] * repeats}
 
 
+def pofazen_preset(width: int, pattern: str, repeats: int, vocab: int = 32768, head_dim: int = 128,
+                   window: int = 512, keep_first: int = 4) -> dict:
+    """A Pofazen configuration of realistic layer sizes for synthetic benchmarks: `pattern` is a string over
+    p (parallel attention and delta rule + feed-forward), w (wkv + feed-forward) and v (wkv alone), repeated `repeats`
+    times."""
+    H = width // head_dim
+    kv = max(1, H // 4)
+    dense = {"kind": "dense", "ff": 3 * width}
+    parallel = {"left": {"heads": H, "kv_heads": kv, "dim": head_dim, "vdim": head_dim, "scale": head_dim ** -0.5,
+                         "mask": {"size": window, "keep_first": keep_first},
+                         "rot": {"dims": head_dim // 2, "base": 5e5,
+                                 "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 2048}}},
+                "right": {"heads": H, "kv_heads": max(1, H // 2), "dim": head_dim, "vdim": head_dim, "conv": 4},
+                "left_scale": 1.0, "right_scale": 0.75}
+    wkv = {"heads": H, "dim": head_dim, "decay_rank": 64}
+    entry = {"p": {"type": "parallel", "mixer": parallel, "mlp": dense},
+             "w": {"type": "wkv", "mixer": wkv, "mlp": dense},
+             "v": {"type": "wkv", "mixer": wkv, "mlp": None}}
+    return {"architecture": "Pofazen", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "postln_alpha": 1.5,
+            "layers": [entry[ch] for ch in pattern] * repeats}
+
+
 def preset_hf_config(name: str):
     """Architecture presets built offline from the public model cards."""
     from transformers import LlamaConfig, Qwen3Config, Qwen3MoeConfig
@@ -165,6 +187,12 @@ def preset_hf_config(name: str):
         return NativeConfig(nurilorn_preset(2048, "aeae", 4, vocab=128256, head_dim=64))
     if key == "tiny-nurilorn":
         return NativeConfig(nurilorn_preset(128, "aen", 1, vocab=512, head_dim=32))
+    if key == "pofazen-1k":          # 28 layers at width 1024: the size class of nirelix-1k and zegopel-1k
+        return NativeConfig(pofazen_preset(1024, "pvwvpvw", 4, vocab=151936))
+    if key == "pofazen-2k":          # 16 layers at width 2048, head size 64: the size class of nirelix-2k
+        return NativeConfig(pofazen_preset(2048, "pvwv", 4, vocab=128256, head_dim=64))
+    if key == "tiny-pofazen":
+        return NativeConfig(pofazen_preset(128, "pwv", 1, vocab=512, head_dim=32, window=24))
     if key == "tiny-fitevik":
         return NativeConfig(fitevik_preset(128, "hgab", 1, vocab=512, head_dim=32, window=24, max_positions=512))
     if key == "qwen3-0.6b":

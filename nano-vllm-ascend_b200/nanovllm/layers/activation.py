@@ -1,5 +1,5 @@
 """SiluAndMul on the F3 kernel (reference: layers/activation.py:6-13), and the dense feed-forward with a clamped
-gated unit that several of the listed-layer decoders share."""
+gated unit and the one with act(gate) * up that several of the listed-layer decoders share."""
 import torch
 from torch import nn
 
@@ -24,3 +24,17 @@ class ClampedGatedFeedForward(nn.Module):
 
     def forward(self, h):
         return self.down_proj(ops.glu_clamped(self.gate_up_proj(h), self.alpha, self.limit))
+
+
+class GatedFeedForward(nn.Module):
+    """W_down(act(W_gate h) * W_up h) on the kernels that take any size and 16- or 32-bit elements; act: silu, relu or
+    gelu_tanh."""
+
+    def __init__(self, width: int, ff: int, act: str = "silu"):
+        super().__init__()
+        self.act = act
+        self.gate_up_proj = MergedColumnParallelLinear(width, [ff, ff])
+        self.down_proj = RowParallelLinear(ff, width)
+
+    def forward(self, h):
+        return self.down_proj(ops.act_and_mul(self.gate_up_proj(h), self.act))

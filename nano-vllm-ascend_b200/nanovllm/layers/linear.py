@@ -117,12 +117,14 @@ class MergedColumnParallelLinear(ColumnParallelLinear):
 
 
 class PaddedMergedLinear(ReplicatedLinear):
-    """Several small matrices that read the same input, stacked with each part padded to a multiple of 8 rows (so
+    """Several matrices that read the same input, stacked with each part padded to a multiple of 8 rows (so
     that every part of the output starts on a 16-byte boundary) and, for ``pad_input``, the input columns padded
-    to a multiple of 8 as well (the consumer of a padded part). Padding stays zero. Not sharded."""
+    to a multiple of 8 as well (the consumer of a padded part). A part may itself be a list of matrices, stacked without
+    padding between them and loaded as shard (part, matrix). Padding stays zero. Not sharded."""
 
     def __init__(self, input_size, output_sizes, pad_input=False):
-        self.output_sizes = list(output_sizes)
+        self.groups = [list(n) if isinstance(n, (list, tuple)) else [n] for n in output_sizes]
+        self.output_sizes = [sum(g) for g in self.groups]
         self.padded_sizes = [-(-n // 8) * 8 for n in self.output_sizes]
         self.true_input = input_size
         super().__init__(-(-input_size // 8) * 8 if pad_input else input_size, sum(self.padded_sizes))
@@ -144,9 +146,62 @@ class PaddedMergedLinear(ReplicatedLinear):
             off += pad
         self.weight.data[:, self.true_input:].zero_()
 
-    def weight_loader(self, param, loaded_weight, loaded_shard_id: int = 0):
-        start = sum(self.padded_sizes[:loaded_shard_id])
+    def weight_loader(self, param, loaded_weight, loaded_shard_id=0):
+        part, inner = loaded_shard_id if isinstance(loaded_shard_id, tuple) else (loaded_shard_id, 0)
+        start = sum(self.padded_sizes[:part]) + sum(self.groups[part][:inner])
         param.data[start:start + loaded_weight.shape[0], :loaded_weight.shape[1]].copy_(loaded_weight)
+
+
+class StackedLinear(nn.Module):
+    """``parts`` matrices of one shape, each on an input of its own: x [parts, T, in] -> [parts, T, out] as one batched
+    library product. Not sharded."""
+
+    def __init__(self, parts, input_size, output_size):
+        super().__init__()
+        self.weight = nn.Parameter(torch.empty(parts, output_size, input_size))
+        self.weight.weight_loader = lambda p, w, part: p.data[part].copy_(w)
+
+    def forward(self, x):
+        return torch.bmm(x, self.weight.transpose(1, 2))
+
+
+class ConcatInputLinear(ReplicatedLinear):
+    """The sum of several matrices applied to inputs of their own, as one product: their columns side by side, each part
+    padded to a multiple of 8 columns (so that every part of the input row starts on a 16-byte boundary). ``empty_input``
+    gives the input row block and ``part`` the view of it that a producer writes. Padding stays zero. Not sharded."""
+
+    def __init__(self, input_sizes, output_size):
+        self.input_sizes = list(input_sizes)
+        self.padded_sizes = [-(-n // 8) * 8 for n in self.input_sizes]
+        super().__init__(sum(self.padded_sizes), output_size)
+        self.weight.data.zero_()
+
+    def empty_input(self, rows, like):
+        make = torch.empty if self.padded_sizes == self.input_sizes else torch.zeros
+        return make(rows, sum(self.padded_sizes), dtype=like.dtype, device=like.device)
+
+    def part(self, x, i):
+        start = sum(self.padded_sizes[:i])
+        return x[:, start:start + self.input_sizes[i]]
+
+    def zero_padding(self):
+        off = 0
+        for n, pad in zip(self.input_sizes, self.padded_sizes):
+            self.weight.data[:, off + n:off + pad].zero_()
+            off += pad
+
+    def weight_loader(self, param, loaded_weight, loaded_shard_id: int):
+        start = sum(self.padded_sizes[:loaded_shard_id])
+        param.data[:, start:start + loaded_weight.shape[1]].copy_(loaded_weight)
+
+
+class F32OutLinear(ReplicatedLinear):
+    """A product whose result stays in fp32 (a 16-bit model's accumulators, unrounded): projections that go on in 32-bit."""
+
+    def forward(self, x):
+        if x.dtype == torch.float32:
+            return F.linear(x, self.weight)
+        return torch.mm(x, self.weight.t(), out_dtype=torch.float32)
 
 
 class QKVParallelLinear(ColumnParallelLinear):

@@ -1,9 +1,10 @@
 """Building blocks of hybrid decoders: a short causal convolution with a carried tail, linear recurrences
 with an fp32 state (constant decay per head, the selective state-space form, a forget gate per key channel that also
-decides what is written, or the gated delta rule with a decay per key channel), the gated norms that follow them,
-rotary positions on part of a head (plain, or with frequencies stretched by a ramp between a fast and a slow band),
-causal softmax attention whose key and value sizes may differ (optionally inside a sliding window, with capped scores,
-a sink in the denominator and a gate per head), attention whose heads are mixed before the softmax (with a distance bias, a sink, and keys and
+decides what is written, the gated delta rule with a decay per key channel or per head, or the wkv form with a bonus
+for the current token), the mixes of a token with the token before that the wkv form reads, the gated norms that follow,
+rotary positions on part of a head (plain, or with frequencies stretched by a ramp between a fast and a slow band or
+between a short and a long wavelength), causal softmax attention whose key and value sizes may differ (optionally inside
+a sliding window with first tokens that stay visible, with capped scores, a sink in the denominator and a gate per head), attention whose heads are mixed before the softmax (with a distance bias, a sink, and keys and
 values that may be another layer's), attention over a cached latent, and the mixing weights of a residual that is
 kept in several streams.
 
@@ -123,24 +124,27 @@ class GatedNorm(nn.Module):
         else:
             self.register_parameter("weight", None)
 
-    def forward(self, y: torch.Tensor, gate: torch.Tensor | None, dtype=None) -> torch.Tensor:
-        """gate None: the grouped norm alone, written in ``dtype``."""
-        return ops.gated_norm(y, gate, self.weight, self.eps, self.groups, self.gate_first, self.gate_act, dtype=dtype)
+    def forward(self, y: torch.Tensor, gate: torch.Tensor | None, dtype=None, out=None, scale: float = 1.0) -> torch.Tensor:
+        """gate None: the grouped norm alone, written in ``dtype``. The result times ``scale``, in ``out`` when given (a
+        slice of a wider row)."""
+        return ops.gated_norm(y, gate, self.weight, self.eps, self.groups, self.gate_first, self.gate_act, dtype=dtype,
+                              out=out, scale=scale)
 
 
 class VarSizeAttention(nn.Module):
     """Causal softmax attention with ``dim``-wide queries/keys and ``vdim``-wide values over paged caches
     ``k_cache`` [nb, bs, G*dim] / ``v_cache`` [nb, bs, G*vdim] (bound by the runner; K/V rows are written by the
-    caller's fused epilogue). 16-bit models with dim == vdim in {64, 128} run on the tcgen05 prefill kernel and
+    caller's fused epilogue). 16-bit models with dim and vdim in {64, 128} run on the tcgen05 prefill kernel and
     the paged decode kernel of the dense decoders; everything else (other sizes, fp32) on the generic kernel.
+    ``window`` w > 0: position i sees the keys j <= i with i - j < w, and those with j < ``keep_first``.
     ``softcap`` c > 0 turns every score s into c tanh(s / c); ``sink`` (a logit) adds exp(sink) to every softmax
     denominator, an entry without key or value; ``forward(..., gate)`` multiplies head h of token t by sigmoid(gate[t, h])."""
 
     def __init__(self, num_heads: int, num_kv_heads: int, dim: int, vdim: int, scale: float, window: int = 0,
-                 softcap: float = 0.0, sink: float | None = None):
+                 softcap: float = 0.0, sink: float | None = None, keep_first: int = 0):
         super().__init__()
         self.num_heads, self.num_kv_heads, self.dim, self.vdim, self.scale = num_heads, num_kv_heads, dim, vdim, scale
-        self.window = int(window)                       # > 0: position i sees keys j with 0 <= i - j < window
+        self.window, self.keep_first = int(window), int(keep_first)
         self.softcap = float(softcap or 0.0)
         if sink is not None:
             self.register_buffer("sink", torch.full((num_heads,), float(sink), dtype=F32), persistent=False)
@@ -156,9 +160,8 @@ class VarSizeAttention(nn.Module):
 
     def _fast(self, q) -> bool:
         rep, G = self.num_heads // self.num_kv_heads, self.num_kv_heads
-        return (not self.force_generic and not self.window
-                and q.dtype in (torch.bfloat16, torch.float16) and self.dim == self.vdim
-                and self.dim in (64, 128) and rep <= 8 and (G in (1, 2, 4) or G % 8 == 0))
+        return (not self.force_generic and q.dtype in (torch.bfloat16, torch.float16)
+                and self.dim in (64, 128) and self.vdim in (64, 128) and rep <= 8 and (G in (1, 2, 4) or G % 8 == 0))
 
     def forward(self, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: torch.Tensor | None = None) -> torch.Tensor:
         """q [T, H, dim]; k [T, G, dim], v [T, G, vdim]: this step's rows (used when no cache is bound); gate [T, H]
@@ -167,10 +170,12 @@ class VarSizeAttention(nn.Module):
         paged = self.k_cache.numel() > 0 and ctx.block_tables is not None
         if self._fast(q) and (paged or ctx.is_prefill):
             out = None
-            soft = dict(softcap=self.softcap, sink=self.sink)
-            # a score cap or a sink: the tcgen05 kernel only, whose TMA maps want 16-byte row strides and blocks that
+            soft = dict(softcap=self.softcap, sink=self.sink, vdim=self.vdim, window=self.window,
+                        keep_first=self.keep_first)
+            plain = not self.softcap and self.sink is None and not self.window and self.dim == self.vdim
+            # a score cap, a sink, a window or unequal head sizes: the tcgen05 kernel only, whose TMA maps want 16-byte row strides and blocks that
             # tile its 128-key steps
-            tma_ok = not (self.softcap or self.sink is not None) or (
+            tma_ok = plain or (
                 q.stride(0) % 8 == 0 and (paged and (ctx.block_size % 128 == 0 or 128 % ctx.block_size == 0) or
                                           not paged and k.stride(0) % 8 == 0 and v.stride(0) % 8 == 0))
             if not ctx.is_prefill:
@@ -187,7 +192,7 @@ class VarSizeAttention(nn.Module):
                 out = out.view(q.shape[0], self.num_heads * self.vdim)
                 return out if gate is None else ops.head_gate_(out, gate, self.num_heads)
         spans = ops.StepSpans.of(ctx)
-        extras = dict(window=self.window, softcap=self.softcap, sink=self.sink, gate=gate)
+        extras = dict(window=self.window, keep_first=self.keep_first, softcap=self.softcap, sink=self.sink, gate=gate)
         if paged:
             return ops.attn_generic(q, self.k_cache, self.v_cache, spans, self.scale, self.num_kv_heads, self.vdim,
                                     block_tables=ctx.block_tables, **extras)
@@ -354,31 +359,74 @@ class MixedHeadAttention(nn.Module):
 
 
 class DeltaRule(nn.Module):
-    """Gated delta rule with one decay per head and key channel, state S fp32 [kdim, vdim] per head in ``state``:
-    S <- diag(g) S; w = beta (v - S^T k); S <- S + k w^T; o = S^T q, with g = exp(-exp(A_log_h) softplus(a + dt_bias)),
+    """Gated delta rule with one decay per head and key channel (``per_head``: one per head), state S fp32 [kdim, vdim] per
+    head in ``state``: S <- diag(g) S; w = beta (v - S^T k); S <- S + k w^T; o = S^T q, with g = exp(-exp(A_log_h) softplus(a + dt_bias)),
     beta = sigmoid(b), q and k divided by sqrt(sum x^2 + unit_eps) per head and q times ``q_scale``. Everything but the
     projected activations is fp32."""
 
     def __init__(self, num_heads: int, groups: int, kdim: int, vdim: int, unit_eps: float = 1e-6,
-                 q_scale: float | None = None):
+                 q_scale: float | None = None, per_head: bool = False):
         super().__init__()
         self.num_heads, self.groups, self.kdim, self.vdim = num_heads, groups, kdim, vdim
-        self.unit_eps = unit_eps
+        self.unit_eps, self.per_head = unit_eps, bool(per_head)
         self.q_scale = kdim ** -0.5 if q_scale is None else q_scale
-        self.A_log, self.dt_bias = small_param(num_heads), small_param(num_heads * kdim)
+        self.A_log, self.dt_bias = small_param(num_heads), small_param(num_heads * (1 if per_head else kdim))
         self.state = None
 
     def state_shapes(self):
         return {"state": ((self.num_heads, self.kdim, self.vdim), F32)}
 
     def forward(self, qk, v, a, b) -> torch.Tensor:
-        """qk [T, 2*groups*kdim] (q heads, then k heads), v [T, H*vdim], a [T, H*kdim], b [T, H] -> fp32 [T, H*vdim]."""
+        """qk [T, 2*groups*kdim] (q heads, then k heads), v [T, H*vdim], a [T, H*kdim] (per_head: [T, H]), b [T, H] -> fp32
+        [T, H*vdim]."""
         ctx, spans, bound = _spans_and_slots(self.state)
         qk32, g, beta = ops.delta_prep(qk, a, b, self.dt_bias, self.A_log, self.num_heads, self.groups, self.kdim,
-                                       self.unit_eps, self.q_scale)
+                                       self.unit_eps, self.q_scale, per_head=self.per_head)
         n = self.groups * self.kdim
         return ops.delta_rule(qk32[:, :n], qk32[:, n:], v, g, beta, spans, self.num_heads, self.groups, self.kdim,
                               self.vdim, self.state if bound else None, ctx.state_slots if bound else None)
+
+
+class TokenShift(nn.Module):
+    """``mixes`` mixes of every token with the token before it, h_t + (h_(t-1) - h_t) * mu[m] (zeros before a sequence's
+    start): [T, width] -> [mixes, T, width]. ``shift_state`` keeps each sequence's last row."""
+
+    def __init__(self, width: int, mixes: int):
+        super().__init__()
+        self.width = width
+        self.mu = small_param(mixes, width)
+        self.mu.weight_loader = lambda p, w, m: p.data[m].copy_(w)
+        self.shift_state = None
+
+    def state_shapes(self):
+        return {"shift_state": ((self.width,), None)}
+
+    def forward(self, h: torch.Tensor) -> torch.Tensor:
+        ctx, spans, bound = _spans_and_slots(self.shift_state)
+        return ops.token_shift(h, self.mu, spans, self.shift_state if bound else None, ctx.state_slots if bound else None)
+
+
+class WkvRecurrence(nn.Module):
+    """o_t = (S + diag(u) k_t v_t^T)^T r_t, then S <- diag(w_t) S + k_t v_t^T per head, S fp32 [dim, dim] in ``state``: the
+    read-out comes before the write, the current token counts through its bonus u. w = exp(-exp(z + w0)) per key channel
+    from a projected z. Everything but the projected r, k, v is fp32."""
+
+    def __init__(self, num_heads: int, dim: int):
+        super().__init__()
+        self.num_heads, self.dim = num_heads, dim
+        self.w0, self.u = small_param(num_heads * dim), small_param(num_heads * dim)
+        self.u.weight_loader = lambda p, w: p.data.copy_(w.reshape(-1))
+        self.state = None
+
+    def state_shapes(self):
+        return {"state": ((self.num_heads, self.dim, self.dim), F32)}
+
+    def forward(self, r, k, v, z) -> torch.Tensor:
+        """r, k, v [T, H*dim] in the model dtype, z fp32 [T, H*dim] -> fp32 [T, H*dim]."""
+        ctx, spans, bound = _spans_and_slots(self.state)
+        r32, k32, decay, bonus = ops.wkv_prep(r, k, z, self.w0, self.u, self.num_heads, self.dim)
+        return ops.wkv(r32, k32, v, decay, bonus, spans, self.num_heads, self.dim, self.dim,
+                       self.state if bound else None, ctx.state_slots if bound else None)
 
 
 class Rotary:
@@ -394,34 +442,16 @@ class Rotary:
                                 out_f32=out_f32, split=split, scale_lo=scale_lo, scale_hi=scale_hi)
 
 
-class BandScaledRotary:
-    """Rotary positions whose frequencies are stretched band by band: f_i = base^(-2i/dims), i < dims/2; with
-    n(t) = dims ln(original / (2 pi t)) / (2 ln base) (the pair index that makes t turns over the original length),
-    lo = max(floor(n(fast)), 0), hi = min(ceil(n(slow)), dims - 1) and ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1)
-    the frequency becomes f_i / factor * ramp_i + f_i (1 - ramp_i): pairs that turn fast keep their frequency, slow
-    ones are divided by ``factor``, and cos and sin are multiplied by 0.1 ln(factor) + 1. Without ``scaling`` the
-    frequencies are the plain ones. The step's (cos, sin) table is computed once per pass (fp64 angles) and shared by
-    all layers with the same constants; the rotation itself runs fused with the layer's cache write
-    (ops.rope_mix_cache)."""
+class TableRotary:
+    """Rotary positions from a table of frequencies [dims / 2] (times a magnitude on cos and sin), pairs (2i, 2i+1)
+    (``interleaved``) or (i, i + dims/2). The step's (cos, sin) table is computed once per pass (fp64 angles) and shared by
+    all layers with the same constants; the rotation itself runs fused with the layer's cache write (ops.rope_mix_cache,
+    ops.norm_rope_cache)."""
 
-    MAGNITUDE_SLOPE = 0.1
-
-    def __init__(self, dims: int, base: float, interleaved: bool = True, scaling: dict | None = None):
-        import math
-        self.dims, self.base, self.interleaved = int(dims), float(base), bool(interleaved)
-        half = self.dims // 2
-        f = [self.base ** (-2.0 * i / self.dims) for i in range(half)]
-        self.magnitude = 1.0
-        if scaling:
-            factor, original = float(scaling["factor"]), float(scaling["original"])
-            turns_at = lambda t: self.dims * math.log(original / (2 * math.pi * t)) / (2 * math.log(self.base))
-            lo = max(math.floor(turns_at(float(scaling["fast"]))), 0)
-            hi = min(math.ceil(turns_at(float(scaling["slow"]))), self.dims - 1)
-            ramp = [min(1.0, max(0.0, (i - lo) / max(hi - lo, 0.001))) for i in range(half)]
-            f = [fi / factor * r + fi * (1 - r) for fi, r in zip(f, ramp)]
-            self.magnitude = self.MAGNITUDE_SLOPE * math.log(factor) + 1.0
-        self.freq = torch.tensor(f, dtype=torch.float64)
-        self.key = ("rotary table", self.dims, self.interleaved, self.magnitude, tuple(f))
+    def __init__(self, dims: int, freq: list, interleaved: bool = True, magnitude: float = 1.0):
+        self.dims, self.interleaved, self.magnitude = int(dims), bool(interleaved), float(magnitude)
+        self.freq = torch.tensor(freq, dtype=torch.float64)
+        self.key = ("rotary table", self.dims, self.interleaved, self.magnitude, tuple(freq))
 
     def table(self, positions: torch.Tensor) -> torch.Tensor | None:
         """fp32 [T, dims/2, 2] for this pass's positions, from the context's per-pass scratch."""
@@ -434,6 +464,55 @@ class BandScaledRotary:
                 self.freq = self.freq.to(positions.device)
             t = ctx.scratch[self.key] = ops.rotary_table(positions, self.freq, self.magnitude)
         return t
+
+
+class WavelengthScaledRotary(TableRotary):
+    """Rotary positions whose frequencies f_i = base^(-2i/dims) depend on their wavelength l = 2 pi / f_i: kept where
+    l < original / high, divided by ``factor`` where l > original / low, and with s = (original / l - low) / (high - low)
+    blended to (1 - s) f_i / factor + s f_i between the two. Without ``scaling`` the frequencies are the plain ones."""
+
+    def __init__(self, dims: int, base: float, interleaved: bool = True, scaling: dict | None = None):
+        import math
+        dims, base = int(dims), float(base)
+        f = [base ** (-2.0 * i / dims) for i in range(dims // 2)]
+        if scaling:
+            factor, original = float(scaling["factor"]), float(scaling["original"])
+            low, high = float(scaling["low"]), float(scaling["high"])
+            for i, fi in enumerate(f):
+                wave = 2 * math.pi / fi
+                if wave > original / low:
+                    f[i] = fi / factor
+                elif wave >= original / high:
+                    s = (original / wave - low) / (high - low) if high != low else 1.0
+                    f[i] = (1 - s) * fi / factor + s * fi
+        super().__init__(dims, f, interleaved)
+
+
+class BandScaledRotary(TableRotary):
+    """Rotary positions whose frequencies are stretched band by band: f_i = base^(-2i/dims), i < dims/2; with
+    n(t) = dims ln(original / (2 pi t)) / (2 ln base) (the pair index that makes t turns over the original length),
+    lo = max(floor(n(fast)), 0), hi = min(ceil(n(slow)), dims - 1) and ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1)
+    the frequency becomes f_i / factor * ramp_i + f_i (1 - ramp_i): pairs that turn fast keep their frequency, slow
+    ones are divided by ``factor``, and cos and sin are multiplied by 0.1 ln(factor) + 1. Without ``scaling`` the
+    frequencies are the plain ones."""
+
+    MAGNITUDE_SLOPE = 0.1
+
+    def __init__(self, dims: int, base: float, interleaved: bool = True, scaling: dict | None = None):
+        import math
+        dims, base = int(dims), float(base)
+        half = dims // 2
+        f = [base ** (-2.0 * i / dims) for i in range(half)]
+        magnitude = 1.0
+        if scaling:
+            factor, original = float(scaling["factor"]), float(scaling["original"])
+            turns_at = lambda t: dims * math.log(original / (2 * math.pi * t)) / (2 * math.log(base))
+            lo = max(math.floor(turns_at(float(scaling["fast"]))), 0)
+            hi = min(math.ceil(turns_at(float(scaling["slow"]))), dims - 1)
+            ramp = [min(1.0, max(0.0, (i - lo) / max(hi - lo, 0.001))) for i in range(half)]
+            f = [fi / factor * r + fi * (1 - r) for fi, r in zip(f, ramp)]
+            magnitude = self.MAGNITUDE_SLOPE * math.log(factor) + 1.0
+        super().__init__(dims, f, interleaved, magnitude)
 
 
 def prompt_chunk_plan(ctx, paged, device, chunk: int, window: int, min_tokens: int):

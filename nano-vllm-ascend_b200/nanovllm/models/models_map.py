@@ -6,8 +6,9 @@ which this build deliberately leaves out. Zegopel (a hybrid of softmax attention
 Mamba-2 layers) and Nirelix (retention, gated delta rule and latent attention on a residual kept in several
 streams) and Fitevik (HGRN2 recurrences and attention with mixed heads, a distance bias and a sink, on a residual
 with the norm on each sublayer's output) and Nurilorn (gated attention with capped scores, a sink, rotary positions
-stretched band by band and values blended across layers, on a residual with scaled branches and grouped norms) are
-additions; their config.json names them with an ``"architecture"`` string (config.NativeConfig). Qwen2 checkpoints are served by the Qwen3 class, as in the reference:
+stretched band by band and values blended across layers, on a residual with scaled branches and grouped norms) and
+Pofazen (windowed gated attention beside a gated delta rule in one mixer, and wkv recurrences with a token shift, on a
+residual whose norm is taken of the sum) are additions; their config.json names them with an ``"architecture"`` string (config.NativeConfig). Qwen2 checkpoints are served by the Qwen3 class, as in the reference:
 the config's ``attention_bias`` decides between QKV bias (Qwen2) and QK-norm (Qwen3).
 """
 from __future__ import annotations
@@ -18,6 +19,7 @@ from .qwen3_moe import Qwen3MoeForCausalLM
 from .fitevik import FitevikForCausalLM
 from .nirelix import NirelixForCausalLM
 from .nurilorn import NurilornForCausalLM
+from .pofazen import PofazenForCausalLM
 from .zegopel import ZegopelForCausalLM
 
 model_dict: dict[str, type] = {}
@@ -34,5 +36,6 @@ for _arch, _cls in (("Qwen3ForCausalLM", Qwen3ForCausalLM),
                     ("Zegopel", ZegopelForCausalLM),
                     ("Nirelix", NirelixForCausalLM),
                     ("Fitevik", FitevikForCausalLM),
-                    ("Nurilorn", NurilornForCausalLM)):
+                    ("Nurilorn", NurilornForCausalLM),
+                    ("Pofazen", PofazenForCausalLM)):
     register(_arch, _cls)

@@ -123,9 +123,10 @@ def decode_workspace(batch, num_heads, num_kv_heads, head_dim, device) -> torch.
 
 
 def paged_decode_attn(q, k_cache, v_cache, block_tables, context_lens, scale, num_kv_heads,
-                      out=None, workspace=None, num_ctas=0, softcap=0.0, sink=None):
-    """K6. q [B, H, D] (token-strided view allowed) -> out [B, H*D]. softcap > 0: scores become softcap *
-    tanh(score / softcap); sink fp32 [H]: exp(sink[h]) joins the softmax denominator (no key, no value)."""
+                      out=None, workspace=None, num_ctas=0, softcap=0.0, sink=None, vdim=None, window=0, keep_first=0):
+    """K6. q [B, H, D] (token-strided view allowed) -> out [B, H*vdim] (vdim: width of a value head, D by default).
+    softcap > 0: scores become softcap * tanh(score / softcap); sink fp32 [H]: exp(sink[h]) joins the softmax denominator
+    (no key, no value). window > 0: a row sees its last `window` keys and those below keep_first."""
     _need_cuda(q, k_cache, v_cache, block_tables, context_lens, sink)
     _f32(sink)
     B, H, D = q.shape
@@ -138,16 +139,19 @@ def paged_decode_attn(q, k_cache, v_cache, block_tables, context_lens, scale, nu
     if block_tables.dim() != 2 or block_tables.stride(1) != 1 or not context_lens.is_contiguous():
         raise ValueError("block_tables must be [B, max_blocks] row-major, context_lens contiguous")
     nb, bs = _cache_dims(k_cache, num_kv_heads * D)
+    vdim = D if vdim is None else int(vdim)
+    if vdim != D:
+        _cache_dims(v_cache, num_kv_heads * vdim)
     if out is None:
-        out = torch.empty(B, H * D, dtype=q.dtype, device=q.device)
+        out = torch.empty(B, H * vdim, dtype=q.dtype, device=q.device)
     if workspace is None:
-        workspace = decode_workspace(B, H, num_kv_heads, D, q.device)
-    _C.check(_C.load().b200_paged_decode_attn_capped(
+        workspace = decode_workspace(B, H, num_kv_heads, vdim, q.device)
+    _C.check(_C.load().b200_paged_decode_attn_windowed(
         out.data_ptr(), q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(),
-        block_tables.data_ptr(), context_lens.data_ptr(), B, H, num_kv_heads, D,
-        q.stride(0) if B > 1 else H * D, out.stride(0) if B > 1 else H * D, nb, bs,
-        block_tables.stride(0), float(scale), float(softcap or 0.0), _ptr(sink), workspace.data_ptr(),
-        workspace.numel(), int(num_ctas), _dt(q), _stream()), "b200_paged_decode_attn")
+        block_tables.data_ptr(), context_lens.data_ptr(), B, H, num_kv_heads, D, vdim,
+        q.stride(0) if B > 1 else H * D, out.stride(0) if B > 1 else H * vdim, nb, bs,
+        block_tables.stride(0), float(scale), float(softcap or 0.0), _ptr(sink), int(window), int(keep_first),
+        workspace.data_ptr(), workspace.numel(), int(num_ctas), _dt(q), _stream()), "b200_paged_decode_attn")
     return out
 
 
@@ -217,11 +221,13 @@ def prefill_workspace(device, head_dim: int) -> torch.Tensor:
 
 
 def prefill_varlen_attn(q, k, v, cu_seqlens_q, cu_seqlens_k, max_seqlen_q, max_seqlen_k, scale,
-                        num_kv_heads, block_tables=None, out=None, workspace="auto", softcap=0.0, sink=None):
+                        num_kv_heads, block_tables=None, out=None, workspace="auto", softcap=0.0, sink=None, vdim=None,
+                        window=0, keep_first=0):
     """K4/K5. q [Tq, H, D]; packed mode: k/v [Tk, Hkv, D]; paged mode (block_tables given):
     k/v are the caches [nb, bs, Hkv*D]. Returns out [Tq, H*D]. workspace: "auto" (the per-device
-    split-KV workspace), None (never split the keys across CTAs) or a uint8 CUDA tensor. softcap, sink as in
-    paged_decode_attn (the tcgen05 kernel only)."""
+    split-KV workspace), None (never split the keys across CTAs) or a uint8 CUDA tensor. softcap, sink, vdim, window,
+    keep_first as in paged_decode_attn (the tcgen05 kernel only); position i sees j <= i with i - j < window or
+    j < keep_first."""
     _need_cuda(q, k, v, cu_seqlens_q, cu_seqlens_k, block_tables, sink)
     _f32(sink)
     Tq, H, D = q.shape
@@ -232,30 +238,33 @@ def prefill_varlen_attn(q, k, v, cu_seqlens_q, cu_seqlens_k, max_seqlen_q, max_s
     if cu_seqlens_q.dtype != torch.int32 or cu_seqlens_k.dtype != torch.int32:
         raise TypeError("cu_seqlens must be int32")
     num_seqs = cu_seqlens_q.numel() - 1
+    vdim = D if vdim is None else int(vdim)
     if out is None:
-        out = torch.empty(Tq, H * D, dtype=q.dtype, device=q.device)
+        out = torch.empty(Tq, H * vdim, dtype=q.dtype, device=q.device)
     if block_tables is not None:
         if block_tables.dtype != torch.int32 or block_tables.stride(1) != 1:
             raise TypeError("block_tables must be row-major int32")
         nb, bs = _cache_dims(k, num_kv_heads * D)
-        ks = vs = num_kv_heads * D
+        _cache_dims(v, num_kv_heads * vdim)
+        ks, vs = num_kv_heads * D, num_kv_heads * vdim
         bt_ptr, bt_stride = block_tables.data_ptr(), block_tables.stride(0)
     else:
-        if k.stride(2) != 1 or k.stride(1) != D or v.stride(2) != 1 or v.stride(1) != D:
+        if k.stride(2) != 1 or k.stride(1) != D or v.stride(2) != 1 or v.stride(1) != vdim:
             raise ValueError("k/v must be contiguous in (heads, head_dim)")
         nb = bs = 0
         ks = k.stride(0) if k.shape[0] > 1 else num_kv_heads * D
-        vs = v.stride(0) if v.shape[0] > 1 else num_kv_heads * D
+        vs = v.stride(0) if v.shape[0] > 1 else num_kv_heads * vdim
         bt_ptr, bt_stride = None, 0
     if isinstance(workspace, str):
-        workspace = prefill_workspace(q.device, D)
+        workspace = prefill_workspace(q.device, vdim)
     ws_ptr, ws_bytes = (None, 0) if workspace is None else (workspace.data_ptr(), workspace.numel())
-    _C.check(_C.load().b200_prefill_varlen_attn_capped(
+    _C.check(_C.load().b200_prefill_varlen_attn_windowed(
         out.data_ptr(), q.data_ptr(), k.data_ptr(), v.data_ptr(), cu_seqlens_q.data_ptr(),
         cu_seqlens_k.data_ptr(), num_seqs, Tq, 0 if block_tables is not None else k.shape[0],
         int(max_seqlen_q), int(max_seqlen_k), H, num_kv_heads,
-        D, q.stride(0) if Tq > 1 else H * D, ks, vs, out.stride(0) if Tq > 1 else H * D, bt_ptr,
-        bt_stride, nb, bs, float(scale), float(softcap or 0.0), _ptr(sink), _dt(q), ws_ptr, ws_bytes, _stream()),
+        D, vdim, q.stride(0) if Tq > 1 else H * D, ks, vs, out.stride(0) if Tq > 1 else H * vdim, bt_ptr,
+        bt_stride, nb, bs, float(scale), float(softcap or 0.0), _ptr(sink), int(window), int(keep_first), _dt(q), ws_ptr,
+        ws_bytes, _stream()),
         "b200_prefill_varlen_attn")
     return out
 
@@ -794,10 +803,11 @@ def unitnorm_temp_cache(qkv, positions, eps, temp_coef, temp_every, num_heads, n
     return qkv
 
 
-def gated_norm(y, gate, weight, eps, groups=1, gate_first=False, gate_act="sigmoid", dtype=None):
+def gated_norm(y, gate, weight, eps, groups=1, gate_first=False, gate_act="sigmoid", dtype=None, out=None, scale=1.0):
     """y [rows, n] (fp32 or gate's dtype), gate [rows, n] (row-strided view allowed) -> [rows, n] in gate's dtype.
     weight fp32 [n]: RMS norm over each of `groups` equal parts, before (gate_first=False) or after the gate;
-    weight None: the gate alone. gate None (with a weight): the grouped norm alone, output in `dtype`."""
+    weight None: the gate alone. gate None (with a weight): the grouped norm alone, output in `dtype`. The result is
+    multiplied by `scale` before it is rounded; out: a row-strided view that receives it (a slice of a wider row)."""
     _need_cuda(y, gate, weight)
     _f32(weight)
     rows, n = y.shape
@@ -813,11 +823,15 @@ def gated_norm(y, gate, weight, eps, groups=1, gate_first=False, gate_act="sigmo
         raise ValueError("y contiguous [rows, n]")
     if y.dtype not in (torch.float32, dtype):
         raise TypeError("y must be fp32 or of the gate's dtype")
-    out = torch.empty(rows, n, dtype=dtype, device=y.device)
+    if out is None:
+        out = torch.empty(rows, n, dtype=dtype, device=y.device)
+    elif out.shape != y.shape or out.dtype != dtype or out.stride(1) != 1:
+        raise ValueError("out: [rows, n] of the output dtype with unit inner stride")
     _C.check(_C.load().b200_gated_norm(out.data_ptr(), y.data_ptr(), 1 if y.dtype == torch.float32 else 0,
                                        _ptr(gate), (gate.stride(0) if rows > 1 else n) if gate is not None else n,
                                        _ptr(weight), float(eps), rows, n, int(groups), 1 if gate_first else 0,
-                                       {"sigmoid": 0, "silu": 1, "none": 2}[gate_act], _DT3[dtype], _stream()),
+                                       {"sigmoid": 0, "silu": 1, "none": 2}[gate_act], out.stride(0) if rows > 1 else n,
+                                       float(scale), _DT3[dtype], _stream()),
              "b200_gated_norm")
     return out
 
@@ -837,11 +851,11 @@ def act_and_mul(x, act="silu"):
     return out
 
 
-_PLAIN_ACTS = {"silu": 0, "relu": 1, "gelu_tanh": 2, "relu2": 3}
+_PLAIN_ACTS = {"silu": 0, "relu": 1, "gelu_tanh": 2, "relu2": 3, "tanh": 4}
 
 
 def act_only(x, act="relu2"):
-    """act(x) elementwise for a feed-forward without a gate: silu | relu | gelu_tanh | relu2 (the square of relu)."""
+    """act(x) elementwise for a feed-forward without a gate: silu | relu | gelu_tanh | relu2 (the square of relu) | tanh."""
     _need_cuda(x)
     if not x.is_contiguous():
         raise ValueError("act_only input must be contiguous")
@@ -852,9 +866,10 @@ def act_only(x, act="relu2"):
 
 
 def norm_residual_(residual, y, w, b, eps, dtype, kind="layer", offset=0.0, accumulate=True, y_index=None, y2=None,
-                   y2_index=None, want_h=True):
+                   y2_index=None, want_h=True, carry=None):
     """A norm on a sublayer's OUTPUT, then the residual: residual (fp32 [rows, hidden], in place) <- (residual if
-    accumulate else 0) + norm(y [+ y2]); returns the new residual in `dtype` (the next sublayer reads the stream
+    accumulate else 0) + norm(y [+ y2]) -- or, with ``carry`` c, a norm after the sum: residual <- norm(c residual + y
+    [+ y2]); returns the new residual in `dtype` (the next sublayer reads the stream
     itself). kind "layer": (u - mean) / sqrt(var + eps) * w + b; "rms": u / sqrt(mean u^2 + eps) * (offset + w).
     y_index / y2_index (int64 [rows]): rows of y / y2 are gathered by index (clamped to the table) -- token embedding
     plus learned position plus norm in one launch."""
@@ -872,8 +887,9 @@ def norm_residual_(residual, y, w, b, eps, dtype, kind="layer", offset=0.0, accu
     _C.check(_C.load().b200_norm_residual(_ptr(h), residual.data_ptr(), y.data_ptr(), _ptr(y_index), y.shape[0],
                                           _ptr(y2), _ptr(y2_index), y2.shape[0] if y2 is not None else 0,
                                           w.data_ptr(), _ptr(b), float(eps), float(offset),
-                                          {"layer": 0, "rms": 1}[kind], 1 if accumulate else 0, rows, hidden,
-                                          _DT3[dtype], _stream()), "b200_norm_residual")
+                                          {"layer": 0, "rms": 1}[kind], 2 if carry is not None else 1 if accumulate else 0,
+                                          float(carry or 0.0), rows, hidden, _DT3[dtype], _stream()),
+             "b200_norm_residual")
     return h
 
 
@@ -955,11 +971,11 @@ def mixed_attn(q, k, v, spans: StepSpans, scale, num_kv_heads, vdim, block_table
 
 
 def attn_generic(q, k, v, spans: StepSpans, scale, num_kv_heads, vdim, block_tables=None, window=0, softcap=0.0,
-                 sink=None, gate=None):
+                 sink=None, gate=None, keep_first=0):
     """Causal softmax attention for any head sizes and dtypes. q [T, H, dim]; packed mode: k [Tk, G, dim],
     v [Tk, G, vdim] (token-strided views allowed) in the order of spans.cu_k; paged mode (block_tables given):
     k, v are the caches [nb, bs, G*dim], [nb, bs, G*vdim]. Returns [T, H*vdim]. window > 0: position i sees the
-    keys j with 0 <= i - j < window. v None: the values are the first vdim columns of the key rows. softcap > 0:
+    keys j <= i with i - j < window or j < keep_first. v None: the values are the first vdim columns of the key rows. softcap > 0:
     scores become softcap * tanh(score / softcap). sink fp32 [H]: exp(sink[h]) joins the softmax denominator (no key,
     no value). gate [T, H] (q's dtype, row-strided view allowed): head h of token t is multiplied by sigmoid(gate[t, h])."""
     _need_cuda(q, k, v, block_tables, sink, gate)
@@ -992,7 +1008,7 @@ def attn_generic(q, k, v, spans: StepSpans, scale, num_kv_heads, vdim, block_tab
     _C.check(_C.load().b200_attn_generic(out.data_ptr(), q.data_ptr(), q.stride(0) if T > 1 else H * dim,
                                          k.data_ptr(), ks, _ptr(v), vs, bt_ptr, bt_stride, bs, cu_q, cu_k, ctx,
                                          spans.num_seqs, spans.max_q, H, G, dim, vdim, float(scale), int(window),
-                                         float(softcap), _ptr(sink), _ptr(gate),
+                                         int(keep_first), float(softcap), _ptr(sink), _ptr(gate),
                                          (gate.stride(0) if T > 1 else H) if gate is not None else 0, _dt3(q),
                                          _stream()), "b200_attn_generic")
     return out
@@ -1083,39 +1099,53 @@ def rotary_heads(x, positions, heads, width, dims, base, interleaved, out=None, 
     return out
 
 
-def delta_prep(qk, a, b, dt_bias, a_log, num_heads, groups, dim, unit_eps, q_scale):
+def delta_prep(qk, a, b, dt_bias, a_log, num_heads, groups, dim, unit_eps, q_scale, per_head=False):
     """qk [T, 2*groups*dim] (q heads then k heads), a [T, H*dim], b [T, H] (row-strided views allowed) ->
-    (qk fp32 unit vectors with q scaled, decay fp32 [T, H*dim], beta fp32 [T, H])."""
+    (qk fp32 unit vectors with q scaled, decay fp32 [T, H*dim], beta fp32 [T, H]). per_head: one decay per head, a and
+    decay [T, H]."""
     _need_cuda(qk, a, b, dt_bias, a_log)
     _f32(dt_bias, a_log)
     T = qk.shape[0]
-    if qk.shape[1] != 2 * groups * dim or a.shape != (T, num_heads * dim) or b.shape != (T, num_heads):
+    decays = num_heads * (1 if per_head else dim)
+    if qk.shape[1] != 2 * groups * dim or a.shape != (T, decays) or b.shape != (T, num_heads) or dt_bias.numel() != decays:
         raise ValueError("delta_prep shapes")
     if qk.stride(1) != 1 or a.stride(1) != 1 or b.stride(1) != 1 or a.dtype != qk.dtype or b.dtype != qk.dtype:
         raise ValueError("delta_prep inputs: unit inner stride, one dtype")
     dev = qk.device
     qk32 = torch.empty(T, 2 * groups * dim, dtype=torch.float32, device=dev)
-    decay = torch.empty(T, num_heads * dim, dtype=torch.float32, device=dev)
+    decay = torch.empty(T, decays, dtype=torch.float32, device=dev)
     beta = torch.empty(T, num_heads, dtype=torch.float32, device=dev)
     stride = lambda t: t.stride(0) if T > 1 else t.shape[1]
     _C.check(_C.load().b200_delta_prep(qk32.data_ptr(), decay.data_ptr(), beta.data_ptr(), qk.data_ptr(), stride(qk),
                                        a.data_ptr(), stride(a), b.data_ptr(), stride(b), dt_bias.data_ptr(),
                                        a_log.data_ptr(), T, num_heads, groups, dim, float(unit_eps), float(q_scale),
-                                       _dt3(qk), _stream()), "b200_delta_prep")
+                                       1 if per_head else 0, _dt3(qk), _stream()), "b200_delta_prep")
     return qk32, decay, beta
 
 
 def delta_rule(q, k, v, g, beta, spans: StepSpans, num_heads, groups, kdim, vdim, state=None, state_slots=None):
     """Gated delta rule per head (S fp32 [kdim, vdim], carried in state[slot]): S <- diag(g) S; w = beta (v - S^T k);
     S <- S + k w^T; o = S^T q. q, k fp32 [T, groups*kdim] (row-strided views allowed), g fp32 [T, H*kdim], beta fp32
-    [T, H], v [T, H*vdim] in the model dtype. Returns fp32 [T, H*vdim]."""
+    [T, H], v [T, H*vdim] in the model dtype. Returns fp32 [T, H*vdim]. g [T, H]: one decay per head."""
+    per_head = g.shape[1] != num_heads * kdim or kdim == 1
+    return _fp32_state_rule(1 if per_head else 0, q, k, v, g, beta, spans, num_heads, groups, kdim, vdim, state, state_slots)
+
+
+def wkv(r, k, v, decay, bonus, spans: StepSpans, num_heads, kdim, vdim, state=None, state_slots=None):
+    """Per head o_t = S^T r_t + bonus_t v_t; S <- diag(decay_t) S + k_t v_t^T (S fp32 [kdim, vdim], carried in state[slot];
+    the read-out comes before the write). r, k, decay fp32 [T, H*kdim], bonus fp32 [T, H], v [T, H*vdim] in the model
+    dtype. Returns fp32 [T, H*vdim]."""
+    return _fp32_state_rule(2, r, k, v, decay, bonus, spans, num_heads, num_heads, kdim, vdim, state, state_slots)
+
+
+def _fp32_state_rule(mode, q, k, v, g, beta, spans: StepSpans, num_heads, groups, kdim, vdim, state, state_slots):
     _need_cuda(q, k, v, g, beta, state, state_slots)
     _f32(g, beta, state)
     T = q.shape[0]
     for t, n in ((q, groups * kdim), (k, groups * kdim)):
         if t.dtype != torch.float32 or t.shape != (T, n) or t.stride(1) != 1:
             raise ValueError("q, k fp32 [T, groups*kdim] with unit inner stride")
-    if v.shape != (T, num_heads * vdim) or v.stride(1) != 1 or g.shape != (T, num_heads * kdim) or \
+    if v.shape != (T, num_heads * vdim) or v.stride(1) != 1 or g.shape != (T, num_heads * (1 if mode == 1 else kdim)) or \
             beta.shape != (T, num_heads):
         raise ValueError("delta_rule shapes")
     if state is not None and tuple(state.shape[1:]) != (num_heads, kdim, vdim):
@@ -1127,8 +1157,8 @@ def delta_rule(q, k, v, g, beta, spans: StepSpans, num_heads, groups, kdim, vdim
     stride = lambda t: t.stride(0) if T > 1 else t.shape[1]
     _C.check(_C.load().b200_delta_rule(out.data_ptr(), q.data_ptr(), stride(q), k.data_ptr(), stride(k), v.data_ptr(),
                                        stride(v), g.data_ptr(), beta.data_ptr(), _ptr(state), _ptr(state_slots),
-                                       cu_q, cu_k, ctx, spans.num_seqs, num_heads, groups, kdim, vdim, _dt3(v),
-                                       _stream()), "b200_delta_rule")
+                                       cu_q, cu_k, ctx, spans.num_seqs, num_heads, groups, kdim, vdim, mode,
+                                       _dt3(v), _stream()), "b200_delta_rule")
     return out
 
 
@@ -1337,6 +1367,45 @@ def moe_experts_generic(x, w13, w2, topk_weights, plan: MoePlan, act=None, glu=N
 # ---------------------------------------------------------------------------------------------------
 # Scaled residual with a grouped norm, rotary positions from a frequency table fused with value blending and the K/V
 # scatter, and the per-head output gate (csrc/seq_ops.cu).
+def wkv_prep(r, k, z, w0, u, num_heads, dim):
+    """r, k [T, H*dim] (row-strided views allowed), z fp32 [T, H*dim]; w0, u fp32 [H*dim] -> (r fp32, k fp32, decay =
+    exp(-exp(z + w0)) fp32 [T, H*dim], bonus fp32 [T, H] = sum_i r_i u_i k_i per head): what ops.wkv reads besides v."""
+    _need_cuda(r, k, z, w0, u)
+    _f32(z, w0, u)
+    T, n = r.shape
+    if n != num_heads * dim or k.shape != r.shape or z.shape != r.shape or w0.numel() != n or u.numel() != n:
+        raise ValueError("wkv_prep shapes")
+    if r.stride(1) != 1 or k.stride(1) != 1 or k.dtype != r.dtype:
+        raise ValueError("r, k: unit inner stride, one dtype")
+    r32, k32, decay = (torch.empty(T, n, dtype=torch.float32, device=r.device) for _ in range(3))
+    bonus = torch.empty(T, num_heads, dtype=torch.float32, device=r.device)
+    stride = lambda t: t.stride(0) if T > 1 else n
+    _C.check(_C.load().b200_wkv_prep(r32.data_ptr(), k32.data_ptr(), decay.data_ptr(), bonus.data_ptr(), r.data_ptr(),
+                                     stride(r), k.data_ptr(), stride(k), z.data_ptr(), w0.data_ptr(), u.data_ptr(), T,
+                                     num_heads, dim, _dt3(r), _stream()), "b200_wkv_prep")
+    return r32, k32, decay, bonus
+
+
+def token_shift(h, mu, spans: StepSpans, state=None, state_slots=None):
+    """h [T, W] (row-strided view allowed), mu fp32 [M, W] -> [M, T, W]: h_t + (h_(t-1) - h_t) * mu[m], with zeros before a
+    sequence's start. state [slots, W] in h's dtype keeps every sequence's last row between steps."""
+    _need_cuda(h, mu, state, state_slots)
+    _f32(mu)
+    if h.dim() != 2 or h.stride(1) != 1 or mu.dim() != 2 or mu.shape[1] != h.shape[1]:
+        raise ValueError("h [T, W] with unit inner stride, mu [M, W]")
+    T, W = h.shape
+    if state is not None and (state.dtype != h.dtype or not state.is_contiguous() or state.shape[1:] != (W,)):
+        raise ValueError(f"shift state must be a contiguous [slots, {W}] tensor of h's dtype")
+    if state is not None and (state_slots is None or state_slots.dtype != torch.int32):
+        raise TypeError("state_slots must be int32")
+    out = torch.empty(mu.shape[0], T, W, dtype=h.dtype, device=h.device)
+    cu_q, cu_k, ctx = spans.ptrs()
+    _C.check(_C.load().b200_token_shift(out.data_ptr(), T * W, h.data_ptr(), h.stride(0) if T > 1 else W, mu.data_ptr(),
+                                        mu.shape[0], _ptr(state), _ptr(state_slots), cu_q, cu_k, ctx, spans.num_seqs,
+                                        spans.max_q, W, _dt3(h), _stream()), "b200_token_shift")
+    return out
+
+
 def residual_scale_groupnorm_(residual, y, scale, c, w, eps, groups, dtype, offset=0.0, accumulate=True, y_index=None):
     """residual (fp32 [rows, hidden], in place) <- (residual if accumulate else 0) + c * scale * y, with scale fp32
     [hidden] or None and y [rows, hidden] in `dtype` (or, with y_index int64 [rows], a table whose rows are looked up:
@@ -1407,6 +1476,38 @@ def rope_mix_cache(qkv, table, num_heads, num_kv_heads, dim, vdim, dims, interle
         k_cache.data_ptr() if have else None, v_cache.data_ptr() if have else None, slots.data_ptr() if have else None,
         1 if (have and slots.dim() == 2) else 0, bs, T, num_heads, num_kv_heads, dim, vdim, _dt3(qkv), _stream()),
         "b200_rope_mix_cache")
+    return qkv
+
+
+def norm_rope_cache(qkv, wq, wk, eps, table, num_heads, num_kv_heads, dim, vdim, dims, interleaved=True, k_cache=None,
+                    v_cache=None, slots=None):
+    """In place on qkv [T, H*dim | G*dim | G*vdim]: every q (k) head is divided by its root mean square, multiplied by wq
+    (wk), fp32 [dim], and its first `dims` columns are rotated by table [T, dims/2, 2] (rotary_table; None with dims 0); k
+    and v rows are stored at `slots` of the paged caches [nb, bs, G*dim] / [nb, bs, G*vdim] when those are given."""
+    _need_cuda(qkv, wq, wk, table, k_cache, v_cache, slots)
+    _f32(wq, wk)
+    T = qkv.shape[0]
+    if qkv.dim() != 2 or qkv.stride(1) != 1 or qkv.shape[1] != num_heads * dim + num_kv_heads * (dim + vdim):
+        raise ValueError("qkv must be [T, H*dim + G*dim + G*vdim] with unit inner stride")
+    if wq.numel() != dim or wk.numel() != dim:
+        raise ValueError("one norm weight per column of a head")
+    if dims and (table is None or table.dtype != torch.float32 or not table.is_contiguous() or
+                 table.shape != (T, dims // 2, 2)):
+        raise ValueError("table: contiguous fp32 [T, dims/2, 2]")
+    have = k_cache is not None and k_cache.numel() > 0
+    bs = 0
+    if have:
+        _, bs = _cache_dims(k_cache, num_kv_heads * dim)
+        _cache_dims(v_cache, num_kv_heads * vdim)
+        if slots.dtype != torch.int32 or not slots.is_contiguous():
+            raise TypeError("slots must be contiguous int32")
+        if k_cache.dtype != qkv.dtype or v_cache.dtype != qkv.dtype:
+            raise TypeError("caches must have the activations' dtype")
+    _C.check(_C.load().b200_norm_rope_cache(
+        qkv.data_ptr(), qkv.stride(0) if T > 1 else qkv.shape[1], wq.data_ptr(), wk.data_ptr(), float(eps), _ptr(table),
+        int(dims), 1 if interleaved else 0, k_cache.data_ptr() if have else None, v_cache.data_ptr() if have else None,
+        slots.data_ptr() if have else None, 1 if (have and slots.dim() == 2) else 0, bs, T, num_heads, num_kv_heads, dim,
+        vdim, _dt3(qkv), _stream()), "b200_norm_rope_cache")
     return qkv
 
 
