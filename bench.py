@@ -26,7 +26,8 @@ the all-reduce form and its latency, and the same workload at TP=1 (rank 0) for 
 (prefill and decode throughput through the engine) and the rooflines of its kernels beside their like kernels;
 `--hybrid --design nirelix` does the same for the Nirelix decoder beside the Zegopel decoder of the same width, and
 `--hybrid --design fitevik` for the Fitevik decoder beside the Nirelix decoder of the same width, and
-`--hybrid --design nurilorn` for the Nurilorn decoder beside the Zegopel decoder of the same width.
+`--hybrid --design nurilorn` for the Nurilorn decoder beside the Zegopel decoder of the same width, and
+`--hybrid --design pofazen` for the Pofazen decoder beside the Nirelix decoder of the same width.
 """
 from __future__ import annotations
 
@@ -114,8 +115,9 @@ def parse_args():
                     help="model:model,... (default zegopel-1k:qwen3-0.6b,zegopel-2k:llama-3.2-1b; with --design "
                          "nirelix: nirelix-1k:zegopel-1k,nirelix-2k:zegopel-2k; with --design fitevik: "
                          "fitevik-1k:nirelix-1k,fitevik-2k:nirelix-2k; with --design nurilorn: "
-                         "nurilorn-1k:zegopel-1k,nurilorn-2k:zegopel-2k)")
-    ap.add_argument("--design", default="zegopel", choices=["zegopel", "nirelix", "fitevik", "nurilorn"],
+                         "nurilorn-1k:zegopel-1k,nurilorn-2k:zegopel-2k; with --design pofazen: "
+                         "pofazen-1k:nirelix-1k,pofazen-2k:nirelix-2k)")
+    ap.add_argument("--design", default="zegopel", choices=["zegopel", "nirelix", "fitevik", "nurilorn", "pofazen"],
                     help="with --hybrid: whose presets and kernel table are measured")
     ap.add_argument("--kv-cache-dtype", default="auto", choices=["auto", "fp8"],
                     help="fp8: e4m3 KV cache (an extra line; the contract line is the default bf16 cache)")
@@ -1166,6 +1168,161 @@ def nurilorn_kernel_table(width, head_dim, tokens, seqs, peak_gbs):
     return rows
 
 
+def pofazen_kernel_table(width, head_dim, tokens, seqs, peak_gbs):
+    """The kernels that the Pofazen decoder adds or extends, alone, at the layer sizes of a `width`-wide model, as a prompt
+    step (`seqs` x tokens/seqs) and as a decode step (`seqs` rows at that context), each beside the like kernel of the
+    Nirelix, Fitevik or Zegopel decoder. frac = algorithmic bytes / time / measured copy bandwidth."""
+    from nanovllm import ops
+    from nanovllm.layers.seq_mixers import WavelengthScaledRotary
+    dev, bf = "cuda", torch.bfloat16
+    g = torch.Generator(device=dev).manual_seed(0)
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    rnd = lambda *shape: torch.randn(*shape, device=dev, generator=g)
+    H = width // head_dim
+    G = max(1, H // 4)
+    rows = []
+
+    def add(name, step, fn, nbytes, like=None, like_fn=None, like_bytes=None, flops=None, like_flops=None):
+        t = _timed(fn, flush)
+        row = {"kernel": name, "step": step, "us": round(t * 1e6, 1), "GB/s": round(nbytes / t / 1e9),
+               "frac_of_measured_copy": round(nbytes / t / 1e9 / peak_gbs, 3)}
+        if flops:
+            row["TFLOP/s"] = round(flops / t / 1e12, 2)
+        if like_fn is not None:
+            tl = _timed(like_fn, flush)
+            row["like"] = {"kernel": like, "us": round(tl * 1e6, 1),
+                           "frac_of_measured_copy": round(like_bytes / tl / 1e9 / peak_gbs, 3)}
+            row["times_as_far_from_roofline_as_like"] = round((like_bytes / tl) / (nbytes / t), 2)
+            if flops and like_flops:
+                row["like"]["TFLOP/s"] = round(like_flops / tl / 1e12, 2)
+                row["times_as_far_from_flop_roofline_as_like"] = round((like_flops / tl) / (flops / t), 2)
+        rows.append(row)
+
+    rot = WavelengthScaledRotary(head_dim // 2, 5e5, True, {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 2048})
+    for step, T in (("prompt", tokens), ("decode", seqs)):
+        per = T // seqs if step == "prompt" else 1
+        ctx = tokens // seqs
+        if step == "prompt":
+            cu = torch.arange(0, T + 1, per, dtype=torch.int32, device=dev)
+            spans = ops.StepSpans(cu, cu, None, per)
+        else:
+            spans = ops.StepSpans(None, None, torch.full((T,), ctx, dtype=torch.int32, device=dev))
+        slots = torch.arange(seqs, dtype=torch.int32, device=dev)
+        pos = (torch.arange(T, device=dev) % max(per, 1) + (0 if step == "prompt" else ctx - 1)).contiguous()
+        # residual path: the norm of the sum (like: add + two norms of the Zegopel decoder)
+        y, res = rnd(T, width).to(bf), rnd(T, width)
+        w1, w2 = rnd(width), rnd(width)
+        add("norm_residual(norm of the sum)", step,
+            lambda: ops.norm_residual_(res, y, w1, None, 1e-6, bf, kind="rms", carry=1.5), T * width * 12,
+            "residual_add_norms", lambda: ops.residual_add_norms_(y, res, w1, w2, 1e-6), T * width * 12)
+        ff = 3 * width
+        gu = rnd(T, 2 * ff).to(bf)
+        add("act_and_mul(silu)", step, lambda: ops.act_and_mul(gu, "silu"), T * ff * 6,
+            "act_and_mul(relu)", lambda: ops.act_and_mul(gu, "relu"), T * ff * 6)
+        # attention branch: head norms + rotation + scatter (like: unit norms + temperature + scatter of the Zegopel decoder)
+        nq, nk = H * head_dim, G * head_dim
+        C = nq + 2 * nk
+        qkv = rnd(T, C + nq).to(bf)
+        nb = (T + 15) // 16 + 1
+        kc = torch.zeros(nb, 16, nk, dtype=bf, device=dev)
+        vc = torch.zeros(nb, 16, nk, dtype=bf, device=dev)
+        sl = torch.arange(T, dtype=torch.int32, device=dev)
+        tab = ops.rotary_table(pos, rot.freq.to(dev))
+        hw = rnd(head_dim)
+        prep_bytes = T * (2 * (nq + nk) * 2 + nk * 2 + 2 * nk * 2)
+        add("norm_rope_cache", step,
+            lambda: ops.norm_rope_cache(qkv[:, :C], hw, hw, 1e-6, tab, H, G, head_dim, head_dim, rot.dims, True, kc, vc, sl),
+            prep_bytes + T * rot.dims * 4, "unitnorm_temp_cache",
+            lambda: ops.unitnorm_temp_cache(qkv[:, :C], pos, 1e-6, 0.1, 1024, H, G, head_dim, head_dim, kc, vc, sl),
+            prep_bytes)
+        o, wide = rnd(T, nq).to(bf), torch.empty(T, 2 * nq, dtype=bf, device=dev)
+        add("gated_norm(gate alone, scaled slice)", step,
+            lambda: ops.gated_norm(o, qkv[:, C:], None, 1e-6, out=wide[:, :nq], scale=1.2), T * nq * 6,
+            "gated_norm(gate alone)", lambda: ops.gated_norm(o, qkv[:, C:], None, 1e-6), T * nq * 6)
+        # attention over a paged cache in a window of 512 keys and 4 kept ones (like: the same kernels without a window)
+        bs, window, keep = 64, 512, 4
+        per_seq = -(-ctx // bs)
+        nblk = seqs * per_seq
+        tables = torch.randperm(nblk, device=dev, generator=g).to(torch.int32).view(seqs, per_seq)
+        qh = (rnd(T, H, head_dim) * 0.5).to(bf)
+        scale = head_dim ** -0.5
+        see = min(window + keep, ctx)
+        win = dict(window=window, keep_first=keep)
+        kcache, vcache = rnd(nblk + 1, bs, nk).to(bf), rnd(nblk + 1, bs, nk).to(bf)
+        all_bytes = T * 2 * nq * 2 + seqs * ctx * 2 * nk * 2
+        win_bytes = all_bytes if step == "prompt" else T * 2 * nq * 2 + seqs * see * 2 * nk * 2
+        pairs_all = seqs * (per * (per + 1) / 2) if step == "prompt" else seqs * ctx
+        pairs_win = seqs * sum(min(i + 1, window + min(keep, max(0, i + 1 - window))) for i in range(per)) \
+            if step == "prompt" else seqs * see
+        if step == "prompt":
+            fast = lambda v=vcache, dv=head_dim, **kw: ops.prefill_varlen_attn(
+                qh, kcache, v, spans.cu_q, spans.cu_k, per, per, scale, G, block_tables=tables, vdim=dv, **kw)
+            name = "prefill_varlen_attn (tcgen05)"
+        else:
+            fast = lambda v=vcache, dv=head_dim, **kw: ops.paged_decode_attn(
+                qh, kcache, v, tables, spans.ctx_lens, scale, G, vdim=dv, **kw)
+            name = "paged_decode_attn"
+        per_pair = 4.0 * H * head_dim
+        add(name + ", window 512 + 4 kept", step, lambda: fast(**win), win_bytes, name + ", plain", lambda: fast(), all_bytes,
+            flops=pairs_win * per_pair, like_flops=pairs_all * per_pair)
+        dv2 = 192 - head_dim                                       # values unlike keys: 64 beside 128, 128 beside 64
+        vc2 = rnd(nblk + 1, bs, G * dv2).to(bf)
+        add(name + f", window 512 + 4 kept, values of {dv2}", step, lambda: fast(vc2, dv2, **win),
+            win_bytes * (head_dim + dv2) // (2 * head_dim), name + ", plain", lambda: fast(), all_bytes,
+            flops=pairs_win * 2.0 * H * (head_dim + dv2), like_flops=pairs_all * per_pair)
+        generic = lambda **kw: ops.attn_generic(qh, kcache, vcache, spans, scale, G, head_dim, block_tables=tables, **kw)
+        add("attn_generic, window 512 + 4 kept", step, lambda: generic(**win), win_bytes, "attn_generic, plain",
+            lambda: generic(), all_bytes, flops=pairs_win * per_pair, like_flops=pairs_all * per_pair)
+        # delta branch: one decay per head (like: one per key channel, as the Nirelix decoder runs it)
+        Gd = max(1, H // 2)
+        ng = Gd * head_dim
+        qkc = rnd(T, 2 * ng + nq).to(bf)
+        a_ch, a_hd, b_in = rnd(T, nq).to(bf), rnd(T, H).to(bf), rnd(T, H).to(bf)
+        dtb, alog = rnd(nq), -torch.rand(H, device=dev, generator=g) * 2 - 1
+        prep = lambda a, bias, **kw: ops.delta_prep(qkc[:, :2 * ng], a, b_in, bias, alog, H, Gd, head_dim, 1e-6,
+                                                    head_dim ** -0.5, **kw)
+        dtb_h = dtb[:H].contiguous()
+        add("delta_prep, a decay per head", step, lambda: prep(a_hd, dtb_h, per_head=True), T * (2 * ng * 6 + H * 12),
+            "delta_prep, a decay per channel", lambda: prep(a_ch, dtb), T * (2 * ng * 6 + nq * 6 + H * 6))
+        q32, dec_h, beta = prep(a_hd, dtb_h, per_head=True)
+        dec_c = prep(a_ch, dtb)[1]
+        st = torch.zeros(seqs + 1, H, head_dim, head_dim, device=dev)
+        state_bytes = 2 * seqs * H * head_dim * head_dim * 4 if step == "decode" else 0
+        rule = lambda dec: ops.delta_rule(q32[:, :ng], q32[:, ng:], qkc[:, 2 * ng:], dec, beta, spans, H, Gd, head_dim,
+                                          head_dim, st, slots)
+        fl = 8.0 * T * H * head_dim * head_dim
+        add("delta_rule, a decay per head", step, lambda: rule(dec_h), T * (2 * ng * 4 + H * 8 + nq * 6) + state_bytes,
+            "delta_rule, a decay per channel", lambda: rule(dec_c), T * (2 * ng * 4 + nq * 4 + nq * 6) + state_bytes,
+            flops=fl, like_flops=fl)
+        o32, gate, ones = rnd(T, nq), rnd(T, nq).to(bf), torch.ones(nq, device=dev)
+        add("gated_norm(a norm per head, silu gate, scaled slice)", step,
+            lambda: ops.gated_norm(o32, gate, ones, 1e-6, groups=H, gate_act="silu", out=wide[:, nq:], scale=0.7), T * nq * 8,
+            "gated_norm(a norm per head, silu gate)",
+            lambda: ops.gated_norm(o32, gate, ones, 1e-6, groups=H, gate_act="silu"), T * nq * 8)
+        # wkv: mixes with the token before (like: the short convolution), the recurrence's inputs, the recurrence (like:
+        # the tied-gate recurrence of the Fitevik decoder, which also decays per key channel, and its preparation)
+        h, mu = rnd(T, width).to(bf), torch.rand(5, width, device=dev, generator=g)
+        last = torch.zeros(seqs + 1, width, dtype=bf, device=dev)
+        cw = rnd(width, 4)
+        tail = torch.zeros(seqs + 1, 3, width, dtype=bf, device=dev)
+        add("token_shift(5 mixes)", step, lambda: ops.token_shift(h, mu, spans, last, slots), T * width * 12,
+            "causal_conv(4 taps)", lambda: ops.causal_conv(h, cw, None, spans, tail, slots, "silu"), T * width * 4)
+        low = rnd(T, 64).to(bf)
+        add("act_only(tanh, rank 64)", step, lambda: ops.act_only(low, "tanh"), T * 64 * 4,
+            "act_only(relu2)", lambda: ops.act_only(low, "relu2"), T * 64 * 4)
+        rk, z, w0, u = rnd(2, T, nq).to(bf), rnd(T, nq), rnd(nq) - 3, rnd(nq)
+        lower = torch.rand(nq, device=dev, generator=g)
+        add("wkv_prep", step, lambda: ops.wkv_prep(rk[0], rk[1], z, w0, u, H, head_dim), T * (nq * 20 + H * 4),
+            "gate_prep", lambda: ops.gate_prep(rk[0], rk[1], w0, lower), T * nq * 12)
+        r32, k32, decay, bonus = ops.wkv_prep(rk[0], rk[1], z, w0, u, H, head_dim)
+        fl = 6.0 * T * H * head_dim * head_dim
+        add("wkv", step, lambda: ops.wkv(r32, k32, gate, decay, bonus, spans, H, head_dim, head_dim, st, slots),
+            T * nq * 18 + state_bytes, "linear_recurrence(tied gate)",
+            lambda: ops.linear_recurrence(r32, decay, gate, spans, H, H, head_dim, head_dim, st, slots, tied_gate=True),
+            T * nq * 14 + state_bytes, flops=fl, like_flops=fl)
+    return rows
+
+
 def hybrid_compare(args):
     """--hybrid: the Zegopel presets beside the dense presets of the same width and depth, each through the engine
     (LLM.add_request / LLM.step; prompt steps, then CUDA-graph decode steps), plus the kernel table."""
@@ -1181,7 +1338,8 @@ def hybrid_compare(args):
                       "kernel table: 256 MB flush before every timed launch"}, "models": [], "peak_source": peak_src}
     pairs = args.hybrid_pairs or {"nirelix": "nirelix-1k:zegopel-1k,nirelix-2k:zegopel-2k",
                                   "fitevik": "fitevik-1k:nirelix-1k,fitevik-2k:nirelix-2k",
-                                  "nurilorn": "nurilorn-1k:zegopel-1k,nurilorn-2k:zegopel-2k"}.get(
+                                  "nurilorn": "nurilorn-1k:zegopel-1k,nurilorn-2k:zegopel-2k",
+                                  "pofazen": "pofazen-1k:nirelix-1k,pofazen-2k:nirelix-2k"}.get(
         args.design, "zegopel-1k:qwen3-0.6b,zegopel-2k:llama-3.2-1b")
     out["design"] = args.design
     for pair in pairs.split(","):
@@ -1204,7 +1362,7 @@ def hybrid_compare(args):
             del llm
             torch.cuda.empty_cache()
     table = {"nirelix": nirelix_kernel_table, "fitevik": fitevik_kernel_table,
-             "nurilorn": nurilorn_kernel_table}.get(args.design, hybrid_kernel_table)
+             "nurilorn": nurilorn_kernel_table, "pofazen": pofazen_kernel_table}.get(args.design, hybrid_kernel_table)
     out["kernels"] = {"width_1024_head_128": table(1024, 128, 16384, 16, peak),
                       "width_2048_head_64": table(2048, 64, 16384, 16, peak)}
     out["clocks"] = clocks.stop()

@@ -11,12 +11,14 @@
 // steps in a slot, exactly as the other recurrences: [slots, H, kdim, vdim] fp32; a span that starts at position 0
 // ignores what the slot held.
 //
-// One CTA = 128 threads = one (sequence, head) and a band of value columns. A thread owns ONE value column and
-// KPT <= 64 key rows of S in registers (NS = 1, 2 or 4 adjacent lanes share a column when kdim > 64). Per token the delta
-// rule makes two passes over its rows -- decay + the projection S^T k, then the rank-one write + the read-out S^T q --
-// and wkv one, with k, q, g read as float4 broadcasts from shared memory; the dot products are finished with NS - 1
-// shuffles each. Tokens are staged kDeltaTok at a time; where the rows allow 16-byte copies (VEC) the next batch arrives by
-// cp.async in a second set of buffers while the current one is consumed, otherwise batches are loaded in place.
+// One CTA = 32 NS threads = one (sequence, head) and a band of 32 NC value columns. A thread owns NC neighbouring value
+// columns and KPT key rows of S in registers; NS adjacent lanes share the columns, a slice of KPT rows each. Per token the
+// delta rule makes two passes over its rows -- decay + the projection S^T k, then the rank-one write + the read-out S^T q --
+// and wkv one, with k, q, g read as float4 broadcasts from shared memory; the dot products are finished by xor shuffles
+// among the NS lanes. The broadcasts bound the kernel, so a thread uses each of them for NC columns, and the slices of a
+// row lie KPT + 4 floats apart: the NS lanes of a column group read different banks. Tokens are staged kDeltaTok at a
+// time; where the rows allow 16-byte copies (VEC) the next batch arrives by cp.async in a second set of buffers while the
+// current one is consumed, otherwise batches are loaded in place.
 #include "seq_common.cuh"
 
 namespace b200 {
@@ -41,33 +43,33 @@ __device__ __forceinline__ void cp_async_4(uint32_t smem_addr, const void* gptr,
   asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(smem_addr), "l"(gptr), "r"(bytes) : "memory");
 }
 
-template <typename TV, int KPT, int NS, bool VEC, int MODE>
-__global__ void __launch_bounds__(128)
+template <typename TV, int KPT, int NS, int NC, bool VEC, int MODE>
+__global__ void __launch_bounds__(32 * NS)
 delta_rule_kernel(const DeltaParams P) {
   extern __shared__ __align__(16) float smem[];
   pdl_wait();
-  constexpr int KP = NS * KPT;                       // padded key rows
-  constexpr int CC = 128 / NS;                       // value columns per CTA
+  constexpr int NTH = 32 * NS;
+  constexpr int KS = KPT + 4;                        // slice stride: NS lanes, different banks
+  constexpr int KP = NS * KS;                        // row of padded keys
+  constexpr int CC = 32 * NC;                        // value columns per CTA
   const int s = blockIdx.z, h = blockIdx.y;
   const SeqSpan sp = seq_span(P.cu_q, P.cu_k, P.ctx_lens, s);
   if (sp.q_len == 0) return;
   const int kdim = P.kdim, vdim = P.vdim;
-  const int ksl = threadIdx.x % NS, cl = threadIdx.x / NS;
+  const int ksl = threadIdx.x % NS, cl = (threadIdx.x / NS) * NC;
   const int c0 = blockIdx.x * CC, col = c0 + cl;
-  const bool col_ok = col < vdim;
-  const bool warp_live = c0 + (int)((threadIdx.x & ~31u) / NS) < vdim;
   const int grp = h / (P.H / P.groups);
   constexpr int NB = VEC ? 2 : 1;                    // sets of staging buffers
   constexpr int QK = kDeltaTok * KP;
+  constexpr int GT = MODE == kDecayPerHead ? 1 : KP; // decays per token
   float* sq = smem;                                  // [NB][kDeltaTok][KP]
   float* sk = sq + NB * QK;
-  float* sg = sk + NB * QK;
-  constexpr int GT = MODE == kDecayPerHead ? 1 : KP; // decays per token
+  float* sg = sk + NB * QK;                          // [NB][kDeltaTok][GT]
   float* sb = sg + NB * kDeltaTok * GT;              // [NB][kDeltaTok]
   float* sx = sb + NB * kDeltaTok;                   // [kDeltaTok][CC] fp32 (in-place form)
   TV* sxr = reinterpret_cast<TV*>(sb + NB * kDeltaTok);   // [2][kDeltaTok][CC] as stored (cp.async form)
 
-  float S[KPT];
+  float S[NC][KPT];
   float* slot = P.state != nullptr
                     ? P.state + (((int64_t)P.state_slots[s] * P.H + h) * kdim) * (int64_t)vdim
                     : nullptr;
@@ -75,7 +77,9 @@ delta_rule_kernel(const DeltaParams P) {
 #pragma unroll
   for (int r = 0; r < KPT; ++r) {
     const int i = ksl * KPT + r;
-    S[r] = (carried && col_ok && i < kdim) ? slot[(int64_t)i * vdim + col] : 0.f;
+#pragma unroll
+    for (int c = 0; c < NC; ++c)
+      S[c][r] = (carried && col + c < vdim && i < kdim) ? slot[(int64_t)i * vdim + col + c] : 0.f;
   }
   const float* q = P.q + (int64_t)grp * kdim;
   const float* k = P.k + (int64_t)grp * kdim;
@@ -83,22 +87,22 @@ delta_rule_kernel(const DeltaParams P) {
   const TV* v = (const TV*)P.v + (int64_t)h * vdim + c0;
   const int vcols = min(CC, vdim - c0);
   const int64_t g_stride = (int64_t)P.H * (MODE == kDecayPerHead ? 1 : kdim);
+  auto word = [](int i) { return (i / KPT) * KS + i % KPT; };      // key row i of a token's padded row
 
   auto issue = [&](int t0, int b) {                  // cp.async form: batch t0 into buffer set b (zero-filled padding)
     const int nt = min(kDeltaTok, sp.q_len - t0);
     const int64_t tok0 = sp.q_start + t0;
-    constexpr int K4 = KP / 4, VE = 16 / (int)sizeof(TV);
-    for (int e = threadIdx.x; e < kDeltaTok * K4; e += 128) {
+    constexpr int K4 = NS * KPT / 4, VE = 16 / (int)sizeof(TV);
+    for (int e = threadIdx.x; e < kDeltaTok * K4; e += NTH) {
       const int tt = e / K4, i = (e % K4) * 4;
       const bool ok = tt < nt && i < kdim;
       const int64_t tok = tok0 + (tt < nt ? tt : 0);
-      const int ii = ok ? i : 0;
-      cp_async_16(smem_u32(sq + b * QK + tt * KP + i), q + tok * P.q_stride + ii, ok);
-      cp_async_16(smem_u32(sk + b * QK + tt * KP + i), k + tok * P.k_stride + ii, ok);
-      if constexpr (MODE != kDecayPerHead)
-        cp_async_16(smem_u32(sg + b * QK + tt * KP + i), g + tok * g_stride + ii, ok);
+      const int ii = ok ? i : 0, at = b * QK + tt * KP + word(i);
+      cp_async_16(smem_u32(sq + at), q + tok * P.q_stride + ii, ok);
+      cp_async_16(smem_u32(sk + at), k + tok * P.k_stride + ii, ok);
+      if constexpr (MODE != kDecayPerHead) cp_async_16(smem_u32(sg + at), g + tok * g_stride + ii, ok);
     }
-    for (int e = threadIdx.x; e < kDeltaTok * CC / VE; e += 128) {
+    for (int e = threadIdx.x; e < kDeltaTok * CC / VE; e += NTH) {
       const int tt = e / (CC / VE), c = (e % (CC / VE)) * VE;
       const bool ok = tt < nt && c < vcols;
       cp_async_16(smem_u32(sxr + (b * kDeltaTok + tt) * CC + c), v + (tok0 + (tt < nt ? tt : 0)) * P.v_stride + (ok ? c : 0), ok);
@@ -122,14 +126,14 @@ delta_rule_kernel(const DeltaParams P) {
       if (t0 + kDeltaTok < sp.q_len) issue(t0 + kDeltaTok, b ^ 1);
     } else {
       __syncthreads();                               // the previous batch has been consumed
-      for (int e = threadIdx.x; e < kDeltaTok * KP; e += 128) {
-        const int tt = e / KP, i = e % KP;
+      for (int e = threadIdx.x; e < kDeltaTok * NS * KPT; e += NTH) {
+        const int tt = e / (NS * KPT), i = e % (NS * KPT), at = tt * KP + word(i);
         const bool ok = tt < nt && i < kdim;
-        sq[e] = ok ? q[(tok0 + tt) * P.q_stride + i] : 0.f;
-        sk[e] = ok ? k[(tok0 + tt) * P.k_stride + i] : 0.f;
-        if constexpr (MODE != kDecayPerHead) sg[e] = ok ? g[(tok0 + tt) * g_stride + i] : 0.f;
+        sq[at] = ok ? q[(tok0 + tt) * P.q_stride + i] : 0.f;
+        sk[at] = ok ? k[(tok0 + tt) * P.k_stride + i] : 0.f;
+        if constexpr (MODE != kDecayPerHead) sg[at] = ok ? g[(tok0 + tt) * g_stride + i] : 0.f;
       }
-      for (int e = threadIdx.x; e < kDeltaTok * CC; e += 128) {
+      for (int e = threadIdx.x; e < kDeltaTok * CC; e += NTH) {
         const int tt = e / CC, c = e % CC;
         sx[e] = (tt < nt && c < vcols) ? to_f32<TV>(v[(tok0 + tt) * P.v_stride + c]) : 0.f;
       }
@@ -139,108 +143,137 @@ delta_rule_kernel(const DeltaParams P) {
       }
       __syncthreads();
     }
-    if (!warp_live) continue;
     float* outp = P.out + tok0 * ((int64_t)P.H * vdim) + (int64_t)h * vdim + col;
     for (int tt = 0; tt < nt; ++tt) {
-      const float4* q4 = reinterpret_cast<const float4*>(sq + b * QK + tt * KP + ksl * KPT);
-      const float4* k4 = reinterpret_cast<const float4*>(sk + b * QK + tt * KP + ksl * KPT);
-      const float4* g4 = reinterpret_cast<const float4*>(sg + b * kDeltaTok * GT + tt * GT + ksl * (MODE == kDecayPerHead ? 0 : KPT));
-      const float x = VEC ? to_f32<TV>(sxr[(b * kDeltaTok + tt) * CC + cl]) : sx[tt * CC + cl];
-      float o0 = 0.f, o1 = 0.f, o2 = 0.f, o3 = 0.f, o_now = 0.f;
+      const int at = b * QK + tt * KP + ksl * KS;
+      const float4* q4 = reinterpret_cast<const float4*>(sq + at);
+      const float4* k4 = reinterpret_cast<const float4*>(sk + at);
+      const float4* g4 = reinterpret_cast<const float4*>(sg + at);       // (one decay per head: not read)
+      const float coef = sb[b * kDeltaTok + tt];
+      float x[NC], o[NC][2];                         // two partial sums per column
+#pragma unroll
+      for (int c = 0; c < NC; ++c) {
+        x[c] = VEC ? to_f32<TV>(sxr[(b * kDeltaTok + tt) * CC + cl + c]) : sx[tt * CC + cl + c];
+        o[c][0] = o[c][1] = 0.f;
+      }
       if constexpr (MODE == kWkv) {
 #pragma unroll
         for (int r4 = 0; r4 < KPT / 4; ++r4) {
           const float4 gg = g4[r4], kk = k4[r4], qq = q4[r4];
-          o0 += S[r4 * 4 + 0] * qq.x;
-          S[r4 * 4 + 0] = fmaf(S[r4 * 4 + 0], gg.x, kk.x * x);
-          o1 += S[r4 * 4 + 1] * qq.y;
-          S[r4 * 4 + 1] = fmaf(S[r4 * 4 + 1], gg.y, kk.y * x);
-          o2 += S[r4 * 4 + 2] * qq.z;
-          S[r4 * 4 + 2] = fmaf(S[r4 * 4 + 2], gg.z, kk.z * x);
-          o3 += S[r4 * 4 + 3] * qq.w;
-          S[r4 * 4 + 3] = fmaf(S[r4 * 4 + 3], gg.w, kk.w * x);
+#pragma unroll
+          for (int c = 0; c < NC; ++c) {
+            float* Sc = S[c] + r4 * 4;
+            o[c][0] += Sc[0] * qq.x;
+            Sc[0] = fmaf(Sc[0], gg.x, kk.x * x[c]);
+            o[c][1] += Sc[1] * qq.y;
+            Sc[1] = fmaf(Sc[1], gg.y, kk.y * x[c]);
+            o[c][0] += Sc[2] * qq.z;
+            Sc[2] = fmaf(Sc[2], gg.z, kk.z * x[c]);
+            o[c][1] += Sc[3] * qq.w;
+            Sc[3] = fmaf(Sc[3], gg.w, kk.w * x[c]);
+          }
         }
-        o_now = sb[b * kDeltaTok + tt] * x;
       } else {
-      const float g1 = MODE == kDecayPerHead ? sg[b * kDeltaTok + tt] : 0.f;
-      float d0 = 0.f, d1 = 0.f, d2 = 0.f, d3 = 0.f;
+        const float g1 = MODE == kDecayPerHead ? sg[b * kDeltaTok + tt] : 0.f;
+        float d[NC][2];
 #pragma unroll
-      for (int r4 = 0; r4 < KPT / 4; ++r4) {
-        const float4 kk = k4[r4];
-        const float4 gg = MODE == kDecayPerHead ? make_float4(g1, g1, g1, g1) : g4[r4];
-        S[r4 * 4 + 0] *= gg.x;
-        d0 += S[r4 * 4 + 0] * kk.x;
-        S[r4 * 4 + 1] *= gg.y;
-        d1 += S[r4 * 4 + 1] * kk.y;
-        S[r4 * 4 + 2] *= gg.z;
-        d2 += S[r4 * 4 + 2] * kk.z;
-        S[r4 * 4 + 3] *= gg.w;
-        d3 += S[r4 * 4 + 3] * kk.w;
+        for (int c = 0; c < NC; ++c) d[c][0] = d[c][1] = 0.f;
+#pragma unroll
+        for (int r4 = 0; r4 < KPT / 4; ++r4) {
+          const float4 kk = k4[r4];
+          const float4 gg = MODE == kDecayPerHead ? make_float4(g1, g1, g1, g1) : g4[r4];
+#pragma unroll
+          for (int c = 0; c < NC; ++c) {
+            float* Sc = S[c] + r4 * 4;
+            Sc[0] *= gg.x;
+            d[c][0] += Sc[0] * kk.x;
+            Sc[1] *= gg.y;
+            d[c][1] += Sc[1] * kk.y;
+            Sc[2] *= gg.z;
+            d[c][0] += Sc[2] * kk.z;
+            Sc[3] *= gg.w;
+            d[c][1] += Sc[3] * kk.w;
+          }
+        }
+#pragma unroll
+        for (int c = 0; c < NC; ++c) {
+          float dc = d[c][0] + d[c][1];
+#pragma unroll
+          for (int off = 1; off < NS; off <<= 1) dc += __shfl_xor_sync(0xffffffffu, dc, off);
+          x[c] = coef * (x[c] - dc);                 // what is written
+        }
+#pragma unroll
+        for (int r4 = 0; r4 < KPT / 4; ++r4) {
+          const float4 kk = k4[r4], qq = q4[r4];
+#pragma unroll
+          for (int c = 0; c < NC; ++c) {
+            float* Sc = S[c] + r4 * 4;
+            Sc[0] += kk.x * x[c];
+            o[c][0] += Sc[0] * qq.x;
+            Sc[1] += kk.y * x[c];
+            o[c][1] += Sc[1] * qq.y;
+            Sc[2] += kk.z * x[c];
+            o[c][0] += Sc[2] * qq.z;
+            Sc[3] += kk.w * x[c];
+            o[c][1] += Sc[3] * qq.w;
+          }
+        }
       }
-      float d = (d0 + d1) + (d2 + d3);
 #pragma unroll
-      for (int off = 1; off < NS; off <<= 1) d += __shfl_xor_sync(0xffffffffu, d, off);
-      const float w = sb[b * kDeltaTok + tt] * (x - d);
+      for (int c = 0; c < NC; ++c) {
+        float oc = o[c][0] + o[c][1];
 #pragma unroll
-      for (int r4 = 0; r4 < KPT / 4; ++r4) {
-        const float4 kk = k4[r4], qq = q4[r4];
-        S[r4 * 4 + 0] += kk.x * w;
-        o0 += S[r4 * 4 + 0] * qq.x;
-        S[r4 * 4 + 1] += kk.y * w;
-        o1 += S[r4 * 4 + 1] * qq.y;
-        S[r4 * 4 + 2] += kk.z * w;
-        o2 += S[r4 * 4 + 2] * qq.z;
-        S[r4 * 4 + 3] += kk.w * w;
-        o3 += S[r4 * 4 + 3] * qq.w;
+        for (int off = 1; off < NS; off <<= 1) oc += __shfl_xor_sync(0xffffffffu, oc, off);
+        if (MODE == kWkv) oc += coef * x[c];
+        if (ksl == c % NS && col + c < vdim) outp[(int64_t)tt * ((int64_t)P.H * vdim) + c] = oc;
       }
-      }
-      float o = (o0 + o1) + (o2 + o3);
-#pragma unroll
-      for (int off = 1; off < NS; off <<= 1) o += __shfl_xor_sync(0xffffffffu, o, off);
-      if (ksl == 0 && col_ok) outp[(int64_t)tt * ((int64_t)P.H * vdim)] = o + o_now;
     }
   }
-  if (slot != nullptr && col_ok) {
+  if (slot != nullptr) {
 #pragma unroll
     for (int r = 0; r < KPT; ++r) {
       const int i = ksl * KPT + r;
-      if (i < kdim) slot[(int64_t)i * vdim + col] = S[r];
+#pragma unroll
+      for (int c = 0; c < NC; ++c)
+        if (i < kdim && col + c < vdim) slot[(int64_t)i * vdim + col + c] = S[c][r];
     }
   }
 }
 
-template <typename TV, int KPT, int NS, int MODE>
+template <typename TV, int KPT, int NS, int NC, int MODE>
 static void delta_launch_as(const DeltaParams& P, int num_seqs, cudaStream_t stream) {
-  constexpr int CC = 128 / NS;
+  constexpr int CC = 32 * NC, KP = NS * (KPT + 4);
   constexpr int VE = 16 / (int)sizeof(TV);
   const dim3 grid((P.vdim + CC - 1) / CC, P.H, num_seqs);
-  constexpr int GT = MODE == kDecayPerHead ? 1 : NS * KPT;
+  constexpr int GT = MODE == kDecayPerHead ? 1 : KP;
   const bool vec = P.kdim % 4 == 0 && P.q_stride % 4 == 0 && P.k_stride % 4 == 0 && aligned16(P.q) && aligned16(P.k) &&
                    (MODE == kDecayPerHead || aligned16(P.g)) && P.vdim % VE == 0 && P.v_stride % VE == 0 && aligned16(P.v);
   if (vec) {
-    const size_t smem = (size_t)2 * kDeltaTok * (2 * NS * KPT + GT + 1) * sizeof(float) +
-                        (size_t)2 * kDeltaTok * CC * sizeof(TV);
+    const size_t smem = (size_t)2 * kDeltaTok * (2 * KP + GT + 1) * sizeof(float) + (size_t)2 * kDeltaTok * CC * sizeof(TV);
     static bool configured = false;                   // one flag per instantiation
     if (!configured && smem > 48 * 1024) {
-      cudaFuncSetAttribute(delta_rule_kernel<TV, KPT, NS, true, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      cudaFuncSetAttribute(delta_rule_kernel<TV, KPT, NS, NC, true, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
       configured = true;
     }
-    launch_pdl(delta_rule_kernel<TV, KPT, NS, true, MODE>, grid, dim3(128), smem, stream, P);
+    launch_pdl(delta_rule_kernel<TV, KPT, NS, NC, true, MODE>, grid, dim3(32 * NS), smem, stream, P);
   } else {
-    const size_t smem = (size_t)kDeltaTok * (2 * NS * KPT + GT + 1 + CC) * sizeof(float);
-    launch_pdl(delta_rule_kernel<TV, KPT, NS, false, MODE>, grid, dim3(128), smem, stream, P);
+    const size_t smem = (size_t)kDeltaTok * (2 * KP + GT + 1 + CC) * sizeof(float);
+    launch_pdl(delta_rule_kernel<TV, KPT, NS, NC, false, MODE>, grid, dim3(32 * NS), smem, stream, P);
   }
 }
 
 template <typename TV, int MODE>
 static int delta_launch(const DeltaParams& P, int num_seqs, cudaStream_t stream) {
-  // 64 rows per thread wherever the key size allows: 32 rows on twice the lanes measured 3.6x slower at key size 128
-  // (the lanes of a column then read four different slices of k, q, g per token instead of two)
-  if (P.kdim <= 16) delta_launch_as<TV, 16, 1, MODE>(P, num_seqs, stream);
-  else if (P.kdim <= 32) delta_launch_as<TV, 32, 1, MODE>(P, num_seqs, stream);
-  else if (P.kdim <= 64) delta_launch_as<TV, 64, 1, MODE>(P, num_seqs, stream);
-  else if (P.kdim <= 128) delta_launch_as<TV, 64, 2, MODE>(P, num_seqs, stream);
-  else delta_launch_as<TV, 64, 4, MODE>(P, num_seqs, stream);
+  // measured on 16 x 1024-token prompts, us at 8 heads of 128 / 32 heads of 64 (rows x columns per thread): delta rule with
+  // a decay per head 64x1 601 / 566, 32x1 871 / 742, 32x2 523 / 480, 16x4 589 / 1035; wkv 64x1 564 / 501, 32x2 589 / 521,
+  // 16x4 406 / 755. Decode steps of 256 rows: 32x2 72 / 67, 16x4 120 / 81.
+  if (P.kdim <= 16) delta_launch_as<TV, 16, 1, 1, MODE>(P, num_seqs, stream);
+  else if (P.kdim <= 32) delta_launch_as<TV, 32, 1, 1, MODE>(P, num_seqs, stream);
+  else if (P.kdim <= 64) delta_launch_as<TV, 32, 2, 2, MODE>(P, num_seqs, stream);
+  else if (P.kdim <= 128) {
+    if (MODE == kWkv && P.cu_q != nullptr) delta_launch_as<TV, 16, 8, 4, MODE>(P, num_seqs, stream);
+    else delta_launch_as<TV, 32, 4, 2, MODE>(P, num_seqs, stream);
+  } else delta_launch_as<TV, 32, 8, 2, MODE>(P, num_seqs, stream);
   return finish_launch();
 }
 
