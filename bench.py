@@ -1270,6 +1270,19 @@ def pofazen_kernel_table(width, head_dim, tokens, seqs, peak_gbs):
         add(name + f", window 512 + 4 kept, values of {dv2}", step, lambda: fast(vc2, dv2, **win),
             win_bytes * (head_dim + dv2) // (2 * head_dim), name + ", plain", lambda: fast(), all_bytes,
             flops=pairs_win * 2.0 * H * (head_dim + dv2), like_flops=pairs_all * per_pair)
+        if step == "decode":                # enough rows that the cache bytes, not the two launches, are the time
+            R = 256
+            lens = torch.full((R,), ctx, dtype=torch.int32, device=dev)
+            qm = (rnd(R, H, head_dim) * 0.5).to(bf)
+            big = [rnd(R * per_seq, bs, G * n).to(bf) for n in (head_dim, head_dim, dv2)]
+            many = torch.randperm(R * per_seq, device=dev, generator=g).to(torch.int32).view(R, per_seq)
+            run = lambda i, dv, **kw: ops.paged_decode_attn(qm, big[0], big[i], many, lens, scale, G, vdim=dv, **kw)
+            io = lambda dv, keys: R * nq * 2 * (head_dim + dv) // head_dim + R * keys * G * (head_dim + dv) * 2
+            add("paged_decode_attn, 256 rows, window 512 + 4 kept", step, lambda: run(1, head_dim, **win), io(head_dim, see),
+                "paged_decode_attn, 256 rows, plain", lambda: run(1, head_dim), io(head_dim, ctx))
+            add(f"paged_decode_attn, 256 rows, window 512 + 4 kept, values of {dv2}", step, lambda: run(2, dv2, **win),
+                io(dv2, see), "paged_decode_attn, 256 rows, plain", lambda: run(1, head_dim), io(head_dim, ctx))
+            del big
         generic = lambda **kw: ops.attn_generic(qh, kcache, vcache, spans, scale, G, head_dim, block_tables=tables, **kw)
         add("attn_generic, window 512 + 4 kept", step, lambda: generic(**win), win_bytes, "attn_generic, plain",
             lambda: generic(), all_bytes, flops=pairs_win * per_pair, like_flops=pairs_all * per_pair)
