@@ -584,8 +584,8 @@ int b200_attn_generic(void* out, const void* q, int64_t q_stride, const void* k,
                       const void* v, int64_t v_stride, const int32_t* block_tables, int32_t bt_stride,
                       int32_t block_size, const int32_t* cu_q, const int32_t* cu_k, const int32_t* ctx_lens,
                       int32_t num_seqs, int32_t max_q, int32_t num_heads, int32_t num_kv_heads, int32_t dim,
-                      int32_t vdim, float scale, int32_t window, int32_t keep_first, float softcap, const float* sink, const void* gate,
-                      int64_t gate_stride, int32_t dtype, b200_stream_t stream);
+                      int32_t vdim, float scale, int32_t window, int32_t keep_first, float softcap, const float* sink,
+                      const void* gate, int64_t gate_stride, int32_t dtype, b200_stream_t stream);
 
 /* Per head S_t = a_t S_(t-1) + k_t (b_t v_t)^T, o_t = S_t^T q_t; S fp32 [kdim, vdim] in state
  * [slots, H, kdim, vdim]. q, k [T, groups*kdim] (head h reads group h / (H / groups)), v [T, H*vdim];

@@ -252,7 +252,8 @@ static void delta_launch_as(const DeltaParams& P, int num_seqs, cudaStream_t str
     const size_t smem = (size_t)2 * kDeltaTok * (2 * KP + GT + 1) * sizeof(float) + (size_t)2 * kDeltaTok * CC * sizeof(TV);
     static bool configured = false;                   // one flag per instantiation
     if (!configured && smem > 48 * 1024) {
-      cudaFuncSetAttribute(delta_rule_kernel<TV, KPT, NS, NC, true, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      cudaFuncSetAttribute(delta_rule_kernel<TV, KPT, NS, NC, true, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                           (int)smem);
       configured = true;
     }
     launch_pdl(delta_rule_kernel<TV, KPT, NS, NC, true, MODE>, grid, dim3(32 * NS), smem, stream, P);

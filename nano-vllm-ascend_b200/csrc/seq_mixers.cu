@@ -3,8 +3,8 @@
 //   attn_generic       causal softmax attention for ANY head sizes (key size != value size, sizes that are
 //                      not 64 or 128), any element type including fp32, packed or paged keys, and any mix of
 //                      prompt portions and single tokens in one launch. fp32 scores, softmax and accumulation.
-//                      Optional: a sliding window (with first tokens that stay visible), scores capped by cap * tanh(s / cap), a sink logit per head that
-//                      joins the softmax denominator without a value, an output gate sigmoid(logit) per (token, head).
+//                      Optional: a sliding window (with first tokens that stay visible), scores capped by
+//                      cap * tanh(s / cap), a sink logit per head that joins the softmax denominator without a value, an output gate sigmoid(logit) per (token, head).
 //   linear_recurrence  S_t = a_t S_(t-1) + k_t (b_t v_t)^T, o_t = S_t^T q_t (+ d v_t) per head with the state S
 //                      [key size x value size] held in fp32 registers and carried between steps in a slot.
 //                      Three forms: a constant decay per head (lightning attention), a decay and a step size
@@ -662,8 +662,8 @@ extern "C" int b200_attn_generic(void* out, const void* q, int64_t q_stride, con
                                  int32_t bt_stride, int32_t block_size, const int32_t* cu_q,
                                  const int32_t* cu_k, const int32_t* ctx_lens, int32_t num_seqs, int32_t max_q,
                                  int32_t num_heads, int32_t num_kv_heads, int32_t dim, int32_t vdim,
-                                 float scale, int32_t window, int32_t keep_first, float softcap, const float* sink, const void* gate,
-                                 int64_t gate_stride, int32_t dtype, b200_stream_t stream) {
+                                 float scale, int32_t window, int32_t keep_first, float softcap,
+                                 const float* sink, const void* gate, int64_t gate_stride, int32_t dtype, b200_stream_t stream) {
   B200_RETURN_IF(num_seqs < 0 || max_q < 0 || num_heads <= 0 || num_kv_heads <= 0 || dim <= 0 || vdim <= 0 ||
                      num_heads % num_kv_heads != 0, B200_ERR_BAD_SHAPE);
   B200_RETURN_IF(vdim > 32 * kAttnMaxVChunks, B200_ERR_UNSUPPORTED);
