@@ -129,13 +129,14 @@ int b200_paged_decode_attn_capped(void* out, const void* q, const void* k_cache,
                                   void* workspace, size_t workspace_bytes, int32_t num_ctas, int32_t dtype,
                                   b200_stream_t stream);
 /* The general form: keys of head_dim and values of value_dim (each 64 or 128; the workspace is sized by value_dim);
- * window > 0: a row of n keys sees the last `window` of them and those below keep_first (window 0: all). */
+ * window > 0: a row of n keys sees the last `window` of them and those below keep_first (window 0: all); chunk > 0 (without a
+ * window): a row sees the keys of its own chunk, counted from position 0. */
 int b200_paged_decode_attn_windowed(void* out, const void* q, const void* k_cache, const void* v_cache,
                                     const int32_t* block_tables, const int32_t* context_lens, int32_t batch,
                                     int32_t num_heads, int32_t num_kv_heads, int32_t head_dim, int32_t value_dim,
                                     int64_t q_stride, int64_t out_stride, int32_t num_blocks, int32_t block_size,
                                     int32_t block_table_stride, float scale, float softcap, const float* sink,
-                                    int32_t window, int32_t keep_first, void* workspace, size_t workspace_bytes,
+                                    int32_t window, int32_t keep_first, int32_t chunk, void* workspace, size_t workspace_bytes,
                                     int32_t num_ctas, int32_t dtype, b200_stream_t stream);
 
 
@@ -222,7 +223,7 @@ int b200_prefill_varlen_attn_capped(void* out, const void* q, const void* k, con
 
 /* The general form: keys of head_dim and values of value_dim (each 64 or 128; out [total_q, num_heads*value_dim], v rows and
  * caches value_dim wide per head); window > 0: the query at position i sees keys j <= i with i - j < window or
- * j < keep_first (window 0: every earlier key). Served by the tcgen05 kernel only, like the capped form. */
+ * j < keep_first (window 0: every earlier key); chunk > 0 (without a window): those with j / chunk == i / chunk. Served by the tcgen05 kernel only, like the capped form. */
 int b200_prefill_varlen_attn_windowed(void* out, const void* q, const void* k, const void* v,
                                       const int32_t* cu_seqlens_q, const int32_t* cu_seqlens_k, int32_t num_seqs,
                                       int32_t total_q, int32_t total_k, int32_t max_seqlen_q, int32_t max_seqlen_k,
@@ -230,7 +231,7 @@ int b200_prefill_varlen_attn_windowed(void* out, const void* q, const void* k, c
                                       int64_t q_stride, int64_t k_stride, int64_t v_stride, int64_t out_stride,
                                       const int32_t* block_tables, int32_t block_table_stride, int32_t num_blocks,
                                       int32_t block_size, float scale, float softcap, const float* sink, int32_t window,
-                                      int32_t keep_first, int32_t dtype, void* workspace, int64_t workspace_bytes,
+                                      int32_t keep_first, int32_t chunk, int32_t dtype, void* workspace, int64_t workspace_bytes,
                                       b200_stream_t stream);
 
 /* Bytes of split-KV workspace that let b200_prefill_varlen_attn use every SM for ANY launch it would
@@ -286,7 +287,7 @@ int b200_silu_and_mul(void* out, const void* x, int32_t rows, int32_t inter, int
 /* f2 (SURVEY 8f "next"): greedy/temperature sampling tail without the fp32 logits
  * round trip. Replaces layers/sampler.py:9-17 for the greedy parity path (argmax) and
  * for temperature sampling via the Gumbel-max trick with a counter-based RNG.
- * logits: [rows, vocab] in dtype (row stride logits_stride elements);
+ * logits: [rows, vocab] in dtype (16-bit or fp32; row stride logits_stride elements);
  * temperatures: [rows] fp32 or NULL; a row whose temperature is NULL/<= 0 takes the argmax.
  * out_tokens: [rows] int64. step_offset: optional DEVICE int64 added to `step` at run time, so
  * a captured CUDA graph draws fresh randomness on every replay (NULL = none).
@@ -326,8 +327,10 @@ int b200_sample_shard(int64_t* out_keys, const void* logits, const float* temper
  *   pos_of_pair int32 [num_pairs] (-1 = not local); counts int32 [num_local] is scratch.
  * b200_moe_gemm_gate_up: h[pos, :inter] = SiluAndMul(x[sorted_pair[pos] / top_k] . w13[e]^T) for the
  *   rows pos of every local expert e; w13 [num_local, 2*inter, hidden] (gate rows, then up rows);
- *   hidden % 64 == 0, inter % 64 == 0.
- * b200_moe_gemm_down: y[pos, :hidden] = (h[pos] . w2[e]^T in dtype) * topk_weights[sorted_pair[pos]];
+ *   hidden % 64 == 0, inter % 64 == 0. in_scale (fp32 [tokens * top_k] or NULL): a weight per pair on the expert's
+ *   input row (it multiplies both products in fp32).
+ * b200_moe_gemm_down: y[pos, :hidden] = (h[pos] . w2[e]^T in dtype) * topk_weights[sorted_pair[pos]]
+ *   (topk_weights NULL: 1);
  *   w2 [num_local, hidden, inter]; inter % 64 == 0, hidden % 128 == 0.
  * b200_moe_combine: out[t] = sum of y[pos_of_pair[t, j]] over t's local pairs in ascending expert
  *   order, rounded to dtype after every add (index_add_ semantics); zeros when none is local.
@@ -339,7 +342,7 @@ int b200_moe_align(int32_t* offsets, int32_t* sorted_pair, int32_t* pos_of_pair,
                    const int32_t* topk_ids, int32_t num_pairs, int32_t expert_begin,
                    int32_t num_local, b200_stream_t stream);
 int b200_moe_gemm_gate_up(void* h, const void* x, const void* w13, const int32_t* offsets,
-                          const int32_t* sorted_pair, int32_t hidden, int32_t inter,
+                          const int32_t* sorted_pair, const float* in_scale, int32_t hidden, int32_t inter,
                           int32_t num_local, int32_t top_k, int64_t x_stride, int32_t dtype,
                           b200_stream_t stream);
 /* b200_moe_gemm_gate_up with the clamped unit in its epilogue: h = g sigmoid(alpha g) (u + 1) with g = min(x Wg^T,
@@ -375,7 +378,7 @@ int b200_moe_gather_rows(void* xs, const void* x, const int32_t* offsets, const 
                          int32_t pairs, int32_t num_local, int32_t top_k, int32_t hidden,
                          int64_t x_stride, int32_t dtype, b200_stream_t stream);
 int b200_moe_gemm_gate_up_umma(void* h, const void* xs, const void* w13, const int32_t* offsets,
-                               int32_t pairs, int32_t hidden, int32_t inter, int32_t num_local,
+                               const int32_t* sorted_pair, const float* in_scale, int32_t pairs, int32_t hidden, int32_t inter, int32_t num_local,
                                int32_t dtype, b200_stream_t stream);
 int b200_moe_gemm_down_umma(void* y, const void* h, const void* w2, const int32_t* offsets,
                             const int32_t* sorted_pair, const void* topk_weights, int32_t pairs,
@@ -568,14 +571,15 @@ int b200_mixed_attn(void* out, const void* q, int64_t q_stride, const void* k, i
                     int32_t window, const float* slopes, const float* talk, const float* sink, int32_t dtype,
                     b200_stream_t stream);
 
-/* out[r, i] = act(x[r, i]) * x[r, inter + i]; act: 0 silu, 1 relu, 2 gelu (tanh form). */
-int b200_act_and_mul(void* out, const void* x, int32_t rows, int32_t inter, int32_t act, int32_t dtype,
+/* out[r, i] = act(x[r, i]) * x[r, inter + i] (x_stride elements between rows); act: 0 silu, 1 relu, 2 gelu (tanh form). */
+int b200_act_and_mul(void* out, const void* x, int64_t x_stride, int32_t rows, int32_t inter, int32_t act, int32_t dtype,
                      b200_stream_t stream);
 
 /* Causal softmax attention for any key size `dim` and value size `vdim` (<= 512), packed keys
  * (block_tables == NULL: k, v are this step's rows in the order of cu_k) or paged caches
  * [nb, bs, G*dim] / [nb, bs, G*vdim]. q [T, H, dim] -> out [T, H*vdim]. fp32 scores and accumulation.
- * window > 0: the query at position i sees keys j <= i with i - j < window or j < keep_first. v == NULL: the values are the
+ * window > 0: the query at position i sees keys j <= i with i - j < window or j < keep_first; chunk > 0 (without a window):
+ * those with j / chunk == i / chunk. v == NULL: the values are the
  * first vdim columns of the key rows (one cached latent row serves as key and as value; vdim <= dim).
  * softcap > 0: scores become softcap * tanh(score / softcap). sink (fp32 [H] or NULL): exp(sink[h]) joins the softmax
  * denominator without a value. gate ([T, gate_stride] of dtype, or NULL): head h of token t is multiplied by
@@ -584,8 +588,8 @@ int b200_attn_generic(void* out, const void* q, int64_t q_stride, const void* k,
                       const void* v, int64_t v_stride, const int32_t* block_tables, int32_t bt_stride,
                       int32_t block_size, const int32_t* cu_q, const int32_t* cu_k, const int32_t* ctx_lens,
                       int32_t num_seqs, int32_t max_q, int32_t num_heads, int32_t num_kv_heads, int32_t dim,
-                      int32_t vdim, float scale, int32_t window, int32_t keep_first, float softcap, const float* sink,
-                      const void* gate, int64_t gate_stride, int32_t dtype, b200_stream_t stream);
+                      int32_t vdim, float scale, int32_t window, int32_t keep_first, int32_t chunk, float softcap,
+                      const float* sink, const void* gate, int64_t gate_stride, int32_t dtype, b200_stream_t stream);
 
 /* Per head S_t = a_t S_(t-1) + k_t (b_t v_t)^T, o_t = S_t^T q_t; S fp32 [kdim, vdim] in state
  * [slots, H, kdim, vdim]. q, k [T, groups*kdim] (head h reads group h / (H / groups)), v [T, H*vdim];
@@ -624,10 +628,10 @@ int b200_stream_mix_norm(void* h, float* x, const void* y, const float* mix, con
  * angle pos * base^(-2i/dims) in pairs (2i, 2i+1) (interleaved) or (i, i + dims/2), the rest pass; heads below
  * `split` are multiplied by scale_lo, the others by scale_hi (after the rotation). Head hd of token t is read at
  * in + t * in_stride + hd * in_head and written at out + t * out_stride + hd * out_head, as fp32 (out_f32) or
- * dtype. Angles are computed in fp64. */
+ * dtype. Angles are computed in fp64; table (fp32 [tokens, dims/2, 2], cos and sin) replaces them when given. */
 int b200_rotary_heads(void* out, int64_t out_stride, int32_t out_head, int32_t out_f32, const void* in,
-                      int64_t in_stride, int32_t in_head, const int64_t* positions, int32_t tokens,
-                      int32_t heads, int32_t width, int32_t dims, double base, int32_t interleaved,
+                      int64_t in_stride, int32_t in_head, const int64_t* positions, const float* table,
+                      int32_t tokens, int32_t heads, int32_t width, int32_t dims, double base, int32_t interleaved,
                       int32_t split, float scale_lo, float scale_hi, int32_t dtype, b200_stream_t stream);
 
 /* Inputs of b200_delta_rule from projected activations: qk [T, 2*groups*dim] fp32 = q and k heads of qk_in
@@ -656,13 +660,13 @@ int b200_wkv_prep(float* r_out, float* k_out, float* decay, float* bonus, const 
                   const void* k, int64_t k_stride, const float* z, const float* w0, const float* u, int32_t tokens,
                   int32_t num_heads, int32_t dim, int32_t dtype, b200_stream_t stream);
 
-/* Latent attention, per token: cq [T, q_rank] = rms(dq) * wq; row = [rms(dkv[:rank]) * wc | rotary(dkv[rank:])]
+/* Latent attention, per token: cq [T, q_rank] = rms(dq) * wq (dq NULL: no query latent); row = [rms(dkv[:rank]) * wc | rotary(dkv[rank:])]
  * (rot columns, the first `dims` rotated) written to kc [T, rank + rot] (optional) and to the paged cache
- * [nb, bs, rank + rot] at `slots` (flat, or (block, offset) pairs; optional). */
+ * [nb, bs, rank + rot] at `slots` (flat, or (block, offset) pairs; optional). table as in b200_rotary_heads. */
 int b200_latent_kv_prep(void* cq, void* kc, void* cache, const int32_t* slots, int32_t slot_pairs,
                         int32_t block_size, const void* dq, int64_t dq_stride, const void* dkv,
                         int64_t dkv_stride, const float* wq, const float* wc, const int64_t* positions,
-                        int32_t tokens, int32_t q_rank, int32_t rank, int32_t rot, int32_t dims, double base,
+                        const float* table, int32_t tokens, int32_t q_rank, int32_t rank, int32_t rot, int32_t dims, double base,
                         int32_t interleaved, float eps, int32_t dtype, b200_stream_t stream);
 
 /* Softmax over a block of fp32 scores s [rows, nk] of `heads` query heads per token. ctx_lens == NULL: the rows
@@ -683,10 +687,12 @@ int b200_glu_clamped(void* out, const void* x, int32_t rows, int32_t inter, floa
 
 /* Router: s = sigmoid(logits) (fp32 [T, E]); choice = s + bias; experts form `groups` equal groups of
  * neighbours, a group scores the sum of its two largest choices and only the `keep` best groups stay in play;
- * the top_k choices are taken (ties to the lower index); weights = s / (sum s + 1e-20) * scale, fp32. */
+ * the top_k choices are taken (ties to the lower index); weights = s / (sum s + 1e-20) * scale
+ * (normalize) or s * scale as it is, fp32. */
 int b200_moe_route_grouped(int32_t* topk_ids, float* topk_weights, const float* router_logits,
                            int64_t logit_stride, const float* bias, int32_t tokens, int32_t num_experts,
-                           int32_t top_k, int32_t groups, int32_t keep, float scale, b200_stream_t stream);
+                           int32_t top_k, int32_t groups, int32_t keep, float scale, int32_t normalize,
+                           b200_stream_t stream);
 
 /* Router: s = softmax(logits) over all experts (fp32 [T, E]); experts form `groups` equal groups of neighbours, a
  * group scores its largest s and only the `keep` best groups stay in play; the top_k s are taken (ties to the lower
@@ -704,13 +710,14 @@ int b200_moe_route_topk(int32_t* topk_ids, float* topk_weights, const float* rou
  * silu(x Wg^T) * (x Wu^T), x rows gathered by sorted_pair / top_k, w [E, 2*n_out, K]. gate_up == 2 + act: out
  * [pairs, n_out] (dtype) = act(x Wu^T) without a gate, w [E, n_out, K], act as in b200_act_only. gate_up == 0: out
  * [pairs, n_out] fp32 = a W^T with a [pairs, K] in plan order, w [E, n_out, K]. gate_up == 1 with glu_limit > 0: the
- * clamped unit g sigmoid(glu_alpha g) (u + 1), g = min(x Wg^T, limit), u = clamp(x Wu^T, +-limit), in place of silu. */
+ * clamped unit g sigmoid(glu_alpha g) (u + 1), g = min(x Wg^T, limit), u = clamp(x Wu^T, +-limit), in place of silu.
+ * in_scale (gate_up == 1; fp32 [tokens * top_k] or NULL): a weight per pair on the expert's input row. */
 int b200_moe_gemm_generic(void* out, const void* a, int64_t a_stride, const void* w, const int32_t* offsets,
-                          const int32_t* sorted_pair, int32_t num_pairs, int32_t K, int32_t n_out,
+                          const int32_t* sorted_pair, const float* in_scale, int32_t num_pairs, int32_t K, int32_t n_out,
                           int32_t num_local, int32_t top_k, int32_t gate_up, float glu_alpha, float glu_limit,
                           int32_t dtype, b200_stream_t stream);
 
-/* out[t] = sum_j topk_weights[t, j] y[pos_of_pair[t, j]] (fp32 accumulation, pairs with pos < 0 skipped). */
+/* out[t] = sum_j topk_weights[t, j] (NULL: 1) y[pos_of_pair[t, j]] (fp32 accumulation, pairs with pos < 0 skipped). */
 int b200_moe_combine_weighted(void* out, const float* y, const float* topk_weights, const int32_t* pos_of_pair,
                               int32_t tokens, int32_t top_k, int32_t hidden, int32_t dtype,
                               b200_stream_t stream);
@@ -754,6 +761,19 @@ int b200_token_shift(void* out, int64_t mix_stride, const void* h, int64_t h_str
                      void* state, const int32_t* state_slots, const int32_t* cu_q, const int32_t* cu_k,
                      const int32_t* ctx_lens, int32_t num_seqs, int32_t max_q, int32_t width, int32_t dtype,
                      b200_stream_t stream);
+
+/* Gated residual with a depth average, per row t of [rows, hidden]: v = (x_in ? x_in : 0) + c * y * (gate ? sigmoid(gate) : 1)
+ * (y_index int64 [rows]: row t of y is y[clamp(y_index[t], 0, y_rows - 1)]; gate has gate_stride elements between rows);
+ * keep <- v when given; with avg (fp32 [n + 1]): v <- sum_(j < n) avg[j] * hist[j * hist_stride ...] + avg[n] * v; x_out <- v
+ * when given; with weight (fp32 [hidden]): h (dtype) = v / sqrt(mean v^2 + eps) * weight. x_in, x_out, keep, hist fp32;
+ * y, gate dtype. x_out may be x_in. */
+int b200_residual_gate_average(void* h, const float* x_in, float* x_out, const void* y, const int64_t* y_index,
+                               int64_t y_rows, const void* gate, int64_t gate_stride, float c, float* keep,
+                               const float* hist, int64_t hist_stride, int32_t n, const float* avg, const float* weight,
+                               float eps, int32_t rows, int32_t hidden, int32_t dtype, b200_stream_t stream);
+
+/* z (fp32, in place) <- cap * tanh(scale * z / cap); cap 0: scale * z. */
+int b200_logit_cap(float* z, int64_t total, float scale, float cap, b200_stream_t stream);
 
 /* out[t, h, :] = x[t, h, :] * sigmoid(gate[t * gate_stride + h]); x, out [rows, num_heads * vdim] contiguous. */
 int b200_head_gate(void* out, const void* x, const void* gate, int64_t gate_stride, int32_t rows, int32_t num_heads,

@@ -21,8 +21,8 @@
 //    heads) is the M dimension of mma.sync m16n8k16 (rows 8-15 are structurally zero), i.e.
 //    the whole group shares a single read of the KV bytes. fp32 online softmax in the exp2
 //    domain; running max/sum per thread, reduced with warp shuffles.
-//  * Optional sliding window with kept first tokens: the work list of a row holds only the tiles that have a visible key
-//    (tile_list), borders are masked element by element. Keys and values may have different head sizes (DK, DV).
+//  * Optional sliding window with kept first tokens, or chunks (a row sees its own chunk, a window of its own length): the
+//    work list of a row holds only the tiles that have a visible key (tile_list), borders are masked element by element. Keys and values may have different head sizes (DK, DV).
 //  Algorithmic bytes per launch: sum_b ctx_b * 2 * Hkv * D * 2 B (+ q, out: negligible).
 #include "decode_common.cuh"
 
@@ -64,7 +64,8 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK,
 
   // ---- tiles per item -> exclusive prefix sum in shared memory
   for (int i = threadIdx.x; i < items; i += blockDim.x) {
-    prefix[i + 1] = tile_list<TILE_TOKENS>(p.context_lens[i / p.hg_count], p.window, p.keep_first).count;
+    const int len = p.context_lens[i / p.hg_count];
+    prefix[i + 1] = tile_list<TILE_TOKENS>(len, p.row_window(len), p.keep_first).count;
   }
   if (threadIdx.x == 0) {
     prefix[0] = 0;
@@ -122,7 +123,7 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK,
         const int j = tt - prefix[it];
         const int b = it / p.hg_count, hg = it - b * p.hg_count;
         const int len = p.context_lens[b];
-        const int tok0 = tile_list<TILE_TOKENS>(len, p.window, p.keep_first).tile(j) * TILE_TOKENS;
+        const int tok0 = tile_list<TILE_TOKENS>(len, p.row_window(len), p.keep_first).tile(j) * TILE_TOKENS;
         nops = min(OPS, (len - tok0 + p.rows_box - 1) / p.rows_box);
         hg0 = hg * HKV_CTA;
 #pragma unroll
@@ -209,8 +210,9 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK,
     const int j1 = min(ntiles, j0 + (hi - t));
     const int b = it / p.hg_count, hg = it - b * p.hg_count;
     const int len = p.context_lens[b];
-    const TileList list = tile_list<TILE_TOKENS>(len, p.window, p.keep_first);
-    const int hidden_hi = p.window > 0 ? len - p.window : 0;   // keys [keep_first, hidden_hi) are hidden
+    const int window = p.row_window(len);
+    const TileList list = tile_list<TILE_TOKENS>(len, window, p.keep_first);
+    const int hidden_hi = window > 0 ? len - window : 0;       // keys [keep_first, hidden_hi) are hidden
     const int kv_head = hg * HKV_CTA + head_local;
 
     // ---- Q fragments for this (sequence, kv head): rows = query heads of the GQA group
@@ -542,7 +544,7 @@ extern "C" int b200_paged_decode_attn_capped(void* out, const void* q, const voi
                                              b200_stream_t stream_) {
   return b200_paged_decode_attn_windowed(out, q, k_cache, v_cache, block_tables, context_lens, batch, num_heads,
                                          num_kv_heads, head_dim, head_dim, q_stride, out_stride, num_blocks, block_size,
-                                         block_table_stride, scale, softcap, sink, 0, 0, workspace, workspace_bytes,
+                                         block_table_stride, scale, softcap, sink, 0, 0, 0, workspace, workspace_bytes,
                                          num_ctas, dtype, stream_);
 }
 
@@ -552,7 +554,7 @@ extern "C" int b200_paged_decode_attn_windowed(void* out, const void* q, const v
                                                int32_t value_dim, int64_t q_stride, int64_t out_stride,
                                                int32_t num_blocks, int32_t block_size, int32_t block_table_stride,
                                                float scale, float softcap, const float* sink, int32_t window,
-                                               int32_t keep_first, void* workspace, size_t workspace_bytes,
+                                               int32_t keep_first, int32_t chunk, void* workspace, size_t workspace_bytes,
                                                int32_t num_ctas, int32_t dtype, b200_stream_t stream_) {
   cudaStream_t stream = (cudaStream_t)stream_;
   B200_RETURN_IF(dtype != B200_DTYPE_BF16 && dtype != B200_DTYPE_F16, B200_ERR_BAD_DTYPE);
@@ -565,7 +567,7 @@ extern "C" int b200_paged_decode_attn_windowed(void* out, const void* q, const v
                      !workspace,
                  B200_ERR_NULL_POINTER);
   B200_RETURN_IF((head_dim != 64 && head_dim != 128) || (value_dim != 64 && value_dim != 128), B200_ERR_UNSUPPORTED);
-  B200_RETURN_IF(window < 0 || keep_first < 0, B200_ERR_BAD_SHAPE);
+  B200_RETURN_IF(window < 0 || keep_first < 0 || chunk < 0 || (window > 0 && chunk > 0), B200_ERR_BAD_SHAPE);
   const int G = num_heads / num_kv_heads;
   const int hkv_cta = hkv_cta_of(num_kv_heads);
   B200_RETURN_IF(G > 8 || hkv_cta == 0, B200_ERR_UNSUPPORTED);
@@ -615,7 +617,7 @@ extern "C" int b200_paged_decode_attn_windowed(void* out, const void* q, const v
   p.scale_log2 = scale * 1.4426950408889634f;
   if (softcap > 0.f) p.cap = softcap, p.cap_pre = scale / softcap;
   p.sink = sink;
-  p.window = window, p.keep_first = window > 0 ? keep_first : 0;
+  p.window = window, p.keep_first = window > 0 ? keep_first : 0, p.chunk = chunk;
 
   const int k_chunks = num_kv_heads * head_dim / 64, v_chunks = num_kv_heads * value_dim / 64;
   CUtensorMap mk, mv;

@@ -30,6 +30,12 @@ struct DecodeParams {
   float cap = 0.f, cap_pre = 0.f;
   const float* sink = nullptr;
   int window = 0, keep_first = 0;   // window > 0: only the last `window` keys and those below keep_first are visible
+  int chunk = 0;                    // chunk > 0: only the keys of the row's own chunk (counted from position 0) are visible
+
+  // how many of a row's `len` keys count back from its end as visible (0: all of them)
+  __device__ __forceinline__ int row_window(int len) const {
+    return chunk > 0 && len > 0 ? len - (len - 1) / chunk * chunk : window;
+  }
 };
 
 // The key tiles (of TT tokens) that a row of `len` keys visits: tile j of the row's list is tile j of its keys for j < kept,

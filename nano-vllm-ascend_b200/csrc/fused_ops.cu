@@ -339,19 +339,27 @@ sample_kernel(int64_t* __restrict__ out, const T* __restrict__ logits,
     }
     if (v > best || (v == best && i < best_i)) best = v, best_i = i;
   };
-  const bool vec_ok = (stride % 8 == 0) && ((reinterpret_cast<uintptr_t>(logits) & 15) == 0);
-  const int nvec = vec_ok ? vocab / 8 : 0;
+  constexpr int V = 16 / sizeof(T);                          // elements per 16-byte load
+  const bool vec_ok = (stride % V == 0) && ((reinterpret_cast<uintptr_t>(logits) & 15) == 0);
+  const int nvec = vec_ok ? vocab / V : 0;
   for (int vi = threadIdx.x; vi < nvec; vi += blockDim.x) {
     const uint4 q = ld_nc_v4(reinterpret_cast<const uint4*>(lrow) + vi);
     const uint32_t w[4] = {q.x, q.y, q.z, q.w};
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
-      const float2 f = unpack2<T>(w[j]);
-      consider(f.x, vi * 8 + 2 * j);
-      consider(f.y, vi * 8 + 2 * j + 1);
+      if constexpr (V == 4) {
+        consider(__uint_as_float(w[j]), vi * 4 + j);
+      } else {
+        const float2 f = unpack2<T>(w[j]);
+        consider(f.x, vi * 8 + 2 * j);
+        consider(f.y, vi * 8 + 2 * j + 1);
+      }
     }
   }
-  for (int i = nvec * 8 + threadIdx.x; i < vocab; i += blockDim.x) consider(to_f32<T>(lrow[i]), i);
+  for (int i = nvec * V + threadIdx.x; i < vocab; i += blockDim.x) {
+    if constexpr (V == 4) consider(lrow[i], i);
+    else consider(to_f32<T>(lrow[i]), i);
+  }
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) {
     const float ov = __shfl_xor_sync(0xffffffffu, best, o);
@@ -526,7 +534,7 @@ extern "C" int b200_sample(int64_t* out_tokens, const void* logits, const float*
                            int32_t rows, int32_t vocab, int64_t logits_stride, uint64_t seed,
                            uint64_t step, const int64_t* step_offset, int32_t dtype,
                            b200_stream_t stream) {
-  B200_RETURN_IF(dtype != B200_DTYPE_BF16 && dtype != B200_DTYPE_F16, B200_ERR_BAD_DTYPE);
+  B200_RETURN_IF(dtype != B200_DTYPE_BF16 && dtype != B200_DTYPE_F16 && dtype != B200_DTYPE_F32, B200_ERR_BAD_DTYPE);
   B200_RETURN_IF(rows < 0 || vocab <= 0 || logits_stride < vocab, B200_ERR_BAD_SHAPE);
   if (rows == 0) return B200_OK;
   B200_RETURN_IF(!out_tokens || !logits, B200_ERR_NULL_POINTER);
@@ -534,6 +542,9 @@ extern "C" int b200_sample(int64_t* out_tokens, const void* logits, const float*
     launch_pdl(sample_kernel<__nv_bfloat16>, dim3(rows), dim3(1024), 0, (cudaStream_t)stream,
                out_tokens, (const __nv_bfloat16*)logits, temperatures, vocab, logits_stride, seed, step,
                step_offset);
+  else if (dtype == B200_DTYPE_F32)
+    launch_pdl(sample_kernel<float>, dim3(rows), dim3(1024), 0, (cudaStream_t)stream, out_tokens,
+               (const float*)logits, temperatures, vocab, logits_stride, seed, step, step_offset);
   else
     launch_pdl(sample_kernel<__half>, dim3(rows), dim3(1024), 0, (cudaStream_t)stream, out_tokens,
                (const __half*)logits, temperatures, vocab, logits_stride, seed, step, step_offset);

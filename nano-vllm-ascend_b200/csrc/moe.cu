@@ -176,8 +176,9 @@ struct MoeGemmParams {
   int64_t a_stride;            // elements between rows of a
   int K, n_out, top_k;
   int act;                     // up alone (mode 2): 0 silu, 1 relu, 2 gelu (tanh form), 3 squared relu
-  float glu_alpha, glu_limit;  // gate_up with glu_limit > 0: the clamped unit g sigmoid(alpha g) (u + 1), g = min(gate,
+  float glu_alpha = 0.f, glu_limit = 0.f;  // gate_up with glu_limit > 0: the clamped unit g sigmoid(alpha g) (u + 1), g = min(gate,
                                // limit), u = clamp(up, +-limit), in place of silu(gate) * up
+  const float* in_scale = nullptr;   // gate_up: weight of every pair on the expert's INPUT (fp32 [tokens * top_k])
 };
 
 constexpr int kMoeStages = 4;
@@ -303,6 +304,11 @@ __device__ __forceinline__ void moe_gemm_pass(const MoeGemmParams& p, uint8_t* s
       if (row >= cnt) continue;
       const int64_t pos = row_begin + row;
       if (kGateUp) {
+        if (p.in_scale != nullptr) {     // the products are linear in the row: the weight multiplies them in fp32
+          const float in = p.in_scale[p.sorted_pair[pos]];
+#pragma unroll
+          for (int nf = 0; nf < 2; ++nf) acc[mf][nf][2 * r] *= in, acc[mf][nf][2 * r + 1] *= in;
+        }
         // gate_up in the model dtype (F.linear), silu in fp32 -> dtype, dtype multiply with `up`
         const float g0 = to_f32<T>(from_f32<T>(acc[mf][0][2 * r])), g1 = to_f32<T>(from_f32<T>(acc[mf][0][2 * r + 1]));
         const float u0 = to_f32<T>(from_f32<T>(acc[mf][1][2 * r])), u1 = to_f32<T>(from_f32<T>(acc[mf][1][2 * r + 1]));
@@ -328,7 +334,8 @@ __device__ __forceinline__ void moe_gemm_pass(const MoeGemmParams& p, uint8_t* s
         }
       } else {
         // expert output in the model dtype, then a dtype multiply with the routing weight
-        const float sc = to_f32<T>(reinterpret_cast<const T*>(p.pair_scale)[p.sorted_pair[pos]]);
+        const float sc =
+            p.pair_scale != nullptr ? to_f32<T>(reinterpret_cast<const T*>(p.pair_scale)[p.sorted_pair[pos]]) : 1.f;
 #pragma unroll
         for (int nf = 0; nf < 2; ++nf) {
           const float y0 = to_f32<T>(from_f32<T>(acc[mf][nf][2 * r])), y1 = to_f32<T>(from_f32<T>(acc[mf][nf][2 * r + 1]));
@@ -489,13 +496,14 @@ static int moe_gemm_check(const void* a, const void* w, void* out, const int32_t
 }
 
 extern "C" int b200_moe_gemm_gate_up(void* h, const void* x, const void* w13, const int32_t* offsets,
-                                     const int32_t* sorted_pair, int32_t hidden, int32_t inter,
-                                     int32_t num_local, int32_t top_k, int64_t x_stride, int32_t dtype,
-                                     b200_stream_t stream) {
+                                     const int32_t* sorted_pair, const float* in_scale, int32_t hidden,
+                                     int32_t inter, int32_t num_local, int32_t top_k, int64_t x_stride,
+                                     int32_t dtype, b200_stream_t stream) {
   const int rc = moe_gemm_check(x, w13, h, offsets, sorted_pair, hidden, inter, 64, num_local, top_k,
                                 x_stride, dtype);
   if (rc != B200_OK) return rc;
   MoeGemmParams p{x, w13, h, offsets, sorted_pair, nullptr, x_stride, hidden, inter, top_k, 0};
+  p.in_scale = in_scale;
   return dtype == B200_DTYPE_BF16 ? moe_gemm_launch<__nv_bfloat16>(1, p, num_local, (cudaStream_t)stream)
                                   : moe_gemm_launch<__half>(1, p, num_local, (cudaStream_t)stream);
 }
@@ -533,7 +541,6 @@ extern "C" int b200_moe_gemm_down(void* y, const void* h, const void* w2, const 
   const int rc = moe_gemm_check(h, w2, y, offsets, sorted_pair, inter, hidden, 128, num_local, top_k,
                                 inter, dtype);
   if (rc != B200_OK) return rc;
-  B200_RETURN_IF(!topk_weights, B200_ERR_NULL_POINTER);
   MoeGemmParams p{h, w2, y, offsets, sorted_pair, topk_weights, inter, inter, hidden, top_k, 0};
   return dtype == B200_DTYPE_BF16 ? moe_gemm_launch<__nv_bfloat16>(0, p, num_local, (cudaStream_t)stream)
                                   : moe_gemm_launch<__half>(0, p, num_local, (cudaStream_t)stream);

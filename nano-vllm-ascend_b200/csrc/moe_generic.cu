@@ -5,7 +5,7 @@
 //   moe_route_grouped    s = sigmoid(z); choice = s + bias; experts form `groups` equal groups of neighbours, a
 //                        group scores the sum of its two largest choices, only the `keep` best groups stay in
 //                        play (the others count as -inf); the top-k choices are taken and weighted by
-//                        s / (sum s + 1e-20) * scale. Ties go to the lower index. fp32 throughout.
+//                        s / (sum s + 1e-20) * scale, or s * scale as it is. Ties go to the lower index. fp32 throughout.
 //   moe_route_grouped_softmax  s = softmax(z) over all experts; a group scores its largest s; the `keep` best groups
 //                        stay in play; the top-k s are taken and weighted by s / (sum s + 1e-20) * scale.
 //   moe_route_topk       the k largest of z + bias; weights = softmax over the chosen logits only. fp32 throughout.
@@ -13,8 +13,9 @@
 //                        g sigmoid(alpha g) (u + 1), g = min(gate, limit), u = clamp(up, +-limit))
 //                        H[pos] = act(X[token(pos)] Wu[e]^T)                               (up alone, no gate)
 //                        Y[pos] = H[pos] W2[e]^T, fp32                                     (down)
-//                        over the dispatch plan of moe_align (pairs sorted by expert); 32 x 64 tiles, fp32 FMA.
-//   moe_combine_weighted out[t] = sum_j w[t][j] Y[pos(t, j)], accumulated in fp32, one rounding.
+//                        over the dispatch plan of moe_align (pairs sorted by expert); 32 x 64 tiles, fp32 FMA. A weight
+//                        per pair on the expert's INPUT multiplies the gate and up products (they are linear in it).
+//   moe_combine_weighted out[t] = sum_j w[t][j] Y[pos(t, j)] (w may be absent: 1), accumulated in fp32, one rounding.
 #include "seq_common.cuh"
 
 namespace b200 {
@@ -27,7 +28,7 @@ constexpr int kRouteMaxGroups = 64;
 __global__ void __launch_bounds__(128)
 moe_route_grouped_kernel(int32_t* __restrict__ ids, float* __restrict__ weights, const float* __restrict__ logits,
                          int64_t logit_stride, const float* __restrict__ bias, int tokens, int E, int top_k,
-                         int groups, int keep, float scale, int kind) {
+                         int groups, int keep, float scale, int kind, int normalize) {
   extern __shared__ float smem[];                    // per warp: choice [E], s [E]
   pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -131,7 +132,7 @@ moe_route_grouped_kernel(int32_t* __restrict__ ids, float* __restrict__ weights,
   }
   if (lane < top_k) {
     ids[t * top_k + lane] = my_id;
-    weights[t * top_k + lane] = kind == 1 ? mine / wsum : mine / (wsum + 1e-20f) * scale;
+    weights[t * top_k + lane] = kind == 1 ? mine / wsum : (normalize ? mine / (wsum + 1e-20f) : mine) * scale;
   }
 }
 
@@ -141,6 +142,7 @@ struct MoeGenericParams {
   const void* w;              // gate_up: [E, 2 * n_out, K]; down: [E, n_out, K]
   void* out;                  // gate_up: [pairs, n_out] element type; down: [pairs, n_out] fp32
   const int32_t *offsets, *sorted_pair;
+  const float* in_scale;      // gate_up: weight of every pair on the expert's INPUT ([tokens * top_k] fp32), or nullptr
   int64_t a_stride;
   int K, n_out, top_k;
   int act;                    // up alone: 0 silu, 1 relu, 2 gelu (tanh form), 3 squared relu
@@ -227,15 +229,19 @@ moe_gemm_generic_kernel(const MoeGenericParams p) {
         if (c >= p.n_out) continue;
         const int64_t o = (int64_t)(row_begin + r) * p.n_out + c;
         if (kGateUp) {
-          float r;
+          if (p.in_scale != nullptr) {                // the products are linear in the row: weigh them in fp32
+            const float in = p.in_scale[p.sorted_pair[row_begin + r]];
+            acc[i][j] *= in, acc2[i][j] *= in;
+          }
+          float u_out;
           if (p.glu_limit > 0.f) {
             const float g = fminf(acc[i][j], p.glu_limit);
             const float u = fminf(fmaxf(acc2[i][j], -p.glu_limit), p.glu_limit);
-            r = g * sigmoid_f(p.glu_alpha * g) * (u + 1.0f);
+            u_out = g * sigmoid_f(p.glu_alpha * g) * (u + 1.0f);
           } else {
-            r = silu_f(acc[i][j]) * acc2[i][j];
+            u_out = silu_f(acc[i][j]) * acc2[i][j];
           }
-          reinterpret_cast<T*>(p.out)[o] = from_f32<T>(r);
+          reinterpret_cast<T*>(p.out)[o] = from_f32<T>(u_out);
         }
         else if (kMode == 2) reinterpret_cast<T*>(p.out)[o] = from_f32<T>(plain_act(acc[i][j], p.act));
         else reinterpret_cast<float*>(p.out)[o] = acc[i][j];
@@ -254,7 +260,7 @@ moe_combine_weighted_kernel(T* __restrict__ out, const float* __restrict__ y, co
     float acc = 0.f;
     for (int j = 0; j < k; ++j) {
       const int ps = pos_of_pair[t * k + j];
-      if (ps >= 0) acc += weights[t * k + j] * y[(int64_t)ps * hidden + i];
+      if (ps >= 0) acc += (weights != nullptr ? weights[t * k + j] : 1.0f) * y[(int64_t)ps * hidden + i];
     }
     out[t * hidden + i] = from_f32<T>(acc);
   }
@@ -267,7 +273,7 @@ using namespace b200;
 extern "C" int b200_moe_route_grouped(int32_t* topk_ids, float* topk_weights, const float* router_logits,
                                       int64_t logit_stride, const float* bias, int32_t tokens,
                                       int32_t num_experts, int32_t top_k, int32_t groups, int32_t keep,
-                                      float scale, b200_stream_t stream) {
+                                      float scale, int32_t normalize, b200_stream_t stream) {
   B200_RETURN_IF(tokens < 0 || num_experts <= 0 || top_k <= 0 || top_k > num_experts || groups <= 0 || keep <= 0 ||
                      keep > groups || num_experts % groups != 0 || (num_experts / groups) * keep < top_k,
                  B200_ERR_BAD_SHAPE);
@@ -277,7 +283,7 @@ extern "C" int b200_moe_route_grouped(int32_t* topk_ids, float* topk_weights, co
   B200_RETURN_IF(!topk_ids || !topk_weights || !router_logits, B200_ERR_NULL_POINTER);
   const size_t smem = (size_t)4 * 2 * num_experts * sizeof(float);
   launch_pdl(moe_route_grouped_kernel, dim3((tokens + 3) / 4), dim3(128), smem, (cudaStream_t)stream, topk_ids,
-             topk_weights, router_logits, logit_stride, bias, tokens, num_experts, top_k, groups, keep, scale, 0);
+             topk_weights, router_logits, logit_stride, bias, tokens, num_experts, top_k, groups, keep, scale, 0, normalize);
   return finish_launch();
 }
 
@@ -295,7 +301,7 @@ extern "C" int b200_moe_route_grouped_softmax(int32_t* topk_ids, float* topk_wei
   const size_t smem = (size_t)4 * 2 * num_experts * sizeof(float);
   launch_pdl(moe_route_grouped_kernel, dim3((tokens + 3) / 4), dim3(128), smem, (cudaStream_t)stream, topk_ids,
              topk_weights, router_logits, logit_stride, (const float*)nullptr, tokens, num_experts, top_k, groups, keep,
-             scale, 2);
+             scale, 2, 1);
   return finish_launch();
 }
 
@@ -308,20 +314,20 @@ extern "C" int b200_moe_route_topk(int32_t* topk_ids, float* topk_weights, const
   B200_RETURN_IF(!topk_ids || !topk_weights || !router_logits, B200_ERR_NULL_POINTER);
   const size_t smem = (size_t)4 * 2 * num_experts * sizeof(float);
   launch_pdl(moe_route_grouped_kernel, dim3((tokens + 3) / 4), dim3(128), smem, (cudaStream_t)stream, topk_ids,
-             topk_weights, router_logits, logit_stride, bias, tokens, num_experts, top_k, 1, 1, 1.0f, 1);
+             topk_weights, router_logits, logit_stride, bias, tokens, num_experts, top_k, 1, 1, 1.0f, 1, 1);
   return finish_launch();
 }
 
 extern "C" int b200_moe_gemm_generic(void* out, const void* a, int64_t a_stride, const void* w,
-                                     const int32_t* offsets, const int32_t* sorted_pair, int32_t num_pairs,
-                                     int32_t K, int32_t n_out, int32_t num_local, int32_t top_k, int32_t gate_up,
+                                     const int32_t* offsets, const int32_t* sorted_pair, const float* in_scale,
+                                     int32_t num_pairs, int32_t K, int32_t n_out, int32_t num_local, int32_t top_k, int32_t gate_up,
                                      float glu_alpha, float glu_limit, int32_t dtype, b200_stream_t stream) {
   B200_RETURN_IF(num_pairs < 0 || K <= 0 || n_out <= 0 || num_local <= 0 || top_k <= 0, B200_ERR_BAD_SHAPE);
   B200_RETURN_IF(num_local > 65535, B200_ERR_UNSUPPORTED);
   if (num_pairs == 0) return B200_OK;
   B200_RETURN_IF(!out || !a || !w || !offsets || !sorted_pair, B200_ERR_NULL_POINTER);
-  B200_RETURN_IF(gate_up < 0 || gate_up > 5, B200_ERR_BAD_SHAPE);
-  MoeGenericParams p{a, w, out, offsets, sorted_pair, a_stride, K, n_out, top_k, gate_up >= 2 ? gate_up - 2 : 0,
+  B200_RETURN_IF(gate_up < 0 || gate_up > 5 || (in_scale && gate_up != 1), B200_ERR_BAD_SHAPE);
+  MoeGenericParams p{a, w, out, offsets, sorted_pair, in_scale, a_stride, K, n_out, top_k, gate_up >= 2 ? gate_up - 2 : 0,
                      glu_alpha, glu_limit};
   int my = (num_pairs + kGM - 1) / kGM;
   if (my > 32) my = 32;
@@ -339,7 +345,7 @@ extern "C" int b200_moe_combine_weighted(void* out, const float* y, const float*
                                          int32_t hidden, int32_t dtype, b200_stream_t stream) {
   B200_RETURN_IF(tokens < 0 || top_k <= 0 || hidden <= 0, B200_ERR_BAD_SHAPE);
   if (tokens == 0) return B200_OK;
-  B200_RETURN_IF(!out || !y || !topk_weights || !pos_of_pair, B200_ERR_NULL_POINTER);
+  B200_RETURN_IF(!out || !y || !pos_of_pair, B200_ERR_NULL_POINTER);
   B200_DISPATCH_3(dtype, T, launch_pdl(moe_combine_weighted_kernel<T>, dim3(tokens), dim3(256), 0, (cudaStream_t)stream,
                                        (T*)out, y, topk_weights, pos_of_pair, top_k, hidden));
   return finish_launch();

@@ -31,6 +31,7 @@ struct MoeUmmaParams {
   void* out;                   // gate_up: H [pairs, n_out]; down: Y [pairs, n_out]
   int num_local, K, n_out;
   int out_f32;                 // plain epilogue only: the fp32 accumulators are stored as they are (out is float*)
+  const float* in_scale = nullptr;   // gate_up: weight of every pair on the expert's INPUT (fp32), or nullptr
 };
 
 // Ring depth: 3 stages (97 KB, two CTAs per SM) for tensor-bound grouped GEMMs, where the second CTA's
@@ -143,6 +144,8 @@ moe_umma_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_const
     mbar_wait(acc_full, 0);
     umma::fence_after_sync();
     if (kGateUp) {
+      // the products are linear in the expert's input: its weight multiplies them in fp32
+      const float in = p.in_scale != nullptr && valid ? p.in_scale[p.sorted_pair[pos]] : 1.f;
 #pragma unroll
       for (int c0 = 0; c0 < 64; c0 += 32) {
         uint32_t g[32], u[32];
@@ -156,10 +159,10 @@ moe_umma_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_const
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
               // gate_up in the model dtype, silu in fp32 -> dtype, dtype multiply (activation.py:11-13)
-              const float g0 = to_f32<T>(from_f32<T>(__uint_as_float(g[c + 2 * j])));
-              const float g1 = to_f32<T>(from_f32<T>(__uint_as_float(g[c + 2 * j + 1])));
-              const float u0 = to_f32<T>(from_f32<T>(__uint_as_float(u[c + 2 * j])));
-              const float u1 = to_f32<T>(from_f32<T>(__uint_as_float(u[c + 2 * j + 1])));
+              const float g0 = to_f32<T>(from_f32<T>(in * __uint_as_float(g[c + 2 * j])));
+              const float g1 = to_f32<T>(from_f32<T>(in * __uint_as_float(g[c + 2 * j + 1])));
+              const float u0 = to_f32<T>(from_f32<T>(in * __uint_as_float(u[c + 2 * j])));
+              const float u1 = to_f32<T>(from_f32<T>(in * __uint_as_float(u[c + 2 * j + 1])));
               const float s0 = to_f32<T>(from_f32<T>(__fdividef(g0, 1.0f + __expf(-g0))));
               const float s1 = to_f32<T>(from_f32<T>(__fdividef(g1, 1.0f + __expf(-g1))));
               w[j] = pack2<T>(__fmul_rn(s0, u0), __fmul_rn(s1, u1));
@@ -284,7 +287,7 @@ extern "C" int b200_moe_gather_rows(void* xs, const void* x, const int32_t* offs
 static int moe_umma_common(bool gate_up, void* out, const void* a, const void* w, const int32_t* offsets,
                            const int32_t* sorted_pair, const void* pair_scale, int32_t pairs, int32_t K,
                            int32_t n_out, int32_t num_local, int32_t dtype, b200_stream_t stream,
-                           int out_f32 = 0) {
+                           int out_f32 = 0, const float* in_scale = nullptr) {
   B200_RETURN_IF(dtype != B200_DTYPE_BF16 && dtype != B200_DTYPE_F16, B200_ERR_BAD_DTYPE);
   B200_RETURN_IF(pairs < 0 || K <= 0 || n_out <= 0 || num_local <= 0, B200_ERR_BAD_SHAPE);
   B200_RETURN_IF(K % 64 != 0 || n_out % (gate_up ? 64 : 128) != 0 || num_local > 256, B200_ERR_UNSUPPORTED);
@@ -298,16 +301,18 @@ static int moe_umma_common(bool gate_up, void* out, const void* a, const void* w
   const int64_t w_rows = (int64_t)num_local * (gate_up ? 2 : 1) * n_out;
   rc = get_panel_map(w, w_rows, (int64_t)K * 2, K / 64, 64, 1, dtype, &mw);
   if (rc != B200_OK) return rc;
-  MoeUmmaParams p{offsets, sorted_pair, pair_scale, out, num_local, K, n_out, out_f32};
+  MoeUmmaParams p{offsets, sorted_pair, pair_scale, out, num_local, K, n_out, out_f32, in_scale};
   return dtype == B200_DTYPE_BF16 ? moe_umma_launch<__nv_bfloat16>(gate_up, ma, mw, p, pairs, (cudaStream_t)stream)
                                   : moe_umma_launch<__half>(gate_up, ma, mw, p, pairs, (cudaStream_t)stream);
 }
 
 extern "C" int b200_moe_gemm_gate_up_umma(void* h, const void* xs, const void* w13, const int32_t* offsets,
-                                          int32_t pairs, int32_t hidden, int32_t inter, int32_t num_local,
-                                          int32_t dtype, b200_stream_t stream) {
-  return moe_umma_common(true, h, xs, w13, offsets, nullptr, nullptr, pairs, hidden, inter, num_local, dtype,
-                         stream);
+                                          const int32_t* sorted_pair, const float* in_scale, int32_t pairs,
+                                          int32_t hidden, int32_t inter, int32_t num_local, int32_t dtype,
+                                          b200_stream_t stream) {
+  B200_RETURN_IF(in_scale && !sorted_pair, B200_ERR_NULL_POINTER);
+  return moe_umma_common(true, h, xs, w13, offsets, sorted_pair, nullptr, pairs, hidden, inter, num_local, dtype,
+                         stream, 0, in_scale);
 }
 
 extern "C" int b200_moe_gemm_down_umma(void* y, const void* h, const void* w2, const int32_t* offsets,

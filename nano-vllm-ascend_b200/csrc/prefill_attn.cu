@@ -249,7 +249,7 @@ int prefill_umma_launch(void* out, const void* q, const void* k, const void* v, 
                         int bt_stride, int num_blocks, int block_size, float scale, int dtype,
                         void* workspace, int64_t workspace_bytes, int max_seqlen_k,
                         cudaStream_t stream, float softcap, const float* sink, int window,
-                        int keep_first);       // prefill_umma.cu
+                        int keep_first, int chunk);       // prefill_umma.cu
 void prefill_force_query_tiles(int qt);        // prefill_umma.cu
 // B200_PREFILL_KERNEL=mma_sync forces the kernel in this file (A/B checks); default = prefill_umma.cu.
 static int prefill_kernel_choice() {
@@ -306,7 +306,7 @@ extern "C" int b200_prefill_varlen_attn_capped(void* out, const void* q, const v
   return b200_prefill_varlen_attn_windowed(out, q, k, v, cu_seqlens_q, cu_seqlens_k, num_seqs, total_q, total_k,
                                            max_seqlen_q, max_seqlen_k, num_heads, num_kv_heads, head_dim, head_dim,
                                            q_stride, k_stride, v_stride, out_stride, block_tables, block_table_stride,
-                                           num_blocks, block_size, scale, softcap, sink, 0, 0, dtype, workspace,
+                                           num_blocks, block_size, scale, softcap, sink, 0, 0, 0, dtype, workspace,
                                            workspace_bytes, stream);
 }
 
@@ -319,7 +319,7 @@ extern "C" int b200_prefill_varlen_attn_windowed(void* out, const void* q, const
                                                  int64_t out_stride, const int32_t* block_tables,
                                                  int32_t block_table_stride, int32_t num_blocks, int32_t block_size,
                                                  float scale, float softcap, const float* sink, int32_t window,
-                                                 int32_t keep_first, int32_t dtype, void* workspace,
+                                                 int32_t keep_first, int32_t chunk, int32_t dtype, void* workspace,
                                                  int64_t workspace_bytes, b200_stream_t stream) {
   B200_RETURN_IF(dtype != B200_DTYPE_BF16 && dtype != B200_DTYPE_F16, B200_ERR_BAD_DTYPE);
   B200_RETURN_IF(num_seqs < 0 || max_seqlen_q < 0 || max_seqlen_k < 0 || num_heads <= 0 ||
@@ -327,7 +327,7 @@ extern "C" int b200_prefill_varlen_attn_windowed(void* out, const void* q, const
                  B200_ERR_BAD_SHAPE);
   B200_RETURN_IF(num_heads % num_kv_heads != 0, B200_ERR_BAD_SHAPE);
   B200_RETURN_IF((head_dim != 64 && head_dim != 128) || (value_dim != 64 && value_dim != 128), B200_ERR_UNSUPPORTED);
-  B200_RETURN_IF(window < 0 || keep_first < 0, B200_ERR_BAD_SHAPE);
+  B200_RETURN_IF(window < 0 || keep_first < 0 || chunk < 0 || (window > 0 && chunk > 0), B200_ERR_BAD_SHAPE);
   if (num_seqs == 0 || max_seqlen_q == 0) return B200_OK;
   B200_RETURN_IF(!out || !q || !k || !v || !cu_seqlens_q || !cu_seqlens_k, B200_ERR_NULL_POINTER);
   B200_RETURN_IF(num_seqs > 65535 || num_heads > 65535, B200_ERR_UNSUPPORTED);
@@ -350,11 +350,11 @@ extern "C" int b200_prefill_varlen_attn_windowed(void* out, const void* q, const
     const int rc = prefill_umma_launch(out, q, k, v, cu_seqlens_q, cu_seqlens_k, num_seqs, total_q,
         total_k, max_seqlen_q, num_heads, num_kv_heads, head_dim, value_dim, q_stride, k_stride,
         v_stride, out_stride, block_tables, block_table_stride, num_blocks, block_size, scale, dtype,
-        workspace, workspace_bytes, max_seqlen_k, s, softcap, sink, window, keep_first);
+        workspace, workspace_bytes, max_seqlen_k, s, softcap, sink, window, keep_first, chunk);
     if (rc != B200_ERR_UNSUPPORTED) return rc;
   }
-  // the mma.sync variant below knows neither a score cap nor a sink, no window and one head size
-  B200_RETURN_IF(softcap > 0.f || sink != nullptr || window > 0 || value_dim != head_dim, B200_ERR_UNSUPPORTED);
+  // the mma.sync variant below knows neither a score cap nor a sink, no window or chunk and one head size
+  B200_RETURN_IF(softcap > 0.f || sink != nullptr || window > 0 || chunk > 0 || value_dim != head_dim, B200_ERR_UNSUPPORTED);
   PrefillParams p;
   p.q = q, p.k = k, p.v = v, p.out = out;
   p.cu_q = cu_seqlens_q, p.cu_k = cu_seqlens_k;

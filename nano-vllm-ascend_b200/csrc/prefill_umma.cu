@@ -34,7 +34,8 @@
 //
 // Sliding window with kept first tokens (window > 0): position i sees j <= i with i - j < window or j < keep_first. A CTA
 // visits the tiles of the kept keys, then those from its first row's window on; the tiles between are skipped by
-// index (p.keep_tiles, `skip`), the borders are masked element by element.
+// index (`kept`, `skip`), the borders are masked element by element. Chunks (chunk > 0: position i sees j <= i of its own
+// chunk) run the same way, with the chunk's start in place of the window's.
 // Keys and values may have different head sizes (DK, DV in {64, 128}); D below stands for the one that applies.
 //
 // Split-KV (few, long rows: the prefix-cache-hit form q_len << k_len): when the grid
@@ -64,6 +65,11 @@ struct PrefillUmmaParams {
   float cap = 0.f, cap_pre = 0.f;
   const float* sink = nullptr;
   int window = 0, keep_first = 0;   // window 0: every earlier key
+  int chunk = 0;                    // chunk > 0: only keys of the row's own chunk (counted from position 0)
+
+  __device__ __forceinline__ bool limited() const { return window > 0 || chunk > 0; }
+  // first key that position `pos` sees besides the kept ones (window or chunk; may be negative)
+  __device__ __forceinline__ int seen_from(int pos) const { return window > 0 ? pos - window + 1 : pos / chunk * chunk; }
 };
 
 constexpr int kUBM = 128, kUBN = 128;
@@ -118,7 +124,7 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   int n_tiles[2] = {0, 0};
   // tiles [0, kept) hold the kept first keys; the next `skip` tiles end before the window of this CTA's first row
   const int kept = p.window > 0 ? (min(p.keep_first, Lk) + kUBN - 1) / kUBN : 0;
-  const int skip = p.window > 0 ? max(0, max(0, m0 + off - p.window + 1) / kUBN - kept) : 0;
+  const int skip = p.limited() ? max(0, max(0, p.seen_from(m0 + off)) / kUBN - kept) : 0;
 #pragma unroll
   for (int t = 0; t < QT; ++t) {
     const int r0 = m0 + t * kUBM;
@@ -319,8 +325,8 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         for (int c = 0; c < 128; ++c)
           if (c > limit) sr[c >> 5][c & 31] = 0xff800000u;   // -inf
       }
-      if (p.window > 0 && n0 + kUBN > p.keep_first && n0 <= warp_row0 + 31 + off - p.window) {
-        const int low = qrow + off - p.window - n0, keep = p.keep_first - n0;   // hidden: keep <= c <= low
+      if (p.limited() && n0 + kUBN > p.keep_first && n0 < p.seen_from(warp_row0 + 31 + off)) {
+        const int low = p.seen_from(qrow + off) - 1 - n0, keep = p.keep_first - n0;   // hidden: keep <= c <= low
 #pragma unroll
         for (int c = 0; c < 128; ++c)
           if (c <= low && c >= keep) sr[c >> 5][c & 31] = 0xff800000u;
@@ -527,7 +533,7 @@ int prefill_umma_launch(void* out, const void* q, const void* k, const void* v,
                          int64_t k_stride, int64_t v_stride, int64_t out_stride,
                         const int32_t* block_tables, int bt_stride, int num_blocks, int block_size,
                         float scale, int dtype, void* workspace, int64_t workspace_bytes, int max_seqlen_k,
-                        cudaStream_t stream, float softcap, const float* sink, int window, int keep_first) {
+                        cudaStream_t stream, float softcap, const float* sink, int window, int keep_first, int chunk) {
   if (q_stride % 8 != 0 || out_stride % 8 != 0 || !aligned16(out)) return B200_ERR_UNSUPPORTED;
   if (total_q <= 0) return B200_ERR_UNSUPPORTED;
   const int CHK = DK / 64, CHV = DV / 64;
@@ -541,10 +547,11 @@ int prefill_umma_launch(void* out, const void* q, const void* k, const void* v,
   p.scale_log2 = scale * 1.4426950408889634f;
   if (softcap > 0.f) p.cap = softcap, p.cap_pre = scale / softcap;
   p.sink = sink;
-  p.window = window, p.keep_first = window > 0 ? keep_first : 0;
+  p.window = window, p.keep_first = window > 0 ? keep_first : 0, p.chunk = chunk;
+  const int span = window > 0 ? window : chunk;
   // keys that a 128-row query tile can see at most: what the choice of layout and of key splits is made on
-  if (window > 0 && max_seqlen_k > window + p.keep_first + 3 * kUBM) max_seqlen_k = window + p.keep_first + 3 * kUBM;
-  const int qt = prefill_query_tiles(num_seqs, H, max_seqlen_q, DV, window > 0 ? max_seqlen_k : max_seqlen_q);
+  if (span > 0 && max_seqlen_k > span + p.keep_first + 3 * kUBM) max_seqlen_k = span + p.keep_first + 3 * kUBM;
+  const int qt = prefill_query_tiles(num_seqs, H, max_seqlen_q, DV, span > 0 ? max_seqlen_k : max_seqlen_q);
   p.kv_splits = (workspace != nullptr && (reinterpret_cast<uintptr_t>(workspace) & 15) == 0)
                     ? prefill_kv_splits(num_seqs, H, max_seqlen_q, max_seqlen_k, total_q, DV, workspace_bytes, qt)
                     : 1;

@@ -3,8 +3,9 @@
 //   attn_generic       causal softmax attention for ANY head sizes (key size != value size, sizes that are
 //                      not 64 or 128), any element type including fp32, packed or paged keys, and any mix of
 //                      prompt portions and single tokens in one launch. fp32 scores, softmax and accumulation.
-//                      Optional: a sliding window (with first tokens that stay visible), scores capped by
-//                      cap * tanh(s / cap), a sink logit per head that joins the softmax denominator without a value, an output gate sigmoid(logit) per (token, head).
+//                      Optional: a sliding window (with first tokens that stay visible) or chunks (a token sees its
+//                      own chunk only), scores capped by cap * tanh(s / cap), a sink logit per head that joins the
+//                      softmax denominator without a value, an output gate sigmoid(logit) per (token, head).
 //   linear_recurrence  S_t = a_t S_(t-1) + k_t (b_t v_t)^T, o_t = S_t^T q_t (+ d v_t) per head with the state S
 //                      [key size x value size] held in fp32 registers and carried between steps in a slot.
 //                      Three forms: a constant decay per head (lightning attention), a decay and a step size
@@ -29,7 +30,7 @@ attn_generic_kernel(T* __restrict__ out, const T* __restrict__ q, int64_t q_stri
                     int64_t k_stride, const T* __restrict__ v, int64_t v_stride,
                     const int* __restrict__ block_tables, int bt_stride, int block_size,
                     const int* __restrict__ cu_q, const int* __restrict__ cu_k, const int* __restrict__ ctx_lens,
-                    int H, int G, int dim, int vdim, float scale, int window, int keep_first, float softcap,
+                    int H, int G, int dim, int vdim, float scale, int window, int keep_first, int chunk, float softcap,
                     const float* __restrict__ sink, const T* __restrict__ gate, int64_t gate_stride) {
   extern __shared__ float smem[];
   pdl_wait();
@@ -52,7 +53,8 @@ attn_generic_kernel(T* __restrict__ out, const T* __restrict__ q, int64_t q_stri
   const bool live = r < rows;
   const int tok = live ? r / rep : 0, head = g * rep + (live ? r % rep : 0);
   const int pos = sp.first_pos() + tok;               // this row sees keys lo .. pos, and those below keep_first
-  const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+  auto seen_from = [&](int p) { return window > 0 ? max(0, p - window + 1) : chunk > 0 ? p / chunk * chunk : 0; };
+  const int lo = seen_from(pos);
   if (live) {
     const T* qr = q + (int64_t)(sp.q_start + tok) * q_stride + (int64_t)head * dim;
     for (int i = lane; i < dim; i += 32) sq[warp * dim + i] = to_f32<T>(qr[i]);
@@ -67,7 +69,7 @@ attn_generic_kernel(T* __restrict__ out, const T* __restrict__ q, int64_t q_stri
   for (int c = 0; c < kAttnMaxVChunks; ++c) acc[c] = 0.f;
 
   const int min_pos = sp.first_pos() + r0 / rep;
-  const int first_key = window > 0 ? max(0, min_pos - window + 1) : 0;
+  const int first_key = seen_from(min_pos);
   // tiles of the kept keys first, then from the first key of the earliest row's window on
   const int kept = min(keep_first, first_key);
   for (int j0 = kept > 0 ? 0 : first_key; j0 <= max_pos;
@@ -662,7 +664,7 @@ extern "C" int b200_attn_generic(void* out, const void* q, int64_t q_stride, con
                                  int32_t bt_stride, int32_t block_size, const int32_t* cu_q,
                                  const int32_t* cu_k, const int32_t* ctx_lens, int32_t num_seqs, int32_t max_q,
                                  int32_t num_heads, int32_t num_kv_heads, int32_t dim, int32_t vdim,
-                                 float scale, int32_t window, int32_t keep_first, float softcap,
+                                 float scale, int32_t window, int32_t keep_first, int32_t chunk, float softcap,
                                  const float* sink, const void* gate, int64_t gate_stride, int32_t dtype, b200_stream_t stream) {
   B200_RETURN_IF(num_seqs < 0 || max_q < 0 || num_heads <= 0 || num_kv_heads <= 0 || dim <= 0 || vdim <= 0 ||
                      num_heads % num_kv_heads != 0, B200_ERR_BAD_SHAPE);
@@ -671,7 +673,7 @@ extern "C" int b200_attn_generic(void* out, const void* q, int64_t q_stride, con
   B200_RETURN_IF(!out || !q || !k || (cu_q == nullptr) == (ctx_lens == nullptr) || (cu_q && !cu_k),
                  B200_ERR_NULL_POINTER);
   B200_RETURN_IF(block_tables && block_size <= 0, B200_ERR_BAD_SHAPE);
-  B200_RETURN_IF(window < 0 || keep_first < 0 || (!v && vdim > dim), B200_ERR_BAD_SHAPE);
+  B200_RETURN_IF(window < 0 || keep_first < 0 || chunk < 0 || (window > 0 && chunk > 0) || (!v && vdim > dim), B200_ERR_BAD_SHAPE);
   B200_RETURN_IF(!block_tables && !cu_q, B200_ERR_NULL_POINTER);       // decode rows read the paged cache
   const int rep = num_heads / num_kv_heads;
   const dim3 grid((max_q * rep + kAttnRows - 1) / kAttnRows, num_kv_heads, num_seqs);
@@ -682,8 +684,8 @@ extern "C" int b200_attn_generic(void* out, const void* q, int64_t q_stride, con
       cudaFuncSetAttribute(attn_generic_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     launch_pdl(attn_generic_kernel<T>, grid, dim3(kAttnRows * 32), smem, (cudaStream_t)stream, (T*)out,
                (const T*)q, q_stride, (const T*)k, k_stride, (const T*)v, v_stride, block_tables, bt_stride,
-               block_size, cu_q, cu_k, ctx_lens, num_heads, num_kv_heads, dim, vdim, scale, window, keep_first, softcap,
-               sink,               (const T*)gate, gate_stride);
+               block_size, cu_q, cu_k, ctx_lens, num_heads, num_kv_heads, dim, vdim, scale, window, keep_first, chunk,
+               softcap, sink, (const T*)gate, gate_stride);
   });
   return finish_launch();
 }

@@ -17,6 +17,9 @@
 //                        operand layout of attention composed of batched products
 //   residual_scale_groupnorm  r (+)= c * scale[channel] * y (rows of y optionally gathered by index: the scaled token
 //                        embedding); h = RMS norm of r in equal consecutive groups, times a weight
+//   residual_gate_average  r + sigmoid(gate) * y, kept as one entry of a history; then the weighted sum of the history and
+//                        itself; h = RMS norm of that
+//   logit_cap            logits times a scale, capped by cap * tanh(z / cap), fp32
 //   rotary_table         cos / sin of position * frequency for a table of frequencies (fp64 angles), times a magnitude
 //   rope_mix_cache       rotation of part of every q and k head by that table, values blended with another layer's
 //                        values of the same token, K/V scatter
@@ -428,13 +431,13 @@ gated_norm_kernel(T* __restrict__ out, const Y* __restrict__ y, const T* __restr
 // x: [rows, 2 * inter] (gate | up) -> out [rows, inter]. act: 0 silu, 1 relu, 2 gelu (tanh form).
 template <typename T>
 __global__ void __launch_bounds__(256)
-act_and_mul_kernel(T* __restrict__ out, const T* __restrict__ x, int64_t rows, int inter, int act) {
+act_and_mul_kernel(T* __restrict__ out, const T* __restrict__ x, int64_t x_stride, int64_t rows, int inter, int act) {
   pdl_wait();
   const int64_t total = rows * inter;
   for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (int64_t)gridDim.x * blockDim.x) {
     const int64_t r = i / inter;
     const int c = (int)(i - r * inter);
-    const float g = to_f32<T>(x[r * 2 * inter + c]), u = to_f32<T>(x[r * 2 * inter + inter + c]);
+    const float g = to_f32<T>(x[r * x_stride + c]), u = to_f32<T>(x[r * x_stride + inter + c]);
     const float a = act == 1 ? fmaxf(g, 0.f) : act == 2 ? gelu_tanh_f(g) : silu_f(g);
     out[i] = from_f32<T>(a * u);
   }
@@ -442,15 +445,15 @@ act_and_mul_kernel(T* __restrict__ out, const T* __restrict__ x, int64_t rows, i
 
 template <typename T>
 __global__ void __launch_bounds__(256)
-act_and_mul_vec_kernel(T* __restrict__ out, const T* __restrict__ x, int64_t rows, int inter8, int act) {
+act_and_mul_vec_kernel(T* __restrict__ out, const T* __restrict__ x, int64_t x_stride, int64_t rows, int inter8, int act) {
   pdl_wait();
   const int64_t total = rows * inter8;
   for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (int64_t)gridDim.x * blockDim.x) {
     const int64_t r = i / inter8;
     const int c = (int)(i - r * inter8);
     float g[8], u[8], o[8];
-    load8<T>(x + (r * 2 * inter8 + c) * 8, g);
-    load8<T>(x + (r * 2 * inter8 + inter8 + c) * 8, u);
+    load8<T>(x + r * x_stride + c * 8, g);
+    load8<T>(x + r * x_stride + (inter8 + c) * 8, u);
 #pragma unroll
     for (int e = 0; e < 8; ++e) {
       const float a = act == 1 ? fmaxf(g[e], 0.f) : act == 2 ? gelu_tanh_f(g[e]) : silu_f(g[e]);
@@ -987,6 +990,167 @@ residual_scale_groupnorm_vec_kernel(T* __restrict__ h, float* __restrict__ res, 
   }
 }
 
+// ------------------------------------------------------------------ gated branch, depth average, norm
+// One row of a residual whose branches are gated and whose layers hand on a weighted sum of everything so far:
+//   v = (x_in ? x_in : 0) + c * y * (gate ? sigmoid(gate) : 1)      (y_index: row t of y is y[clamp(y_index[t])])
+//   keep[t] = v                                                     (optional: this layer's result joins the history)
+//   v = sum_(j < n) avg[j] * hist[j][t] + avg[n] * v                (optional: avg [n + 1], hist entry j at hist + j * stride)
+//   x_out[t] = v (optional);  h = v / sqrt(mean v^2 + eps) * w      (skipped when w == nullptr)
+// x, keep, hist are fp32 [rows, hidden]; y, gate and h have the element type. keep may be an entry of hist >= n.
+struct GateAverageParams {
+  void* h;
+  const float* x_in;
+  float* x_out;
+  const void* y;
+  const int64_t* y_index;
+  int64_t y_rows;
+  const void* gate;
+  int64_t gate_stride;
+  float c;
+  float* keep;
+  const float *hist, *avg;
+  int64_t hist_stride;
+  const float* w;
+  float eps;
+  int n, hidden;
+};
+
+template <typename T>
+__device__ __forceinline__ const T* gate_average_row(const GateAverageParams& P) {
+  int64_t src = blockIdx.x;
+  if (P.y_index != nullptr) src = min(max(P.y_index[blockIdx.x], (int64_t)0), P.y_rows - 1);
+  return (const T*)P.y + src * P.hidden;
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+residual_gate_average_kernel(const GateAverageParams P) {
+  extern __shared__ float row[];                     // [hidden]
+  __shared__ float red[32];
+  pdl_wait();
+  const int64_t at = (int64_t)blockIdx.x * P.hidden;
+  const T* yr = gate_average_row<T>(P);
+  const T* gr = P.gate != nullptr ? (const T*)P.gate + (int64_t)blockIdx.x * P.gate_stride : nullptr;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < P.hidden; i += blockDim.x) {
+    float v = P.x_in != nullptr ? P.x_in[at + i] : 0.f;
+    v += P.c * to_f32<T>(yr[i]) * (gr != nullptr ? sigmoid_f(to_f32<T>(gr[i])) : 1.0f);
+    if (P.keep != nullptr) P.keep[at + i] = v;
+    if (P.avg != nullptr) {
+      float s = 0.f;
+      for (int j = 0; j < P.n; ++j) s += P.avg[j] * P.hist[j * P.hist_stride + at + i];
+      v = s + P.avg[P.n] * v;
+    }
+    if (P.x_out != nullptr) P.x_out[at + i] = v;
+    row[i] = v;
+    ss += v * v;
+  }
+  if (P.w == nullptr) return;
+  const float rstd = 1.0f / sqrtf(cta_sum(ss, red) / (float)P.hidden + P.eps);
+  T* o = (T*)P.h + at;
+  for (int i = threadIdx.x; i < P.hidden; i += blockDim.x) o[i] = from_f32<T>(row[i] * rstd * P.w[i]);
+}
+
+// 16-byte form (hidden % 8 == 0, hidden <= 8 * 256 * NV, 16-byte aligned rows): the row stays in registers; four
+// history rows are in flight per step
+template <typename T, int NV>
+__global__ void __launch_bounds__(256)
+residual_gate_average_vec_kernel(const GateAverageParams P) {
+  __shared__ float red[32];
+  pdl_wait();
+  const int nvec = P.hidden / 8;
+  const int64_t at = (int64_t)blockIdx.x * P.hidden;
+  const T* yr = gate_average_row<T>(P);
+  const T* gr = P.gate != nullptr ? (const T*)P.gate + (int64_t)blockIdx.x * P.gate_stride : nullptr;
+  float val[NV][8];
+  float ss = 0.f;
+#pragma unroll
+  for (int m = 0; m < NV; ++m) {
+    const int vi = threadIdx.x + m * blockDim.x;
+    if (vi >= nvec) continue;
+    const int64_t o = at + vi * 8;
+    float sum[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) sum[e] = 0.f;
+    if (P.avg != nullptr) {
+      int j = 0;
+      for (; j + 4 <= P.n; j += 4) {
+        float r[4][8], a[4];
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+          load8<float>(P.hist + (j + u) * P.hist_stride + o, r[u]);
+          a[u] = P.avg[j + u];
+        }
+#pragma unroll
+        for (int u = 0; u < 4; ++u)
+#pragma unroll
+          for (int e = 0; e < 8; ++e) sum[e] += a[u] * r[u][e];
+      }
+      for (; j < P.n; ++j) {
+        float r[8];
+        load8<float>(P.hist + j * P.hist_stride + o, r);
+        const float a = P.avg[j];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) sum[e] += a * r[e];
+      }
+    }
+    float y[8], g[8];
+    load8<T>(yr + vi * 8, y);
+    if (P.x_in != nullptr) {
+      load8<float>(P.x_in + o, val[m]);
+    } else {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) val[m][e] = 0.f;
+    }
+    if (gr != nullptr) {
+      load8<T>(gr + vi * 8, g);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) y[e] *= sigmoid_f(g[e]);
+    }
+#pragma unroll
+    for (int e = 0; e < 8; ++e) val[m][e] += P.c * y[e];
+    if (P.keep != nullptr) store8<float>(P.keep + o, val[m]);
+    if (P.avg != nullptr) {
+      const float a = P.avg[P.n];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) val[m][e] = sum[e] + a * val[m][e];
+    }
+    if (P.x_out != nullptr) store8<float>(P.x_out + o, val[m]);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) ss += val[m][e] * val[m][e];
+  }
+  if (P.w == nullptr) return;
+  const float rstd = 1.0f / sqrtf(cta_sum(ss, red) / (float)P.hidden + P.eps);
+  T* h = (T*)P.h + at;
+#pragma unroll
+  for (int m = 0; m < NV; ++m) {
+    const int vi = threadIdx.x + m * blockDim.x;
+    if (vi >= nvec) continue;
+    float wv[8];
+    load8<float>(P.w + vi * 8, wv);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) val[m][e] *= rstd * wv[e];
+    store8<T>(h + vi * 8, val[m]);
+  }
+}
+
+// ------------------------------------------------------------------ scaled and capped logits
+// z <- cap * tanh(scale * z / cap) in place (cap == 0: scale alone), fp32
+__global__ void __launch_bounds__(256)
+logit_cap_kernel(float* __restrict__ z, int64_t total, float scale, float cap) {
+  pdl_wait();
+  const float pre = cap > 0.f ? scale / cap : scale;
+  const int64_t step = (int64_t)gridDim.x * blockDim.x, nvec = total / 4;
+  for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < nvec; i += step) {
+    float4 v = reinterpret_cast<float4*>(z)[i];
+    v.x *= pre, v.y *= pre, v.z *= pre, v.w *= pre;
+    if (cap > 0.f) v.x = cap * tanhf(v.x), v.y = cap * tanhf(v.y), v.z = cap * tanhf(v.z), v.w = cap * tanhf(v.w);
+    reinterpret_cast<float4*>(z)[i] = v;
+  }
+  for (int64_t i = nvec * 4 + (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += step)
+    z[i] = cap > 0.f ? cap * tanhf(z[i] * pre) : z[i] * pre;
+}
+
 // ------------------------------------------------------------------ rotary positions from a table of frequencies
 // table[t][i] = (cos, sin)(positions[t] * freq[i]) * magnitude: fp64 angle (a position times a frequency loses digits
 // in fp32 at long range), fp32 result. Computed once per step for all layers that share the frequencies.
@@ -1472,24 +1636,24 @@ extern "C" int b200_gated_norm(void* out, const void* y, int32_t y_is_f32, const
   return finish_launch();
 }
 
-extern "C" int b200_act_and_mul(void* out, const void* x, int32_t rows, int32_t inter, int32_t act,
+extern "C" int b200_act_and_mul(void* out, const void* x, int64_t x_stride, int32_t rows, int32_t inter, int32_t act,
                                 int32_t dtype, b200_stream_t stream) {
-  B200_RETURN_IF(rows < 0 || inter <= 0 || act < 0 || act > 2, B200_ERR_BAD_SHAPE);
+  B200_RETURN_IF(rows < 0 || inter <= 0 || x_stride < 2 * (int64_t)inter || act < 0 || act > 2, B200_ERR_BAD_SHAPE);
   if (rows == 0) return B200_OK;
   B200_RETURN_IF(!out || !x, B200_ERR_NULL_POINTER);
-  if (inter % 8 == 0 && aligned16(out) && aligned16(x)) {
+  if (inter % 8 == 0 && x_stride % 8 == 0 && aligned16(out) && aligned16(x)) {
     const int64_t vecs = (int64_t)rows * (inter / 8);
     int vgrid = (int)((vecs + 255) / 256);
     if (vgrid > 148 * 16) vgrid = 148 * 16;
     B200_DISPATCH_3(dtype, T, launch_pdl(act_and_mul_vec_kernel<T>, dim3(vgrid), dim3(256), 0, (cudaStream_t)stream,
-                                         (T*)out, (const T*)x, (int64_t)rows, inter / 8, act));
+                                         (T*)out, (const T*)x, x_stride, (int64_t)rows, inter / 8, act));
     return finish_launch();
   }
   const int64_t total = (int64_t)rows * inter;
   int grid = (int)((total + 255) / 256);
   if (grid > 148 * 16) grid = 148 * 16;
   B200_DISPATCH_3(dtype, T, launch_pdl(act_and_mul_kernel<T>, dim3(grid), dim3(256), 0, (cudaStream_t)stream,
-                                       (T*)out, (const T*)x, (int64_t)rows, inter, act));
+                                       (T*)out, (const T*)x, x_stride, (int64_t)rows, inter, act));
   return finish_launch();
 }
 
@@ -1624,6 +1788,53 @@ extern "C" int b200_residual_scale_groupnorm(void* h, float* residual, const voi
     launch_pdl(residual_scale_groupnorm_kernel<T>, dim3(rows), dim3(256), smem, (cudaStream_t)stream, (T*)h, residual,
                (const T*)y, y_index, y_rows, scale, c, accumulate, weight, offset, eps, hidden, groups);
   });
+  return finish_launch();
+}
+
+extern "C" int b200_residual_gate_average(void* h, const float* x_in, float* x_out, const void* y,
+                                          const int64_t* y_index, int64_t y_rows, const void* gate, int64_t gate_stride,
+                                          float c, float* keep, const float* hist, int64_t hist_stride, int32_t n,
+                                          const float* avg, const float* weight, float eps, int32_t rows, int32_t hidden,
+                                          int32_t dtype, b200_stream_t stream) {
+  B200_RETURN_IF(rows < 0 || hidden <= 0 || n < 0 || (y_index && y_rows <= 0), B200_ERR_BAD_SHAPE);
+  if (rows == 0) return B200_OK;
+  B200_RETURN_IF(!y || (weight && !h) || (avg && n > 0 && !hist), B200_ERR_NULL_POINTER);
+  GateAverageParams P{h, x_in, x_out, y, y_index, y_rows, gate, gate_stride, c, keep, hist, avg, hist_stride, weight, eps,
+                      n, hidden};
+  const bool vec = hidden % 8 == 0 && hidden <= 8 * 256 * kResVecs && aligned16(y) && (!h || aligned16(h)) &&
+                   (!x_in || aligned16(x_in)) && (!x_out || aligned16(x_out)) && (!keep || aligned16(keep)) &&
+                   (!gate || (aligned16(gate) && gate_stride % 8 == 0)) && (!weight || aligned16(weight)) &&
+                   (!avg || n == 0 || (aligned16(hist) && hist_stride % 4 == 0));
+  if (vec) {
+    const int nvec = hidden / 8;
+    const int threads = nvec >= 256 ? 256 : ((nvec + 31) / 32) * 32;
+#define B200_GATE_AVERAGE(NV)                                                                                       \
+  B200_DISPATCH_3(dtype, T, launch_pdl(residual_gate_average_vec_kernel<T, NV>, dim3(rows), dim3(threads), 0,       \
+                                       (cudaStream_t)stream, P))
+    if (nvec <= 256) B200_GATE_AVERAGE(1);
+    else if (nvec <= 512) B200_GATE_AVERAGE(2);
+    else B200_GATE_AVERAGE(kResVecs);
+#undef B200_GATE_AVERAGE
+    return finish_launch();
+  }
+  const size_t smem = (size_t)hidden * sizeof(float);
+  B200_RETURN_IF(smem > 200 * 1024, B200_ERR_UNSUPPORTED);
+  B200_DISPATCH_3(dtype, T, {
+    if (smem > 48 * 1024)
+      cudaFuncSetAttribute(residual_gate_average_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    launch_pdl(residual_gate_average_kernel<T>, dim3(rows), dim3(256), smem, (cudaStream_t)stream, P);
+  });
+  return finish_launch();
+}
+
+extern "C" int b200_logit_cap(float* z, int64_t total, float scale, float cap, b200_stream_t stream) {
+  B200_RETURN_IF(total < 0 || cap < 0.f, B200_ERR_BAD_SHAPE);
+  if (total == 0) return B200_OK;
+  B200_RETURN_IF(!z, B200_ERR_NULL_POINTER);
+  B200_RETURN_IF(!aligned16(z), B200_ERR_MISALIGNED);
+  int64_t grid = (total / 4 + 256) / 256;
+  if (grid > 148 * 16) grid = 148 * 16;
+  launch_pdl(logit_cap_kernel, dim3((unsigned)grid), dim3(256), 0, (cudaStream_t)stream, z, total, scale, cap);
   return finish_launch();
 }
 

@@ -5,13 +5,13 @@
 //                       h = norm(u): the "residual add + next pre-norm" of a multi-stream residual in ONE launch.
 //                       norm is a layer norm with weight and bias, or an RMS norm with a (offset + w) weight.
 //   rotary_heads        rotary positions on the first `dims` columns of every head (pairs (2i, 2i+1) or
-//                       (i, i + dims/2)), a scale per head range, output in fp32 or the element type, with free
+//                       (i, i + dims/2); angles from a base, or a table of cos and sin), a scale per head range, output in fp32 or the element type, with free
 //                       input/output head strides (so that a rotated part can be written into a wider head).
 //   delta_prep          what a gated delta rule reads besides v: q and k as fp32 unit vectors (q scaled), the decay
 //                       exp(-exp(A) softplus(a + bias)) per key channel or per head, and beta = sigmoid(b), all fp32.
 //   wkv_prep            what a wkv recurrence reads besides v: the receptance and k in fp32, the decay exp(-exp(z + w0))
 //                       and the coefficient sum_i r_i u_i k_i with which the current token counts, all fp32.
-//   latent_kv_prep      RMS norm of the query latent; RMS norm of the key/value latent and rotation of the shared
+//   latent_kv_prep      RMS norm of the query latent (where there is one); RMS norm of the key/value latent and rotation of the shared
 //                       rotated key, written as one cache row [latent | rotated key] (packed and/or paged).
 //   glu_clamped         min(g, L) sigmoid(alpha min(g, L)) (clamp(u, -L, L) + 1) for a gated feed-forward.
 //   masked_softmax      softmax over the visible keys of a block of fp32 scores (attention composed of library products).
@@ -196,6 +196,7 @@ struct RotaryParams {
   int64_t in_stride, out_stride;
   int in_head, out_head;
   const int64_t* positions;
+  const float2* table;     // (cos, sin) per (token, pair), or nullptr: computed from positions and log2_base
   int tokens, heads, width, dims, interleaved, split, out_f32;
   int hsplit;                 // threads per (token, pair): each takes every hsplit-th head (few tokens: more threads)
   float scale_lo, scale_hi;   // heads < split are multiplied by scale_lo, the others by scale_hi
@@ -217,10 +218,16 @@ rotary_heads_kernel(const RotaryParams P) {
     float* of = (float*)P.out + (int64_t)t * P.out_stride;
     T* ot = (T*)P.out + (int64_t)t * P.out_stride;
     if (w < half) {
-      const double f = exp2(-(2.0 * (double)w / (double)P.dims) * P.log2_base);
-      double sn, cs;
-      sincos((double)P.positions[t] * f, &sn, &cs);
-      const float c = (float)cs, s = (float)sn;
+      float c, s;
+      if (P.table != nullptr) {
+        const float2 r = P.table[(int64_t)t * half + w];
+        c = r.x, s = r.y;
+      } else {
+        const double f = exp2(-(2.0 * (double)w / (double)P.dims) * P.log2_base);
+        double sn, cs;
+        sincos((double)P.positions[t] * f, &sn, &cs);
+        c = (float)cs, s = (float)sn;
+      }
       const int a = P.interleaved ? 2 * w : w, b = P.interleaved ? 2 * w + 1 : w + half;
       for (int hd = h0; hd < P.heads; hd += P.hsplit) {
         const float sc = hd < P.split ? P.scale_lo : P.scale_hi;
@@ -346,27 +353,29 @@ wkv_prep_kernel(float* __restrict__ r_out, float* __restrict__ k_out, float* __r
 }
 
 // ------------------------------------------------------------------ latents of a latent attention
-// One CTA per token. cq = rms(dq) * wq (element type); row = [rms(c) * wc | rotate(kr)] (element type) into `kc`
+// One CTA per token. cq = rms(dq) * wq (element type; skipped without dq); row = [rms(c) * wc | rotate(kr)] (element type) into `kc`
 // (packed, [tokens, rank + rot]) and, when slots are given, into the paged cache row of the token.
 template <typename T>
 __global__ void __launch_bounds__(128)
 latent_kv_prep_kernel(T* __restrict__ cq, T* __restrict__ kc, T* __restrict__ cache, const int* __restrict__ slots,
                       int slot_pairs, int block_size, const T* __restrict__ dq, int64_t dq_stride,
                       const T* __restrict__ dkv, int64_t dkv_stride, const float* __restrict__ wq,
-                      const float* __restrict__ wc, const int64_t* __restrict__ positions, int q_rank, int rank,
-                      int rot, int dims, int interleaved, double log2_base, float eps) {
+                      const float* __restrict__ wc, const int64_t* __restrict__ positions,
+                      const float2* __restrict__ table, int q_rank, int rank, int rot, int dims, int interleaved, double log2_base, float eps) {
   __shared__ float red[32];
   pdl_wait();
   const int64_t t = blockIdx.x;
-  const T* q = dq + t * dq_stride;
-  float ss = 0.f;
-  for (int i = threadIdx.x; i < q_rank; i += blockDim.x) {
-    const float v = to_f32<T>(q[i]);
-    ss += v * v;
+  float ss = 0.f, rstd;
+  if (dq != nullptr) {
+    const T* q = dq + t * dq_stride;
+    for (int i = threadIdx.x; i < q_rank; i += blockDim.x) {
+      const float v = to_f32<T>(q[i]);
+      ss += v * v;
+    }
+    rstd = 1.0f / sqrtf(cta_sum(ss, red) / (float)q_rank + eps);
+    for (int i = threadIdx.x; i < q_rank; i += blockDim.x)
+      cq[t * q_rank + i] = from_f32<T>(to_f32<T>(q[i]) * rstd * wq[i]);
   }
-  float rstd = 1.0f / sqrtf(cta_sum(ss, red) / (float)q_rank + eps);
-  for (int i = threadIdx.x; i < q_rank; i += blockDim.x)
-    cq[t * q_rank + i] = from_f32<T>(to_f32<T>(q[i]) * rstd * wq[i]);
 
   const T* c = dkv + t * dkv_stride;
   ss = 0.f;
@@ -390,10 +399,16 @@ latent_kv_prep_kernel(T* __restrict__ cq, T* __restrict__ kc, T* __restrict__ ca
   const int half = dims / 2;
   for (int w = threadIdx.x; w < half + (rot - dims); w += blockDim.x) {
     if (w < half) {
-      const double f = exp2(-(2.0 * (double)w / (double)dims) * log2_base);
-      double sn, cs;
-      sincos((double)positions[t] * f, &sn, &cs);
-      const float cc = (float)cs, s = (float)sn;
+      float cc, s;
+      if (table != nullptr) {
+        const float2 r = table[t * half + w];
+        cc = r.x, s = r.y;
+      } else {
+        const double f = exp2(-(2.0 * (double)w / (double)dims) * log2_base);
+        double sn, cs;
+        sincos((double)positions[t] * f, &sn, &cs);
+        cc = (float)cs, s = (float)sn;
+      }
       const int a = interleaved ? 2 * w : w, b = interleaved ? 2 * w + 1 : w + half;
       const float u = to_f32<T>(c[rank + a]), v = to_f32<T>(c[rank + b]);
       const T ra = from_f32<T>(u * cc - v * s), rb = from_f32<T>(v * cc + u * s);
@@ -675,8 +690,8 @@ extern "C" int b200_stream_mix_norm(void* h, float* x, const void* y, const floa
 }
 
 extern "C" int b200_rotary_heads(void* out, int64_t out_stride, int32_t out_head, int32_t out_f32, const void* in,
-                                 int64_t in_stride, int32_t in_head, const int64_t* positions, int32_t tokens,
-                                 int32_t heads, int32_t width, int32_t dims, double base, int32_t interleaved,
+                                 int64_t in_stride, int32_t in_head, const int64_t* positions, const float* table,
+                                 int32_t tokens, int32_t heads, int32_t width, int32_t dims, double base, int32_t interleaved,
                                  int32_t split, float scale_lo, float scale_hi, int32_t dtype,
                                  b200_stream_t stream) {
   B200_RETURN_IF(tokens < 0 || heads <= 0 || width <= 0 || dims < 0 || dims > width || dims % 2 != 0 || base <= 0.0,
@@ -684,6 +699,7 @@ extern "C" int b200_rotary_heads(void* out, int64_t out_stride, int32_t out_head
   if (tokens == 0) return B200_OK;
   B200_RETURN_IF(!out || !in || !positions, B200_ERR_NULL_POINTER);
   RotaryParams P;
+  P.table = reinterpret_cast<const float2*>(table);
   P.in = in, P.out = out, P.in_stride = in_stride, P.out_stride = out_stride, P.in_head = in_head;
   P.out_head = out_head, P.positions = positions, P.tokens = tokens, P.heads = heads, P.width = width;
   P.dims = dims, P.interleaved = interleaved, P.split = split, P.out_f32 = out_f32, P.scale_lo = scale_lo;
@@ -742,17 +758,17 @@ extern "C" int b200_wkv_prep(float* r_out, float* k_out, float* decay, float* bo
 extern "C" int b200_latent_kv_prep(void* cq, void* kc, void* cache, const int32_t* slots, int32_t slot_pairs,
                                    int32_t block_size, const void* dq, int64_t dq_stride, const void* dkv,
                                    int64_t dkv_stride, const float* wq, const float* wc, const int64_t* positions,
-                                   int32_t tokens, int32_t q_rank, int32_t rank, int32_t rot, int32_t dims,
+                                   const float* table, int32_t tokens, int32_t q_rank, int32_t rank, int32_t rot, int32_t dims,
                                    double base, int32_t interleaved, float eps, int32_t dtype,
                                    b200_stream_t stream) {
-  B200_RETURN_IF(tokens < 0 || q_rank <= 0 || rank <= 0 || rot < 0 || dims < 0 || dims > rot || dims % 2 != 0 ||
+  B200_RETURN_IF(tokens < 0 || (dq && q_rank <= 0) || rank <= 0 || rot < 0 || dims < 0 || dims > rot || dims % 2 != 0 ||
                      base <= 0.0, B200_ERR_BAD_SHAPE);
   if (tokens == 0) return B200_OK;
-  B200_RETURN_IF(!cq || !dq || !dkv || !wq || !wc || !positions || (cache && !slots), B200_ERR_NULL_POINTER);
+  B200_RETURN_IF((dq && (!cq || !wq)) || !dkv || !wc || !positions || (cache && !slots), B200_ERR_NULL_POINTER);
   B200_DISPATCH_3(dtype, T, launch_pdl(latent_kv_prep_kernel<T>, dim3(tokens), dim3(128), 0, (cudaStream_t)stream,
                                        (T*)cq, (T*)kc, (T*)cache, slots, slot_pairs, block_size, (const T*)dq,
-                                       dq_stride, (const T*)dkv, dkv_stride, wq, wc, positions, q_rank, rank, rot,
-                                       dims, interleaved, log2(base), eps));
+                                       dq_stride, (const T*)dkv, dkv_stride, wq, wc, positions,
+                                       reinterpret_cast<const float2*>(table), q_rank, rank, rot, dims, interleaved, log2(base), eps));
   return finish_launch();
 }
 

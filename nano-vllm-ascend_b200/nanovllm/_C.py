@@ -59,11 +59,11 @@ PROTOTYPES = {
                                                     c_int32, c_int32, c_int32, c_int32, c_int32, c_int32, c_int32,
                                                     c_int32, c_int64, c_int64, c_int64, c_int64, c_void_p, c_int32,
                                                     c_int32, c_int32, c_float, c_float, c_void_p, c_int32, c_int32,
-                                                    c_int32, c_void_p, c_int64, c_void_p]),
+                                                    c_int32, c_int32, c_void_p, c_int64, c_void_p]),
     "b200_paged_decode_attn_windowed": (c_int32, [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int32,
                                                   c_int32, c_int32, c_int32, c_int32, c_int64, c_int64, c_int32,
                                                   c_int32, c_int32, c_float, c_float, c_void_p, c_int32, c_int32,
-                                                  c_void_p, c_size_t, c_int32, c_int32, c_void_p]),
+                                                  c_int32, c_void_p, c_size_t, c_int32, c_int32, c_void_p]),
     "b200_prefill_workspace_size": (c_int64, [c_int32]),
     "b200_prefill_set_query_tiles": (c_int32, [c_int32]),
     "b200_gather_dequant_fp8": (c_int32, [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int32,
@@ -84,7 +84,7 @@ PROTOTYPES = {
                                  c_int32, c_void_p]),
     "b200_moe_align": (c_int32, [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int32, c_int32,
                                  c_int32, c_void_p]),
-    "b200_moe_gemm_gate_up": (c_int32, [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int32,
+    "b200_moe_gemm_gate_up": (c_int32, [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int32,
                                         c_int32, c_int32, c_int32, c_int64, c_int32, c_void_p]),
     "b200_moe_gemm_gate_up_glu": (c_int32, [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int32,
                                             c_int32, c_int32, c_int32, c_int64, c_float, c_float, c_int32, c_void_p]),
@@ -94,8 +94,8 @@ PROTOTYPES = {
                                      c_int32, c_int32, c_int32, c_int32, c_int32, c_void_p]),
     "b200_moe_gather_rows": (c_int32, [c_void_p, c_void_p, c_void_p, c_void_p, c_int32, c_int32, c_int32,
                                        c_int32, c_int64, c_int32, c_void_p]),
-    "b200_moe_gemm_gate_up_umma": (c_int32, [c_void_p, c_void_p, c_void_p, c_void_p, c_int32, c_int32,
-                                             c_int32, c_int32, c_int32, c_void_p]),
+    "b200_moe_gemm_gate_up_umma": (c_int32, [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int32,
+                                             c_int32, c_int32, c_int32, c_int32, c_void_p]),
     "b200_gemm_f32out_umma": (c_int32, [c_void_p, c_void_p, c_void_p, c_void_p, c_int32, c_int32, c_int32, c_int32,
                                         c_int32, c_void_p]),
     "b200_moe_gemm_down_umma": (c_int32, [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
@@ -135,11 +135,11 @@ PROTOTYPES = {
                                            c_int32, c_int32, c_int32, c_void_p]),
     "b200_gated_norm": (c_int32, [c_void_p, c_void_p, c_int32, c_void_p, c_int64, c_void_p, c_float, c_int32,
                                   c_int32, c_int32, c_int32, c_int32, c_int64, c_float, c_int32, c_void_p]),
-    "b200_act_and_mul": (c_int32, [c_void_p, c_void_p, c_int32, c_int32, c_int32, c_int32, c_void_p]),
+    "b200_act_and_mul": (c_int32, [c_void_p, c_void_p, c_int64, c_int32, c_int32, c_int32, c_int32, c_void_p]),
     "b200_attn_generic": (c_int32, [c_void_p, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_void_p,
                                     c_int32, c_int32, c_void_p, c_void_p, c_void_p, c_int32, c_int32, c_int32,
-                                    c_int32, c_int32, c_int32, c_float, c_int32, c_int32, c_float, c_void_p, c_void_p,
-                                    c_int64, c_int32, c_void_p]),
+                                    c_int32, c_int32, c_int32, c_float, c_int32, c_int32, c_int32, c_float, c_void_p,
+                                    c_void_p, c_int64, c_int32, c_void_p]),
     "b200_linear_recurrence": (c_int32, [c_void_p, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64,
                                          c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int32, c_int32, c_int32,
                                          c_int32, c_int32, c_int32, c_int32, c_int32, c_void_p, c_void_p,
@@ -148,7 +148,7 @@ PROTOTYPES = {
     "b200_stream_mix_norm": (c_int32, [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                        c_void_p, c_void_p, c_float, c_float, c_int32, c_int32, c_int32, c_int32,
                                        c_int32, c_void_p]),
-    "b200_rotary_heads": (c_int32, [c_void_p, c_int64, c_int32, c_int32, c_void_p, c_int64, c_int32, c_void_p,
+    "b200_rotary_heads": (c_int32, [c_void_p, c_int64, c_int32, c_int32, c_void_p, c_int64, c_int32, c_void_p, c_void_p,
                                     c_int32, c_int32, c_int32, c_int32, c_double, c_int32, c_int32, c_float,
                                     c_float, c_int32, c_void_p]),
     "b200_delta_prep": (c_int32, [c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_int64, c_void_p,
@@ -160,13 +160,13 @@ PROTOTYPES = {
                                   c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int32, c_int32,
                                   c_int32, c_int32, c_int32, c_int32, c_int32, c_void_p]),
     "b200_latent_kv_prep": (c_int32, [c_void_p, c_void_p, c_void_p, c_void_p, c_int32, c_int32, c_void_p, c_int64,
-                                      c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int32, c_int32, c_int32,
-                                      c_int32, c_int32, c_double, c_int32, c_float, c_int32, c_void_p]),
+                                      c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_int32, c_int32,
+                                      c_int32, c_int32, c_int32, c_double, c_int32, c_float, c_int32, c_void_p]),
     "b200_masked_softmax": (c_int32, [c_void_p, c_void_p, c_int64, c_int32, c_int32, c_int32, c_int32, c_int32,
                                       c_float, c_void_p, c_void_p, c_void_p, c_int32, c_int32, c_void_p]),
     "b200_glu_clamped": (c_int32, [c_void_p, c_void_p, c_int32, c_int32, c_float, c_float, c_int32, c_void_p]),
     "b200_moe_route_grouped": (c_int32, [c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_int32, c_int32,
-                                         c_int32, c_int32, c_int32, c_float, c_void_p]),
+                                         c_int32, c_int32, c_int32, c_float, c_int32, c_void_p]),
     "b200_moe_route_topk": (c_int32, [c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_int32, c_int32, c_int32,
                                       c_void_p]),
     "b200_act_only": (c_int32, [c_void_p, c_void_p, c_int64, c_int32, c_int32, c_void_p]),
@@ -185,7 +185,7 @@ PROTOTYPES = {
                                   c_int32, c_int32, c_void_p, c_void_p, c_void_p, c_int32, c_int32, c_int32,
                                   c_int32, c_int32, c_int32, c_float, c_int32, c_void_p, c_void_p, c_void_p, c_int32,
                                   c_void_p]),
-    "b200_moe_gemm_generic": (c_int32, [c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int32,
+    "b200_moe_gemm_generic": (c_int32, [c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_int32,
                                         c_int32, c_int32, c_int32, c_int32, c_int32, c_float, c_float, c_int32,
                                         c_void_p]),
     "b200_moe_route_grouped_softmax": (c_int32, [c_void_p, c_void_p, c_void_p, c_int64, c_int32, c_int32, c_int32,
@@ -193,6 +193,10 @@ PROTOTYPES = {
     "b200_residual_scale_groupnorm": (c_int32, [c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_float,
                                                 c_int32, c_void_p, c_float, c_float, c_int32, c_int32, c_int32,
                                                 c_int32, c_void_p]),
+    "b200_residual_gate_average": (c_int32, [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_int64,
+                                             c_float, c_void_p, c_void_p, c_int64, c_int32, c_void_p, c_void_p, c_float,
+                                             c_int32, c_int32, c_int32, c_void_p]),
+    "b200_logit_cap": (c_int32, [c_void_p, c_int64, c_float, c_float, c_void_p]),
     "b200_rotary_table": (c_int32, [c_void_p, c_void_p, c_void_p, c_double, c_int32, c_int32, c_void_p]),
     "b200_rope_mix_cache": (c_int32, [c_void_p, c_int64, c_void_p, c_int32, c_int32, c_void_p, c_int64, c_void_p,
                                       c_void_p, c_void_p, c_void_p, c_int32, c_int32, c_int32, c_int32, c_int32,

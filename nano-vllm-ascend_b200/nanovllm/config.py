@@ -161,6 +161,28 @@ def pofazen_preset(width: int, pattern: str, repeats: int, vocab: int = 32768, h
             "layers": [entry[ch] for ch in pattern] * repeats}
 
 
+def ragilorn_preset(width: int, pattern: str, repeats: int, vocab: int = 32768, head_dim: int = 128,
+                    chunk: int = 512) -> dict:
+    """A Ragilorn configuration of realistic layer sizes for synthetic benchmarks: `pattern` is a string over
+    a (chunked attention + dense feed-forward), e (chunked attention + mixture of experts), l (latent attention + dense
+    feed-forward), m (latent attention + mixture of experts) and n (chunked attention alone), repeated `repeats` times."""
+    H = width // head_dim
+    kv = max(1, H // 4)
+    dr = head_dim // 2
+    stretch = {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}
+    att = {"heads": H, "kv_heads": kv, "dim": head_dim, "vdim": head_dim, "conv": 4, "scale": head_dim ** -0.5,
+           "mask": {"size": chunk}, "rot": {"dims": head_dim // 2, "base": 1e6, "scaling": stretch}}
+    lat = {"heads": H, "dim": head_dim, "rot_dim": dr, "vdim": head_dim, "kv_rank": 4 * head_dim,
+           "scale": (head_dim + dr) ** -0.5, "rot": {"dims": dr, "base": 1e5, "scaling": stretch}}
+    dense = {"kind": "dense", "ff": 3 * width}
+    moe = {"kind": "moe", "expert": {"ff": width // 2}, "router": {"experts": 16, "top": 2}}
+    entry = {"a": ("attention", att, dense), "e": ("attention", att, moe), "n": ("attention", att, None),
+             "l": ("latent_attention", lat, dense), "m": ("latent_attention", lat, moe)}
+    return {"architecture": "Ragilorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+            "embedding": {"scale": float(width) ** 0.5}, "logit_scale": 0.25, "logit_softcap": 30.0,
+            "layers": [{"type": t, "mixer": dict(m), "mlp": f} for t, m, f in (entry[ch] for ch in pattern)] * repeats}
+
+
 def preset_hf_config(name: str):
     """Architecture presets built offline from the public model cards."""
     from transformers import LlamaConfig, Qwen3Config, Qwen3MoeConfig
@@ -193,6 +215,12 @@ def preset_hf_config(name: str):
         return NativeConfig(pofazen_preset(2048, "pvwv", 4, vocab=128256, head_dim=64))
     if key == "tiny-pofazen":
         return NativeConfig(pofazen_preset(128, "pwv", 1, vocab=512, head_dim=32, window=24))
+    if key == "ragilorn-1k":         # 28 layers at width 1024: the size class of nirelix-1k and nurilorn-1k
+        return NativeConfig(ragilorn_preset(1024, "amalama", 4, vocab=151936))
+    if key == "ragilorn-2k":         # 16 layers at width 2048, head size 64: the size class of nirelix-2k
+        return NativeConfig(ragilorn_preset(2048, "amal", 4, vocab=128256, head_dim=64))
+    if key == "tiny-ragilorn":
+        return NativeConfig(ragilorn_preset(128, "amn", 1, vocab=512, head_dim=32, chunk=24))
     if key == "tiny-fitevik":
         return NativeConfig(fitevik_preset(128, "hgab", 1, vocab=512, head_dim=32, window=24, max_positions=512))
     if key == "qwen3-0.6b":

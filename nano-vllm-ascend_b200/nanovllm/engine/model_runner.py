@@ -543,8 +543,6 @@ class ModelRunner:
         logits = self.model.compute_logits(hidden)
         if self.d_logits is not None:
             self.d_logits[:bs].copy_(logits)
-        if logits.dtype == torch.float32:
-            logits = logits.to(torch.bfloat16)         # the sampling kernel reads 16-bit logits
         self.d_rng.add_(1)
         if self.rank == 0:
             self.sampler(logits, self.d_temp[:bs], out=self.d_out[:bs], step_offset=self.d_rng)
@@ -623,8 +621,6 @@ class ModelRunner:
                 reset_context()
                 return out.tolist()
             logits = self.model.compute_logits(self.model(ids, pos))
-            if logits is not None and logits.dtype == torch.float32:
-                logits = logits.to(torch.bfloat16)
             if self.rank == 0:
                 temps = torch.tensor([0.0 if s.greedy else s.temperature for s in seqs],
                                      dtype=torch.float32, pin_memory=True).to(self.device, non_blocking=True)

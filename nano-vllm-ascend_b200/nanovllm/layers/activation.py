@@ -4,7 +4,7 @@ import torch
 from torch import nn
 
 from .. import ops
-from .linear import MergedColumnParallelLinear, RowParallelLinear
+from .linear import MergedColumnParallelLinear, PaddedMergedLinear, RowParallelLinear
 
 
 class SiluAndMul(nn.Module):
@@ -28,13 +28,18 @@ class ClampedGatedFeedForward(nn.Module):
 
 class GatedFeedForward(nn.Module):
     """W_down(act(W_gate h) * W_up h) on the kernels that take any size and 16- or 32-bit elements; act: silu, relu or
-    gelu_tanh."""
+    gelu_tanh. ``extra`` columns (with a bias) that read the same input are computed in the same product: ``forward``
+    then returns them too."""
 
-    def __init__(self, width: int, ff: int, act: str = "silu"):
+    def __init__(self, width: int, ff: int, act: str = "silu", extra: int = 0):
         super().__init__()
-        self.act = act
-        self.gate_up_proj = MergedColumnParallelLinear(width, [ff, ff])
+        self.act, self.extra = act, int(extra)
+        self.gate_up_proj = (PaddedMergedLinear(width, [[ff, ff], extra], bias=True) if extra else
+                             MergedColumnParallelLinear(width, [ff, ff]))
         self.down_proj = RowParallelLinear(ff, width)
 
     def forward(self, h):
-        return self.down_proj(ops.act_and_mul(self.gate_up_proj(h), self.act))
+        p = self.gate_up_proj(h)
+        if not self.extra:
+            return self.down_proj(ops.act_and_mul(p, self.act))
+        return self.down_proj(ops.act_and_mul(self.gate_up_proj.part(p, 0), self.act)), self.gate_up_proj.part(p, 1)

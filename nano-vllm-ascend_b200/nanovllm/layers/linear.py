@@ -120,15 +120,18 @@ class PaddedMergedLinear(ReplicatedLinear):
     """Several matrices that read the same input, stacked with each part padded to a multiple of 8 rows (so
     that every part of the output starts on a 16-byte boundary) and, for ``pad_input``, the input columns padded
     to a multiple of 8 as well (the consumer of a padded part). A part may itself be a list of matrices, stacked without
-    padding between them and loaded as shard (part, matrix). Padding stays zero. Not sharded."""
+    padding between them and loaded as shard (part, matrix); with ``bias`` the bias vectors are loaded under the same shards
+    (a matrix without one keeps zeros). Padding stays zero. Not sharded."""
 
-    def __init__(self, input_size, output_sizes, pad_input=False):
+    def __init__(self, input_size, output_sizes, pad_input=False, bias=False):
         self.groups = [list(n) if isinstance(n, (list, tuple)) else [n] for n in output_sizes]
         self.output_sizes = [sum(g) for g in self.groups]
         self.padded_sizes = [-(-n // 8) * 8 for n in self.output_sizes]
         self.true_input = input_size
-        super().__init__(-(-input_size // 8) * 8 if pad_input else input_size, sum(self.padded_sizes))
+        super().__init__(-(-input_size // 8) * 8 if pad_input else input_size, sum(self.padded_sizes), bias)
         self.weight.data.zero_()
+        if bias:
+            self.bias.data.zero_()
 
     def part(self, y, i):
         """Columns of output y that belong to part i (without its padding)."""
@@ -143,12 +146,17 @@ class PaddedMergedLinear(ReplicatedLinear):
         off = 0
         for n, pad in zip(self.output_sizes, self.padded_sizes):
             self.weight.data[off + n:off + pad].zero_()
+            if self.bias is not None:
+                self.bias.data[off + n:off + pad].zero_()
             off += pad
         self.weight.data[:, self.true_input:].zero_()
 
     def weight_loader(self, param, loaded_weight, loaded_shard_id=0):
         part, inner = loaded_shard_id if isinstance(loaded_shard_id, tuple) else (loaded_shard_id, 0)
         start = sum(self.padded_sizes[:part]) + sum(self.groups[part][:inner])
+        if loaded_weight.dim() == 1:
+            param.data[start:start + loaded_weight.shape[0]].copy_(loaded_weight)
+            return
         param.data[start:start + loaded_weight.shape[0], :loaded_weight.shape[1]].copy_(loaded_weight)
 
 

@@ -4,8 +4,8 @@ decides what is written, the gated delta rule with a decay per key channel or pe
 for the current token), the mixes of a token with the token before that the wkv form reads, the gated norms that follow,
 rotary positions on part of a head (plain, or with frequencies stretched by a ramp between a fast and a slow band or
 between a short and a long wavelength), causal softmax attention whose key and value sizes may differ (optionally inside
-a sliding window with first tokens that stay visible, with capped scores, a sink in the denominator and a gate per head), attention whose heads are mixed before the softmax (with a distance bias, a sink, and keys and
-values that may be another layer's), attention over a cached latent, and the mixing weights of a residual that is
+a sliding window with first tokens that stay visible or inside chunks, with capped scores, a sink in the denominator and a gate per
+head), attention whose heads are mixed before the softmax (with a distance bias, a sink, and keys and values that may be another layer's), attention over a cached latent, and the mixing weights of a residual that is
 kept in several streams.
 
 Every block reads the step's ``Context`` (which tokens belong to which sequence, their cache slots and
@@ -136,15 +136,18 @@ class VarSizeAttention(nn.Module):
     ``k_cache`` [nb, bs, G*dim] / ``v_cache`` [nb, bs, G*vdim] (bound by the runner; K/V rows are written by the
     caller's fused epilogue). 16-bit models with dim and vdim in {64, 128} run on the tcgen05 prefill kernel and
     the paged decode kernel of the dense decoders; everything else (other sizes, fp32) on the generic kernel.
-    ``window`` w > 0: position i sees the keys j <= i with i - j < w, and those with j < ``keep_first``.
+    ``window`` w > 0: position i sees the keys j <= i with i - j < w, and those with j < ``keep_first``; ``chunk`` c > 0
+    (without a window): those with j // c == i // c, chunks counted from position 0.
     ``softcap`` c > 0 turns every score s into c tanh(s / c); ``sink`` (a logit) adds exp(sink) to every softmax
     denominator, an entry without key or value; ``forward(..., gate)`` multiplies head h of token t by sigmoid(gate[t, h])."""
 
     def __init__(self, num_heads: int, num_kv_heads: int, dim: int, vdim: int, scale: float, window: int = 0,
-                 softcap: float = 0.0, sink: float | None = None, keep_first: int = 0):
+                 softcap: float = 0.0, sink: float | None = None, keep_first: int = 0, chunk: int = 0):
         super().__init__()
+        if window and chunk:
+            raise ValueError("attention inside a window or inside chunks, not both")
         self.num_heads, self.num_kv_heads, self.dim, self.vdim, self.scale = num_heads, num_kv_heads, dim, vdim, scale
-        self.window, self.keep_first = int(window), int(keep_first)
+        self.window, self.keep_first, self.chunk = int(window), int(keep_first), int(chunk)
         self.softcap = float(softcap or 0.0)
         if sink is not None:
             self.register_buffer("sink", torch.full((num_heads,), float(sink), dtype=F32), persistent=False)
@@ -171,10 +174,10 @@ class VarSizeAttention(nn.Module):
         if self._fast(q) and (paged or ctx.is_prefill):
             out = None
             soft = dict(softcap=self.softcap, sink=self.sink, vdim=self.vdim, window=self.window,
-                        keep_first=self.keep_first)
-            plain = not self.softcap and self.sink is None and not self.window and self.dim == self.vdim
-            # a score cap, a sink, a window or unequal head sizes: the tcgen05 kernel only, whose TMA maps want 16-byte row strides and blocks that
-            # tile its 128-key steps
+                        keep_first=self.keep_first, chunk=self.chunk)
+            plain = not (self.softcap or self.sink is not None or self.window or self.chunk or self.dim != self.vdim)
+            # a score cap, a sink, a window, chunks or unequal head sizes: the tcgen05 kernel only, whose TMA maps want 16-byte
+            # row strides and blocks that tile its 128-key steps
             tma_ok = plain or (
                 q.stride(0) % 8 == 0 and (paged and (ctx.block_size % 128 == 0 or 128 % ctx.block_size == 0) or
                                           not paged and k.stride(0) % 8 == 0 and v.stride(0) % 8 == 0))
@@ -192,7 +195,8 @@ class VarSizeAttention(nn.Module):
                 out = out.view(q.shape[0], self.num_heads * self.vdim)
                 return out if gate is None else ops.head_gate_(out, gate, self.num_heads)
         spans = ops.StepSpans.of(ctx)
-        extras = dict(window=self.window, keep_first=self.keep_first, softcap=self.softcap, sink=self.sink, gate=gate)
+        extras = dict(window=self.window, keep_first=self.keep_first, chunk=self.chunk, softcap=self.softcap, sink=self.sink,
+                      gate=gate)
         if paged:
             return ops.attn_generic(q, self.k_cache, self.v_cache, spans, self.scale, self.num_kv_heads, self.vdim,
                                     block_tables=ctx.block_tables, **extras)
@@ -446,7 +450,7 @@ class TableRotary:
     """Rotary positions from a table of frequencies [dims / 2] (times a magnitude on cos and sin), pairs (2i, 2i+1)
     (``interleaved``) or (i, i + dims/2). The step's (cos, sin) table is computed once per pass (fp64 angles) and shared by
     all layers with the same constants; the rotation itself runs fused with the layer's cache write (ops.rope_mix_cache,
-    ops.norm_rope_cache)."""
+    ops.norm_rope_cache, ops.latent_kv_prep) or alone (ops.rotary_heads)."""
 
     def __init__(self, dims: int, freq: list, interleaved: bool = True, magnitude: float = 1.0):
         self.dims, self.interleaved, self.magnitude = int(dims), bool(interleaved), float(magnitude)
@@ -464,6 +468,11 @@ class TableRotary:
                 self.freq = self.freq.to(positions.device)
             t = ctx.scratch[self.key] = ops.rotary_table(positions, self.freq, self.magnitude)
         return t
+
+    def __call__(self, x, positions, out=None):
+        """x [T, heads, width] view -> rotated copy (in ``out`` when given, a view of the same shape)."""
+        return ops.rotary_heads(x, positions, x.shape[1], x.shape[2], self.dims, 1.0, self.interleaved, out=out,
+                                table=self.table(positions))
 
 
 class WavelengthScaledRotary(TableRotary):

@@ -8,7 +8,8 @@ streams) and Fitevik (HGRN2 recurrences and attention with mixed heads, a distan
 with the norm on each sublayer's output) and Nurilorn (gated attention with capped scores, a sink, rotary positions
 stretched band by band and values blended across layers, on a residual with scaled branches and grouped norms) and
 Pofazen (windowed gated attention beside a gated delta rule in one mixer, and wkv recurrences with a token shift, on a
-residual whose norm is taken of the sum) are additions; their config.json names them with an ``"architecture"`` string (config.NativeConfig). Qwen2 checkpoints are served by the Qwen3 class, as in the reference:
+residual whose norm is taken of the sum) and Ragilorn (attention inside chunks and latent attention, branches gated element
+by element, each layer handing on a weighted sum of all layers before it) are additions; their config.json names them with an ``"architecture"`` string (config.NativeConfig). Qwen2 checkpoints are served by the Qwen3 class, as in the reference:
 the config's ``attention_bias`` decides between QKV bias (Qwen2) and QK-norm (Qwen3).
 """
 from __future__ import annotations
@@ -20,6 +21,7 @@ from .fitevik import FitevikForCausalLM
 from .nirelix import NirelixForCausalLM
 from .nurilorn import NurilornForCausalLM
 from .pofazen import PofazenForCausalLM
+from .ragilorn import RagilornForCausalLM
 from .zegopel import ZegopelForCausalLM
 
 model_dict: dict[str, type] = {}
@@ -37,5 +39,6 @@ for _arch, _cls in (("Qwen3ForCausalLM", Qwen3ForCausalLM),
                     ("Nirelix", NirelixForCausalLM),
                     ("Fitevik", FitevikForCausalLM),
                     ("Nurilorn", NurilornForCausalLM),
-                    ("Pofazen", PofazenForCausalLM)):
+                    ("Pofazen", PofazenForCausalLM),
+                    ("Ragilorn", RagilornForCausalLM)):
     register(_arch, _cls)

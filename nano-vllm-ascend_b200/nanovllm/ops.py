@@ -123,10 +123,12 @@ def decode_workspace(batch, num_heads, num_kv_heads, head_dim, device) -> torch.
 
 
 def paged_decode_attn(q, k_cache, v_cache, block_tables, context_lens, scale, num_kv_heads,
-                      out=None, workspace=None, num_ctas=0, softcap=0.0, sink=None, vdim=None, window=0, keep_first=0):
+                      out=None, workspace=None, num_ctas=0, softcap=0.0, sink=None, vdim=None, window=0, keep_first=0,
+                      chunk=0):
     """K6. q [B, H, D] (token-strided view allowed) -> out [B, H*vdim] (vdim: width of a value head, D by default).
     softcap > 0: scores become softcap * tanh(score / softcap); sink fp32 [H]: exp(sink[h]) joins the softmax denominator
-    (no key, no value). window > 0: a row sees its last `window` keys and those below keep_first."""
+    (no key, no value). window > 0: a row sees its last `window` keys and those below keep_first; chunk > 0 (without a
+    window): the keys of its own chunk, counted from position 0."""
     _need_cuda(q, k_cache, v_cache, block_tables, context_lens, sink)
     _f32(sink)
     B, H, D = q.shape
@@ -151,7 +153,7 @@ def paged_decode_attn(q, k_cache, v_cache, block_tables, context_lens, scale, nu
         block_tables.data_ptr(), context_lens.data_ptr(), B, H, num_kv_heads, D, vdim,
         q.stride(0) if B > 1 else H * D, out.stride(0) if B > 1 else H * vdim, nb, bs,
         block_tables.stride(0), float(scale), float(softcap or 0.0), _ptr(sink), int(window), int(keep_first),
-        workspace.data_ptr(), workspace.numel(), int(num_ctas), _dt(q), _stream()), "b200_paged_decode_attn")
+        int(chunk), workspace.data_ptr(), workspace.numel(), int(num_ctas), _dt(q), _stream()), "b200_paged_decode_attn")
     return out
 
 
@@ -222,12 +224,12 @@ def prefill_workspace(device, head_dim: int) -> torch.Tensor:
 
 def prefill_varlen_attn(q, k, v, cu_seqlens_q, cu_seqlens_k, max_seqlen_q, max_seqlen_k, scale,
                         num_kv_heads, block_tables=None, out=None, workspace="auto", softcap=0.0, sink=None, vdim=None,
-                        window=0, keep_first=0):
+                        window=0, keep_first=0, chunk=0):
     """K4/K5. q [Tq, H, D]; packed mode: k/v [Tk, Hkv, D]; paged mode (block_tables given):
     k/v are the caches [nb, bs, Hkv*D]. Returns out [Tq, H*D]. workspace: "auto" (the per-device
     split-KV workspace), None (never split the keys across CTAs) or a uint8 CUDA tensor. softcap, sink, vdim, window,
-    keep_first as in paged_decode_attn (the tcgen05 kernel only); position i sees j <= i with i - j < window or
-    j < keep_first."""
+    keep_first, chunk as in paged_decode_attn (the tcgen05 kernel only); position i sees j <= i with i - j < window or
+    j < keep_first, or with j // chunk == i // chunk."""
     _need_cuda(q, k, v, cu_seqlens_q, cu_seqlens_k, block_tables, sink)
     _f32(sink)
     Tq, H, D = q.shape
@@ -263,8 +265,8 @@ def prefill_varlen_attn(q, k, v, cu_seqlens_q, cu_seqlens_k, max_seqlen_q, max_s
         cu_seqlens_k.data_ptr(), num_seqs, Tq, 0 if block_tables is not None else k.shape[0],
         int(max_seqlen_q), int(max_seqlen_k), H, num_kv_heads,
         D, vdim, q.stride(0) if Tq > 1 else H * D, ks, vs, out.stride(0) if Tq > 1 else H * vdim, bt_ptr,
-        bt_stride, nb, bs, float(scale), float(softcap or 0.0), _ptr(sink), int(window), int(keep_first), _dt(q), ws_ptr,
-        ws_bytes, _stream()),
+        bt_stride, nb, bs, float(scale), float(softcap or 0.0), _ptr(sink), int(window), int(keep_first), int(chunk), _dt(q),
+        ws_ptr, ws_bytes, _stream()),
         "b200_prefill_varlen_attn")
     return out
 
@@ -338,7 +340,7 @@ def silu_and_mul(x, out=None):
 
 
 def sample(logits, temperatures=None, seed=0, step=0, out=None, step_offset=None):
-    """argmax (temperatures=None or <= 0) or Gumbel-max sampling over [rows, vocab] bf16/fp16
+    """argmax (temperatures=None or <= 0) or Gumbel-max sampling over [rows, vocab] bf16/fp16/fp32
     logits. step_offset: optional device int64 scalar added to `step` when the kernel runs."""
     _need_cuda(logits, temperatures, step_offset)
     rows, vocab = logits.shape
@@ -351,7 +353,7 @@ def sample(logits, temperatures=None, seed=0, step=0, out=None, step_offset=None
         out = torch.empty(rows, dtype=torch.int64, device=logits.device)
     _C.check(_C.load().b200_sample(out.data_ptr(), logits.data_ptr(), _ptr(temperatures), rows,
                                    vocab, logits.stride(0) if rows > 1 else vocab, int(seed),
-                                   int(step), _ptr(step_offset), _dt(logits), _stream()),
+                                   int(step), _ptr(step_offset), _dt3(logits), _stream()),
              "b200_sample")
     return out
 
@@ -410,7 +412,7 @@ def gate_up_silu_umma(x: torch.Tensor, w_gate_up: torch.Tensor) -> torch.Tensor:
         raise ValueError("gate_up_silu_umma takes contiguous x [M, K] and w [2*I, K]")
     h = torch.empty(M, inter, dtype=x.dtype, device=x.device)
     _C.check(_C.load().b200_moe_gemm_gate_up_umma(h.data_ptr(), x.data_ptr(), w_gate_up.data_ptr(),
-                                                  _dense_plan(M, x.device).data_ptr(), M, K, inter, 1,
+                                                  _dense_plan(M, x.device).data_ptr(), None, None, M, K, inter, 1,
                                                   _dt(x), _stream()), "b200_moe_gemm_gate_up_umma (dense)")
     return h
 
@@ -497,8 +499,10 @@ def moe_align(topk_ids: torch.Tensor, expert_begin: int, num_local: int) -> MoeP
 
 
 def moe_experts(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, topk_ids: torch.Tensor,
-                topk_weights: torch.Tensor, plan: MoePlan, out: torch.Tensor | None = None) -> torch.Tensor:
-    """The expert MLPs of the local experts and the per-token combine.
+                topk_weights: torch.Tensor, plan: MoePlan, out: torch.Tensor | None = None,
+                weigh_input: bool = False) -> torch.Tensor:
+    """The expert MLPs of the local experts and the per-token combine. weigh_input: the routing weights (fp32 [T, k])
+    multiply what the experts read -- the gate and up products, which are linear in it -- and not what they return.
     x [T, hidden]; w13 [num_local, 2*inter, hidden]; w2 [num_local, hidden, inter].
     Returns out [T, hidden]: this rank's partial sum (the full result when it owns every expert)."""
     _need_cuda(x, w13, w2, topk_ids, topk_weights)
@@ -509,23 +513,25 @@ def moe_experts(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, topk_ids: 
         raise ValueError("expert weight shapes do not match")
     if not (w13.is_contiguous() and w2.is_contiguous() and topk_weights.is_contiguous()):
         raise ValueError("expert weights / routing weights must be contiguous")
-    if x.stride(1) != 1 or x.dtype != w13.dtype or x.dtype != w2.dtype or x.dtype != topk_weights.dtype:
+    if x.stride(1) != 1 or x.dtype != w13.dtype or x.dtype != w2.dtype or \
+            topk_weights.dtype != (torch.float32 if weigh_input else x.dtype):
         raise ValueError("x must be row-major and share its dtype with the weights")
     k = plan.top_k
     pairs = T * k
     lib = _C.load()
+    in_w, out_w = (topk_weights, None) if weigh_input else (None, topk_weights)
     if _MOE_BIG_GEMM != "stream" and pairs >= _MOE_BIG_GEMM_ROWS * n_local:
         big = _moe_expert_gemms_umma if _MOE_BIG_GEMM == "umma" else _moe_expert_gemms_library
-        y = big(x, w13, w2, topk_weights, plan)
+        y = big(x, w13, w2, out_w, plan, in_w)
         return _moe_combine(lib, y, topk_ids, plan, T, hidden, out, x)
     h = torch.empty(pairs, inter, dtype=x.dtype, device=x.device)
     y = torch.empty(pairs, hidden, dtype=x.dtype, device=x.device)
     _C.check(lib.b200_moe_gemm_gate_up(h.data_ptr(), x.data_ptr(), w13.data_ptr(), plan.offsets.data_ptr(),
-                                       plan.sorted_pair.data_ptr(), hidden, inter, n_local, k,
+                                       plan.sorted_pair.data_ptr(), _ptr(in_w), hidden, inter, n_local, k,
                                        x.stride(0) if T > 1 else hidden, _dt(x), _stream()),
              "b200_moe_gemm_gate_up")
     _C.check(lib.b200_moe_gemm_down(y.data_ptr(), h.data_ptr(), w2.data_ptr(), plan.offsets.data_ptr(),
-                                    plan.sorted_pair.data_ptr(), topk_weights.data_ptr(), inter, hidden,
+                                    plan.sorted_pair.data_ptr(), _ptr(out_w), inter, hidden,
                                     n_local, k, _dt(x), _stream()), "b200_moe_gemm_down")
     return _moe_combine(lib, y, topk_ids, plan, T, hidden, out, x)
 
@@ -540,7 +546,7 @@ _MOE_BIG_GEMM = "umma"
 _MOE_BIG_GEMM_ROWS = 96
 
 
-def _moe_expert_gemms_umma(x, w13, w2, topk_weights, plan: MoePlan) -> torch.Tensor:
+def _moe_expert_gemms_umma(x, w13, w2, topk_weights, plan: MoePlan, in_weights=None) -> torch.Tensor:
     T, hidden = x.shape
     n_local, two_i, _ = w13.shape
     inter, k = two_i // 2, plan.top_k
@@ -554,11 +560,13 @@ def _moe_expert_gemms_umma(x, w13, w2, topk_weights, plan: MoePlan) -> torch.Ten
                                       x.stride(0) if T > 1 else hidden, _dt(x), _stream()),
              "b200_moe_gather_rows")
     _C.check(lib.b200_moe_gemm_gate_up_umma(h.data_ptr(), xs.data_ptr(), w13.data_ptr(),
-                                            plan.offsets.data_ptr(), pairs, hidden, inter, n_local,
-                                            _dt(x), _stream()), "b200_moe_gemm_gate_up_umma")
+                                            plan.offsets.data_ptr(), plan.sorted_pair.data_ptr(), _ptr(in_weights),
+                                            pairs, hidden, inter, n_local, _dt(x), _stream()),
+             "b200_moe_gemm_gate_up_umma")
     _C.check(lib.b200_moe_gemm_down_umma(y.data_ptr(), h.data_ptr(), w2.data_ptr(), plan.offsets.data_ptr(),
-                                         plan.sorted_pair.data_ptr(), topk_weights.data_ptr(), pairs, inter,
-                                         hidden, n_local, _dt(x), _stream()), "b200_moe_gemm_down_umma")
+                                         plan.sorted_pair.data_ptr() if topk_weights is not None else None,
+                                         _ptr(topk_weights), pairs, inter, hidden, n_local, _dt(x), _stream()),
+             "b200_moe_gemm_down_umma")
     return y
 
 
@@ -652,14 +660,18 @@ def moe_experts_glu_clamped(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor
     return _moe_combine(lib, y, topk_ids, plan, T, hidden, None, x)
 
 
-def _moe_expert_gemms_library(x, w13, w2, topk_weights, plan: MoePlan) -> torch.Tensor:
+def _moe_expert_gemms_library(x, w13, w2, topk_weights, plan: MoePlan, in_weights=None) -> torch.Tensor:
     k = plan.top_k
     pair = plan.sorted_pair.long()                    # tail entries are 0: harmless rows, never combined
     xs = x.index_select(0, pair // k)                 # [pairs, hidden] in expert order
     offs = plan.offsets[1:]
+    if in_weights is not None:
+        xs = (xs * in_weights.reshape(-1)[pair].unsqueeze(1)).to(x.dtype)
     gu = torch._grouped_mm(xs, w13.transpose(1, 2), offs=offs)
     h = silu_and_mul(gu)
     y = torch._grouped_mm(h, w2.transpose(1, 2), offs=offs)
+    if topk_weights is None:
+        return y
     return y * topk_weights.reshape(-1)[pair].unsqueeze(1)      # dtype multiply, as qwen3_moe.py:180-182
 
 
@@ -840,13 +852,13 @@ _ACTS = {"silu": 0, "relu": 1, "gelu_tanh": 2}
 
 
 def act_and_mul(x, act="silu"):
-    """x [rows, 2*inter] = (gate | up) -> act(gate) * up, act in silu | relu | gelu_tanh."""
+    """x [rows, 2*inter] = (gate | up) (a row-strided view allowed) -> act(gate) * up, act in silu | relu | gelu_tanh."""
     _need_cuda(x)
-    if not x.is_contiguous() or x.dim() != 2:
-        raise ValueError("act_and_mul input must be a contiguous matrix")
+    if x.dim() != 2 or x.stride(1) != 1:
+        raise ValueError("act_and_mul input must be a matrix with unit inner stride")
     rows, inter = x.shape[0], x.shape[1] // 2
     out = torch.empty(rows, inter, dtype=x.dtype, device=x.device)
-    _C.check(_C.load().b200_act_and_mul(out.data_ptr(), x.data_ptr(), rows, inter, _ACTS[act], _dt3(x), _stream()),
+    _C.check(_C.load().b200_act_and_mul(out.data_ptr(), x.data_ptr(), x.stride(0) if rows > 1 else x.shape[1], rows, inter, _ACTS[act], _dt3(x), _stream()),
              "b200_act_and_mul")
     return out
 
@@ -971,12 +983,12 @@ def mixed_attn(q, k, v, spans: StepSpans, scale, num_kv_heads, vdim, block_table
 
 
 def attn_generic(q, k, v, spans: StepSpans, scale, num_kv_heads, vdim, block_tables=None, window=0, softcap=0.0,
-                 sink=None, gate=None, keep_first=0):
+                 sink=None, gate=None, keep_first=0, chunk=0):
     """Causal softmax attention for any head sizes and dtypes. q [T, H, dim]; packed mode: k [Tk, G, dim],
     v [Tk, G, vdim] (token-strided views allowed) in the order of spans.cu_k; paged mode (block_tables given):
     k, v are the caches [nb, bs, G*dim], [nb, bs, G*vdim]. Returns [T, H*vdim]. window > 0: position i sees the
-    keys j <= i with i - j < window or j < keep_first. v None: the values are the first vdim columns of the key rows. softcap > 0:
-    scores become softcap * tanh(score / softcap). sink fp32 [H]: exp(sink[h]) joins the softmax denominator (no key,
+    keys j <= i with i - j < window or j < keep_first; chunk > 0 (without a window): those with j // chunk == i // chunk. v
+    None: the values are the first vdim columns of the key rows. softcap > 0: scores become softcap * tanh(score / softcap). sink fp32 [H]: exp(sink[h]) joins the softmax denominator (no key,
     no value). gate [T, H] (q's dtype, row-strided view allowed): head h of token t is multiplied by sigmoid(gate[t, h])."""
     _need_cuda(q, k, v, block_tables, sink, gate)
     _f32(sink)
@@ -1008,7 +1020,7 @@ def attn_generic(q, k, v, spans: StepSpans, scale, num_kv_heads, vdim, block_tab
     _C.check(_C.load().b200_attn_generic(out.data_ptr(), q.data_ptr(), q.stride(0) if T > 1 else H * dim,
                                          k.data_ptr(), ks, _ptr(v), vs, bt_ptr, bt_stride, bs, cu_q, cu_k, ctx,
                                          spans.num_seqs, spans.max_q, H, G, dim, vdim, float(scale), int(window),
-                                         int(keep_first), float(softcap), _ptr(sink), _ptr(gate),
+                                         int(keep_first), int(chunk), float(softcap), _ptr(sink), _ptr(gate),
                                          (gate.stride(0) if T > 1 else H) if gate is not None else 0, _dt3(q),
                                          _stream()), "b200_attn_generic")
     return out
@@ -1076,12 +1088,14 @@ def stream_mix_norm_(x, y, mix, out_w, in_w, w, b, eps, dtype, kind="layer", off
 
 
 def rotary_heads(x, positions, heads, width, dims, base, interleaved, out=None, out_f32=False, split=0,
-                 scale_lo=1.0, scale_hi=1.0):
+                 scale_lo=1.0, scale_hi=1.0, table=None):
     """x [T, heads, width] (a strided view: unit inner stride, any head and token strides). The first `dims` columns
     of every head are rotated by pos * base^(-2i/dims) in pairs (2i, 2i+1) (interleaved) or (i, i + dims/2); heads
     below `split` are then multiplied by scale_lo, the others by scale_hi. out: a view of the same shape (fp32 when
-    out_f32, else x's dtype); by default a new contiguous tensor."""
-    _need_cuda(x, positions, out)
+    out_f32, else x's dtype); by default a new contiguous tensor. table [T, dims/2, 2] (rotary_table): cos and sin are
+    taken from there (base is not used)."""
+    _need_cuda(x, positions, out, table)
+    _rotary_table_check(table, x.shape[0], dims)
     T = x.shape[0]
     if x.dim() != 3 or x.shape[1:] != (heads, width) or x.stride(2) != 1:
         raise ValueError("x must be [T, heads, width] with unit inner stride")
@@ -1093,7 +1107,7 @@ def rotary_heads(x, positions, heads, width, dims, base, interleaved, out=None, 
         raise ValueError("out must be shaped like x, unit inner stride, fp32 or x's dtype")
     _C.check(_C.load().b200_rotary_heads(out.data_ptr(), out.stride(0) if T > 1 else 0, out.stride(1),
                                          1 if out_f32 else 0, x.data_ptr(), x.stride(0) if T > 1 else 0, x.stride(1),
-                                         positions.data_ptr(), T, heads, width, int(dims), float(base),
+                                         positions.data_ptr(), _ptr(table), T, heads, width, int(dims), float(base),
                                          1 if interleaved else 0, int(split), float(scale_lo), float(scale_hi),
                                          _dt3(x), _stream()), "b200_rotary_heads")
     return out
@@ -1162,32 +1176,41 @@ def _fp32_state_rule(mode, q, k, v, g, beta, spans: StepSpans, num_heads, groups
     return out
 
 
-def latent_kv_prep(dq, dkv, wq, wc, positions, rank, rot, dims, base, interleaved, eps, cache=None, slots=None):
+def _rotary_table_check(table, T, dims):
+    if table is not None and (table.dtype != torch.float32 or not table.is_contiguous() or
+                              table.shape != (T, int(dims) // 2, 2)):
+        raise ValueError("table: contiguous fp32 [T, dims/2, 2]")
+
+
+def latent_kv_prep(dq, dkv, wq, wc, positions, rank, rot, dims, base, interleaved, eps, cache=None, slots=None, table=None):
     """dq [T, q_rank], dkv [T, rank + rot] (row-strided views) -> (cq [T, q_rank] = rms(dq) * wq, kc [T, rank + rot] =
     [rms(dkv[:, :rank]) * wc | rotary(dkv[:, rank:])]); kc rows are also stored at `slots` of the paged cache
-    [nb, bs, rank + rot] when given."""
-    _need_cuda(dq, dkv, wq, wc, positions, cache, slots)
+    [nb, bs, rank + rot] when given. dq None: no query latent, cq is None. table as in rotary_heads."""
+    _need_cuda(dq, dkv, wq, wc, positions, cache, slots, table)
     _f32(wq, wc)
-    T, q_rank = dq.shape
-    if dkv.shape != (T, rank + rot) or dq.stride(1) != 1 or dkv.stride(1) != 1 or dq.dtype != dkv.dtype:
+    T = dkv.shape[0]
+    q_rank = dq.shape[1] if dq is not None else 0
+    if dkv.shape != (T, rank + rot) or dkv.stride(1) != 1 or \
+            (dq is not None and (dq.shape[0] != T or dq.stride(1) != 1 or dq.dtype != dkv.dtype)):
         raise ValueError("latent_kv_prep shapes")
+    _rotary_table_check(table, T, dims)
     if positions.dtype != torch.int64 or not positions.is_contiguous():
         raise TypeError("positions must be contiguous int64")
     have = cache is not None and cache.numel() > 0 and slots is not None
     bs = 0
     if have:
         _, bs = _cache_dims(cache, rank + rot)
-        if slots.dtype != torch.int32 or not slots.is_contiguous() or cache.dtype != dq.dtype:
+        if slots.dtype != torch.int32 or not slots.is_contiguous() or cache.dtype != dkv.dtype:
             raise TypeError("slots contiguous int32; cache of the activations' dtype")
-    cq = torch.empty(T, q_rank, dtype=dq.dtype, device=dq.device)
-    kc = torch.empty(T, rank + rot, dtype=dq.dtype, device=dq.device)
+    cq = torch.empty(T, q_rank, dtype=dq.dtype, device=dq.device) if dq is not None else None
+    kc = torch.empty(T, rank + rot, dtype=dkv.dtype, device=dkv.device)
     stride = lambda t: t.stride(0) if T > 1 else t.shape[1]
-    _C.check(_C.load().b200_latent_kv_prep(cq.data_ptr(), kc.data_ptr(), cache.data_ptr() if have else None,
+    _C.check(_C.load().b200_latent_kv_prep(_ptr(cq), kc.data_ptr(), cache.data_ptr() if have else None,
                                            slots.data_ptr() if have else None,
-                                           1 if (have and slots.dim() == 2) else 0, bs, dq.data_ptr(), stride(dq),
-                                           dkv.data_ptr(), stride(dkv), wq.data_ptr(), wc.data_ptr(),
-                                           positions.data_ptr(), T, q_rank, rank, rot, int(dims), float(base),
-                                           1 if interleaved else 0, float(eps), _dt3(dq), _stream()),
+                                           1 if (have and slots.dim() == 2) else 0, bs, _ptr(dq),
+                                           stride(dq) if dq is not None else 0, dkv.data_ptr(), stride(dkv), _ptr(wq),
+                                           wc.data_ptr(), positions.data_ptr(), _ptr(table), T, q_rank, rank, rot, int(dims), float(base),
+                                           1 if interleaved else 0, float(eps), _dt3(dkv), _stream()),
              "b200_latent_kv_prep")
     return cq, kc
 
@@ -1281,9 +1304,10 @@ def glu_clamped(x, alpha, limit):
     return out
 
 
-def moe_route_grouped(router_logits, bias, top_k, groups=1, keep=1, scale=1.0):
+def moe_route_grouped(router_logits, bias, top_k, groups=1, keep=1, scale=1.0, normalize=True):
     """Sigmoid router with a selection bias and group-limited choice. router_logits fp32 [T, E]; bias fp32 [E] or
-    None -> (topk_ids int32 [T, k], topk_weights fp32 [T, k])."""
+    None -> (topk_ids int32 [T, k], topk_weights fp32 [T, k]): the chosen sigmoid scores, divided by their sum
+    (normalize) or as they are, times scale."""
     _need_cuda(router_logits, bias)
     _f32(bias)
     if router_logits.dtype != torch.float32 or router_logits.stride(1) != 1:
@@ -1293,7 +1317,7 @@ def moe_route_grouped(router_logits, bias, top_k, groups=1, keep=1, scale=1.0):
     w = torch.empty(T, top_k, dtype=torch.float32, device=router_logits.device)
     _C.check(_C.load().b200_moe_route_grouped(ids.data_ptr(), w.data_ptr(), router_logits.data_ptr(),
                                               router_logits.stride(0) if T > 1 else E, _ptr(bias), T, E, int(top_k),
-                                              int(groups), int(keep), float(scale), _stream()),
+                                              int(groups), int(keep), float(scale), 1 if normalize else 0, _stream()),
              "b200_moe_route_grouped")
     return ids, w
 
@@ -1331,11 +1355,12 @@ def moe_route_topk(router_logits, bias, top_k):
     return ids, w
 
 
-def moe_experts_generic(x, w13, w2, topk_weights, plan: MoePlan, act=None, glu=None) -> torch.Tensor:
+def moe_experts_generic(x, w13, w2, topk_weights, plan: MoePlan, act=None, glu=None, weigh_input=False) -> torch.Tensor:
     """Expert MLPs and the weighted combine for any sizes and dtypes (fp32 included): x [T, hidden]; w2 [E, hidden,
     inter]; topk_weights fp32 [T, k]. act None: gated experts down(silu(gate x) * up x) with w13 [E, 2*inter, hidden]
     (glu = (alpha, limit): the clamped unit g sigmoid(alpha g) (u + 1) of glu_clamped in place of silu(g) u);
-    act "silu" | "relu" | "gelu_tanh" | "relu2": experts without a gate, down(act(up x)) with w13 [E, inter, hidden]."""
+    act "silu" | "relu" | "gelu_tanh" | "relu2": experts without a gate, down(act(up x)) with w13 [E, inter, hidden].
+    weigh_input (gated experts): the routing weights multiply what the experts read and not what they return."""
     _need_cuda(x, w13, w2, topk_weights)
     _f32(topk_weights)
     T, hidden = x.shape
@@ -1351,21 +1376,22 @@ def moe_experts_generic(x, w13, w2, topk_weights, plan: MoePlan, act=None, glu=N
     y = torch.empty(pairs, hidden, dtype=torch.float32, device=x.device)
     out = torch.empty(T, hidden, dtype=x.dtype, device=x.device)
     _C.check(lib.b200_moe_gemm_generic(h.data_ptr(), x.data_ptr(), x.stride(0) if T > 1 else hidden, w13.data_ptr(),
-                                       plan.offsets.data_ptr(), plan.sorted_pair.data_ptr(), pairs, hidden, inter, E,
+                                       plan.offsets.data_ptr(), plan.sorted_pair.data_ptr(),
+                                       topk_weights.data_ptr() if weigh_input else None, pairs, hidden, inter, E,
                                        k, 1 if act is None else 2 + _PLAIN_ACTS[act], float(glu[0]) if glu else 0.0,
                                        float(glu[1]) if glu else 0.0, _dt3(x), _stream()),
              "b200_moe_gemm_generic (up)")
     _C.check(lib.b200_moe_gemm_generic(y.data_ptr(), h.data_ptr(), inter, w2.data_ptr(), plan.offsets.data_ptr(),
-                                       plan.sorted_pair.data_ptr(), pairs, inter, hidden, E, k, 0, 0.0, 0.0, _dt3(x),
+                                       plan.sorted_pair.data_ptr(), None, pairs, inter, hidden, E, k, 0, 0.0, 0.0, _dt3(x),
                                        _stream()), "b200_moe_gemm_generic (down)")
-    _C.check(lib.b200_moe_combine_weighted(out.data_ptr(), y.data_ptr(), topk_weights.data_ptr(),
+    _C.check(lib.b200_moe_combine_weighted(out.data_ptr(), y.data_ptr(), None if weigh_input else topk_weights.data_ptr(),
                                            plan.pos_of_pair.data_ptr(), T, k, hidden, _dt3(x), _stream()),
              "b200_moe_combine_weighted")
     return out
 
 
 # ---------------------------------------------------------------------------------------------------
-# Scaled residual with a grouped norm, rotary positions from a frequency table fused with value blending and the K/V
+# Scaled residual with a grouped norm, gated residual with a depth average, capped logits, rotary positions from a frequency table fused with value blending and the K/V
 # scatter, and the per-head output gate (csrc/seq_ops.cu).
 def wkv_prep(r, k, z, w0, u, num_heads, dim):
     """r, k [T, H*dim] (row-strided views allowed), z fp32 [T, H*dim]; w0, u fp32 [H*dim] -> (r fp32, k fp32, decay =
@@ -1428,6 +1454,44 @@ def residual_scale_groupnorm_(residual, y, scale, c, w, eps, groups, dtype, offs
                                                      hidden, int(groups), _DT3[dtype], _stream()),
              "b200_residual_scale_groupnorm")
     return h
+
+
+def residual_gate_average(x, y, gate, w, eps, dtype, c=1.0, y_index=None, x_out=None, keep=None, hist=None, n=0, avg=None):
+    """One step of a residual with gated branches whose layers hand on a weighted sum of everything so far:
+    v = (x if x is not None else 0) + c * y * (sigmoid(gate) if gate is not None else 1), kept in `keep` when given; with
+    avg (fp32 [n + 1]): v <- sum_j<n avg[j] hist[j] + avg[n] v; v is written to x_out when given. Returns h = RMS norm of v
+    times w in `dtype`, or None when w is None. x, x_out, keep fp32 [rows, hidden] (x_out may be x, keep an entry of hist
+    not below n), hist fp32 [entries, rows, hidden]; y [rows, hidden] (or with y_index int64 [rows] a table whose rows are
+    looked up) and gate [rows, hidden] (a row-strided view) in `dtype`."""
+    _need_cuda(x, y, gate, w, y_index, x_out, keep, hist, avg)
+    _f32(x, w, x_out, keep, hist, avg)
+    hidden = y.shape[-1]
+    rows = y_index.numel() if y_index is not None else y.shape[0]
+    if not y.is_contiguous() or y.dtype != dtype:
+        raise ValueError("y: contiguous [rows or table, hidden] of the model dtype")
+    if y_index is not None and (y_index.dtype != torch.int64 or not y_index.is_contiguous()):
+        raise TypeError("row indices are contiguous int64 [rows]")
+    if gate is not None and (gate.shape != (rows, hidden) or gate.stride(1) != 1 or gate.dtype != dtype):
+        raise ValueError("gate [rows, hidden] of the model dtype with unit inner stride")
+    if any(t is not None and t.shape != (rows, hidden) for t in (x, x_out, keep)):
+        raise ValueError("x, x_out, keep are [rows, hidden]")
+    if avg is not None and (avg.numel() != n + 1 or (n and (hist is None or hist.shape[0] < n or hist.shape[1:] != (rows, hidden)))):
+        raise ValueError("avg [n + 1] over hist [>= n, rows, hidden]")
+    h = torch.empty(rows, hidden, dtype=dtype, device=y.device) if w is not None else None
+    _C.check(_C.load().b200_residual_gate_average(
+        _ptr(h), _ptr(x), _ptr(x_out), y.data_ptr(), _ptr(y_index), y.shape[0], _ptr(gate),
+        (gate.stride(0) if rows > 1 else hidden) if gate is not None else 0, float(c), _ptr(keep), _ptr(hist),
+        hist.stride(0) if hist is not None else 0, int(n), _ptr(avg), _ptr(w), float(eps), rows, hidden, _DT3[dtype],
+        _stream()), "b200_residual_gate_average")
+    return h
+
+
+def logit_cap_(z, scale, cap=0.0):
+    """z (contiguous fp32, in place) <- cap * tanh(scale * z / cap); cap 0: scale * z."""
+    _need_cuda(z)
+    _f32(z)
+    _C.check(_C.load().b200_logit_cap(z.data_ptr(), z.numel(), float(scale), float(cap), _stream()), "b200_logit_cap")
+    return z
 
 
 def rotary_table(positions, freq, magnitude=1.0):

@@ -572,19 +572,20 @@ def test_moe_entry_points_reject_bad_arguments():
     assert lib.b200_moe_route(one, one, one, 4, 8, 9, 8, 0, None) == -2              # top_k > experts
     assert lib.b200_moe_route(None, one, one, 4, 8, 2, 8, 0, None) == -1
     assert lib.b200_moe_align(one, one, one, one, one, 8, 0, 0, None) == -2
-    assert lib.b200_moe_gemm_gate_up(one, one, one, one, one, 100, 64, 4, 2, 100, 0, None) == -3   # K % 64
-    assert lib.b200_moe_gemm_gate_up(one, one, one, one, one, 128, 96, 4, 2, 128, 0, None) == -3   # inter % 64
+    assert lib.b200_moe_gemm_gate_up(one, one, one, one, one, None, 100, 64, 4, 2, 100, 0, None) == -3   # K % 64
+    assert lib.b200_moe_gemm_gate_up(one, one, one, one, one, None, 128, 96, 4, 2, 128, 0, None) == -3   # inter % 64
     assert lib.b200_moe_gemm_down(one, one, one, one, one, one, 64, 192, 4, 2, 0, None) == -3      # hidden % 128
-    assert lib.b200_moe_gemm_down(one, one, one, one, one, None, 64, 128, 4, 2, 0, None) == -1
+    assert lib.b200_moe_gemm_down(one, one, one, one, None, one, 64, 128, 4, 2, 0, None) == -1
     assert lib.b200_moe_combine(one, one, one, one, 4, 2, 100, 100, 0, None) == -4                 # hidden % 8
     assert lib.b200_moe_combine(one, one, one, one, 0, 2, 128, 128, 0, None) == 0                  # empty batch
     assert lib.b200_sample_shard(one, one, None, 4, 1000, 1000, 2 ** 31 - 500, 0, 0, None, 0, None) == -2   # index overflow
     assert lib.b200_sample_shard(None, one, None, 4, 1000, 1000, 0, 0, 0, None, 0, None) == -1
     # tcgen05 grouped GEMMs (moe_umma.cu)
-    assert lib.b200_moe_gemm_gate_up_umma(one, one, one, one, 256, 100, 64, 4, 0, None) == -3       # K % 64
+    assert lib.b200_moe_gemm_gate_up_umma(one, one, one, one, None, None, 256, 100, 64, 4, 0, None) == -3       # K % 64
+    assert lib.b200_moe_gemm_gate_up_umma(one, one, one, one, None, one, 256, 128, 64, 4, 0, None) == -1       # weights without pairs
     assert lib.b200_moe_gemm_down_umma(one, one, one, one, one, one, 256, 64, 192, 4, 0, None) == -3  # hidden % 128
     assert lib.b200_moe_gemm_down_umma(one, one, one, one, None, one, 256, 64, 128, 4, 0, None) == -1   # scale without pairs
-    assert lib.b200_moe_gemm_gate_up_umma(one, one, one, one, 0, 128, 64, 4, 0, None) == 0          # no pairs
+    assert lib.b200_moe_gemm_gate_up_umma(one, one, one, one, None, None, 0, 128, 64, 4, 0, None) == 0          # no pairs
     assert lib.b200_moe_gather_rows(one, one, one, one, 16, 4, 2, 100, 100, 0, None) == -4          # hidden % 8
 
 

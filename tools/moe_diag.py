@@ -109,7 +109,7 @@ def run_stages(x, w13, w2, ids, w, plan, path, h_override=None):
     h2 = h if h_override is None else h_override.contiguous()
     if path == "stream":
         _C.check(lib.b200_moe_gemm_gate_up(h.data_ptr(), x.data_ptr(), w13.data_ptr(), plan.offsets.data_ptr(),
-                                           plan.sorted_pair.data_ptr(), hidden, inter, n_local, k, x.stride(0),
+                                           plan.sorted_pair.data_ptr(), None, hidden, inter, n_local, k, x.stride(0),
                                            dt, st), "gate_up")
         _C.check(lib.b200_moe_gemm_down(y.data_ptr(), h2.data_ptr(), w2.data_ptr(), plan.offsets.data_ptr(),
                                         plan.sorted_pair.data_ptr(), w.data_ptr(), inter, hidden, n_local, k,
@@ -120,7 +120,7 @@ def run_stages(x, w13, w2, ids, w, plan, path, h_override=None):
                                           plan.sorted_pair.data_ptr(), pairs, n_local, k, hidden, x.stride(0),
                                           dt, st), "gather")
         _C.check(lib.b200_moe_gemm_gate_up_umma(h.data_ptr(), xs.data_ptr(), w13.data_ptr(),
-                                                plan.offsets.data_ptr(), pairs, hidden, inter, n_local, dt, st),
+                                                plan.offsets.data_ptr(), None, None, pairs, hidden, inter, n_local, dt, st),
                  "gate_up_umma")
         _C.check(lib.b200_moe_gemm_down_umma(y.data_ptr(), h2.data_ptr(), w2.data_ptr(), plan.offsets.data_ptr(),
                                              plan.sorted_pair.data_ptr(), w.data_ptr(), pairs, inter, hidden,
