@@ -221,7 +221,7 @@ int b200_prefill_varlen_attn_capped(void* out, const void* q, const void* k, con
                                     int32_t block_size, float scale, float softcap, const float* sink, int32_t dtype,
                                     void* workspace, int64_t workspace_bytes, b200_stream_t stream);
 
-/* The general form: keys of head_dim and values of value_dim (each 64 or 128; out [total_q, num_heads*value_dim], v rows and
+/* The general form: keys of head_dim (64, 128 or 192) and values of value_dim (64 or 128; out [total_q, num_heads*value_dim], v rows and
  * caches value_dim wide per head); window > 0: the query at position i sees keys j <= i with i - j < window or
  * j < keep_first (window 0: every earlier key); chunk > 0 (without a window): those with j / chunk == i / chunk. Served by the tcgen05 kernel only, like the capped form. */
 int b200_prefill_varlen_attn_windowed(void* out, const void* q, const void* k, const void* v,
@@ -668,6 +668,20 @@ int b200_latent_kv_prep(void* cq, void* kc, void* cache, const int32_t* slots, i
                         int64_t dkv_stride, const float* wq, const float* wc, const int64_t* positions,
                         const float* table, int32_t tokens, int32_t q_rank, int32_t rank, int32_t rot, int32_t dims, double base,
                         int32_t interleaved, float eps, int32_t dtype, b200_stream_t stream);
+
+/* Causal softmax attention over latent rows, 16-bit: q [total_q, num_heads, dim]; every head of a token reads the same row
+ * [dim] per key, as key and (its first `rank` columns) as value -> out [total_q, num_heads, rank]. Key rows are packed
+ * (block_tables NULL: in the order of cu_k, k_stride elements apart) or the paged cache [nb, bs, k_stride]. Spans as in
+ * b200_attn_generic (total_q: tokens of the step). window > 0: position i sees the keys j <= i with i - j < window.
+ * dim, rank % 8 == 0, dim <= 576, rank <= 512. splits > 1: the keys of a row tile are split over that many CTAs
+ * (b200_latent_attn_splits) through part_o [total_q * num_heads * splits * rank] and part_ml [.. * 2], fp32. */
+int b200_latent_attn(void* out, const void* q, const void* k, int64_t k_stride, const int32_t* block_tables,
+                     int32_t bt_stride, int32_t block_size, const int32_t* cu_q, const int32_t* cu_k,
+                     const int32_t* ctx_lens, int32_t num_seqs, int32_t max_q, int32_t total_q, int32_t num_heads,
+                     int32_t dim, int32_t rank, float scale, int32_t window, int32_t splits, float* part_o, float* part_ml,
+                     int32_t dtype, b200_stream_t stream);
+/* Key splits for a launch of `ctas` row tiles (rows / 16 or / 32 per sequence) whose sequences have up to max_keys keys. */
+int b200_latent_attn_splits(int64_t ctas, int32_t max_keys);
 
 /* Softmax over a block of fp32 scores s [rows, nk] of `heads` query heads per token. ctx_lens == NULL: the rows
  * are consecutive tokens of one sequence, row r at position first_pos + r / heads, column j the key at position

@@ -326,7 +326,8 @@ extern "C" int b200_prefill_varlen_attn_windowed(void* out, const void* q, const
                      num_kv_heads <= 0,
                  B200_ERR_BAD_SHAPE);
   B200_RETURN_IF(num_heads % num_kv_heads != 0, B200_ERR_BAD_SHAPE);
-  B200_RETURN_IF((head_dim != 64 && head_dim != 128) || (value_dim != 64 && value_dim != 128), B200_ERR_UNSUPPORTED);
+  B200_RETURN_IF((head_dim != 64 && head_dim != 128 && head_dim != 192) || (value_dim != 64 && value_dim != 128),
+                 B200_ERR_UNSUPPORTED);
   B200_RETURN_IF(window < 0 || keep_first < 0 || chunk < 0 || (window > 0 && chunk > 0), B200_ERR_BAD_SHAPE);
   if (num_seqs == 0 || max_seqlen_q == 0) return B200_OK;
   B200_RETURN_IF(!out || !q || !k || !v || !cu_seqlens_q || !cu_seqlens_k, B200_ERR_NULL_POINTER);

@@ -36,7 +36,8 @@
 // visits the tiles of the kept keys, then those from its first row's window on; the tiles between are skipped by
 // index (`kept`, `skip`), the borders are masked element by element. Chunks (chunk > 0: position i sees j <= i of its own
 // chunk) run the same way, with the chunk's start in place of the window's.
-// Keys and values may have different head sizes (DK, DV in {64, 128}); D below stands for the one that applies.
+// Keys and values may have different head sizes (DK in {64, 128, 192}, DV in {64, 128}; 192: one CTA per SM, single-stage
+// rings); D below stands for the one that applies.
 //
 // Split-KV (few, long rows: the prefix-cache-hit form q_len << k_len): when the grid
 // would leave most SMs idle, `kv_splits` CTAs share one (sequence, head, 256 rows), each takes a
@@ -80,11 +81,14 @@ constexpr int kUBM = 128, kUBN = 128;
 // shared memory, 256 TMEM columns, 192 threads -> TWO CTAs per SM: the two chains sharing the tensor pipe
 // are independent CTAs, so one CTA's prologue (barrier init, TMEM alloc, Q load) and epilogue run under
 // the other's main loop and the hardware balances 128-row items.
+// K/V ring depth: QT stages; keys of 192 columns leave shared memory for one
+constexpr int prefill_stages(int dk, int qt) { return dk > 128 ? 1 : qt; }
+
 template <typename T, int DK, int DV, int QT>
-__global__ void __launch_bounds__((4 * QT + 2) * 32, 3 - QT)
+__global__ void __launch_bounds__((4 * QT + 2) * 32, DK > 128 ? 1 : 3 - QT)
 prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                      const __grid_constant__ CUtensorMap tmV, const PrefillUmmaParams p) {
-  constexpr int kUStages = QT;                  // K/V ring depth
+  constexpr int kUStages = prefill_stages(DK, QT);   // K/V ring depth
   constexpr int kTmaWarp = 4 * QT, kMmaWarp = 4 * QT + 1;
   constexpr uint32_t kTmemCols = QT * 256;      // O[t] at 128 t, S[t] at QT * 128 + 128 t
   constexpr uint32_t kSBase = QT * 128;
@@ -473,7 +477,8 @@ static int prefill_umma_launch_t(const CUtensorMap& mq, const CUtensorMap& mk, c
                                  const PrefillUmmaParams& p, int num_seqs, int max_seqlen_q, int total_q,
                                  cudaStream_t stream) {
   constexpr int CHK = DK / 64, CHV = DV / 64;
-  constexpr size_t smem = 1024 + QT * CHK * kUBM * 128 + QT * (CHK + CHV) * kUBN * 128 + 32 * 8 + 16;
+  constexpr size_t smem =
+      1024 + QT * CHK * kUBM * 128 + prefill_stages(DK, QT) * (CHK + CHV) * kUBN * 128 + 32 * 8 + 16;
   auto kern = prefill_umma_kernel<T, DK, DV, QT>;
   static bool attr_set = false;
   if (!attr_set) {
@@ -551,7 +556,9 @@ int prefill_umma_launch(void* out, const void* q, const void* k, const void* v,
   const int span = window > 0 ? window : chunk;
   // keys that a 128-row query tile can see at most: what the choice of layout and of key splits is made on
   if (span > 0 && max_seqlen_k > span + p.keep_first + 3 * kUBM) max_seqlen_k = span + p.keep_first + 3 * kUBM;
-  const int qt = prefill_query_tiles(num_seqs, H, max_seqlen_q, DV, span > 0 ? max_seqlen_k : max_seqlen_q);
+  // one CTA per SM either way with keys of 192 columns: two ping-pong tiles wherever a sequence has them
+  const int qt = DK > 128 ? (max_seqlen_q > kUBM ? 2 : 1)
+                          : prefill_query_tiles(num_seqs, H, max_seqlen_q, DV, span > 0 ? max_seqlen_k : max_seqlen_q);
   p.kv_splits = (workspace != nullptr && (reinterpret_cast<uintptr_t>(workspace) & 15) == 0)
                     ? prefill_kv_splits(num_seqs, H, max_seqlen_q, max_seqlen_k, total_q, DV, workspace_bytes, qt)
                     : 1;
@@ -580,7 +587,8 @@ int prefill_umma_launch(void* out, const void* q, const void* k, const void* v,
   (qt == 2 ? prefill_umma_launch_t<T, K, V, 2>(mq, mk, mv, p, num_seqs, max_seqlen_q, total_q, stream) \
            : prefill_umma_launch_t<T, K, V, 1>(mq, mk, mv, p, num_seqs, max_seqlen_q, total_q, stream))
 #define B200_PREFILL_DISPATCH(T)                                                      \
-  (DK == 128 ? (DV == 128 ? B200_PREFILL_QT(T, 128, 128) : B200_PREFILL_QT(T, 128, 64)) \
+  (DK == 192   ? (DV == 128 ? B200_PREFILL_QT(T, 192, 128) : B200_PREFILL_QT(T, 192, 64)) \
+   : DK == 128 ? (DV == 128 ? B200_PREFILL_QT(T, 128, 128) : B200_PREFILL_QT(T, 128, 64)) \
              : (DV == 128 ? B200_PREFILL_QT(T, 64, 128) : B200_PREFILL_QT(T, 64, 64)))
   return dtype == B200_DTYPE_BF16 ? B200_PREFILL_DISPATCH(__nv_bfloat16) : B200_PREFILL_DISPATCH(__half);
 #undef B200_PREFILL_DISPATCH

@@ -162,6 +162,10 @@ PROTOTYPES = {
     "b200_latent_kv_prep": (c_int32, [c_void_p, c_void_p, c_void_p, c_void_p, c_int32, c_int32, c_void_p, c_int64,
                                       c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_int32, c_int32,
                                       c_int32, c_int32, c_int32, c_double, c_int32, c_float, c_int32, c_void_p]),
+    "b200_latent_attn": (c_int32, [c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_int32, c_int32, c_void_p, c_void_p,
+                                   c_void_p, c_int32, c_int32, c_int32, c_int32, c_int32, c_int32, c_float, c_int32, c_int32,
+                                   c_void_p, c_void_p, c_int32, c_void_p]),
+    "b200_latent_attn_splits": (c_int32, [c_int64, c_int32]),
     "b200_masked_softmax": (c_int32, [c_void_p, c_void_p, c_int64, c_int32, c_int32, c_int32, c_int32, c_int32,
                                       c_float, c_void_p, c_void_p, c_void_p, c_int32, c_int32, c_void_p]),
     "b200_glu_clamped": (c_int32, [c_void_p, c_void_p, c_int32, c_int32, c_float, c_float, c_int32, c_void_p]),

@@ -571,13 +571,27 @@ def prompt_chunk_plan(ctx, paged, device, chunk: int, window: int, min_tokens: i
     return plan
 
 
+def packed_key_slots(ctx, device) -> torch.Tensor:
+    """Cache row of every key of the step's sequences, packed in the order of cu_seqlens_k (int64)."""
+    import numpy as np
+    lens = [kl for _, _, kl in ctx.host_spans]
+    seq = np.repeat(np.arange(len(lens)), lens)
+    pos = np.concatenate([np.arange(n) for n in lens])
+    bs = ctx.block_size
+    dev = lambda a: torch.from_numpy(np.ascontiguousarray(a)).to(torch.int64).to(device, non_blocking=True)
+    blocks = ctx.block_tables.reshape(-1)[dev(seq * ctx.block_tables.shape[1] + pos // bs)]
+    return blocks.long() * bs + dev(pos % bs)
+
+
 class LatentAttention(nn.Module):
     """Softmax attention whose keys and values are up-projections of ONE cached latent row per token:
     score_h(i, j) = scale (q_h^plain . W_uk,h c_j + q_h^rot . r_j), value_h(j) = W_uv,h c_j, with c the normed latent
     [rank] and r the rotated key part [rot] shared by all heads. Only [c | r] is cached (``k_cache`` [nb, bs,
     rank + rot]; there is no value cache). The up-projections are absorbed: the query is moved into latent space
     (q_h^plain W_uk,h, one batched product), attention runs as ONE kv head of key size rank + rot whose values are
-    the first ``rank`` columns of the same rows, and W_uv,h is applied to the attended latent."""
+    the first ``rank`` columns of the same rows, and W_uv,h is applied to the attended latent. Prompt steps of 16-bit models
+    whose sizes fit the tcgen05 prompt kernel up-project instead: one product gives every key and value of the step's
+    sequences (3 to 4 times fewer operations per query and key), see _prefill_up_projected."""
 
     def __init__(self, num_heads: int, dim: int, rot: int, vdim: int, rank: int, scale: float, window: int = 0):
         super().__init__()
@@ -603,13 +617,20 @@ class LatentAttention(nn.Module):
         """q_plain [T, H, dim] (a view); q_rot_writer(out_view [T, H, rot]) fills the rotated query part; kc
         [T, rank + rot] this step's cache rows (used when no cache is bound). Returns [T, H * vdim]."""
         ctx = get_context()
+        if self._up_projects(ctx, q_plain):
+            return self._prefill_up_projected(q_plain, q_rot_writer, kc, ctx)
         T, H, R = q_plain.shape[0], self.num_heads, self.rank
         qx = torch.empty(T, H, R + self.rot, dtype=q_plain.dtype, device=q_plain.device)
         qx[:, :, :R].copy_(torch.bmm(q_plain.transpose(0, 1), self.w_uk).transpose(0, 1))
         q_rot_writer(qx[:, :, R:])
         spans = ops.StepSpans.of(ctx)
         paged = self.k_cache.numel() > 0 and ctx.block_tables is not None
-        if (ctx.is_prefill and ctx.host_spans is not None and qx.dtype != torch.float32 and not self.force_generic
+        own = not self.force_generic and self.OWN_KERNEL and ops.latent_attn_fits(qx, R)
+        if own:
+            lat = ops.latent_attn(qx, self.k_cache if paged else kc, spans, self.scale, R,
+                                  block_tables=ctx.block_tables if paged else None, window=self.window,
+                                  max_keys=ctx.max_seqlen_k if ctx.is_prefill else None)
+        elif (ctx.is_prefill and ctx.host_spans is not None and qx.dtype != torch.float32 and not self.force_generic
                 and ctx.max_seqlen_q >= self.PRODUCT_MIN_TOKENS):
             lat = self._prefill_by_products(qx, kc, ctx, paged)
         elif (not ctx.is_prefill and paged and self.window > 0 and not self.force_generic and
@@ -623,6 +644,58 @@ class LatentAttention(nn.Module):
         out = torch.bmm(lat.view(T, H, R).transpose(0, 1), self.w_uv.transpose(1, 2))      # [H, T, vdim]
         return out.transpose(0, 1).reshape(T, H * self.vdim)
 
+    UP_PROJECT = True             # prompt steps on explicit keys and values where the tcgen05 prompt kernel takes the sizes
+    UP_PROJECT_MIN_TOKENS = 64    # longest portion of a step from which it pays
+    UP_PROJECT_MAX_KEYS = 3       # keys of the step per query token up to which it pays
+
+    def _key_width(self) -> int:
+        return -(-(self.dim + self.rot) // 64) * 64
+
+    def _up_projects(self, ctx, q) -> bool:
+        if not (self.UP_PROJECT and ctx.is_prefill and ctx.host_spans is not None and not self.force_generic and
+                q.dtype != torch.float32 and self.vdim in (64, 128) and self._key_width() <= 192 and
+                (self.rank + self.rot) % 8 == 0 and ctx.max_seqlen_q >= self.UP_PROJECT_MIN_TOKENS):
+            return False
+        keys = sum(kl for _, _, kl in ctx.host_spans)
+        return keys <= self.UP_PROJECT_MAX_KEYS * q.shape[0]
+
+    def _up_matrix(self) -> torch.Tensor:
+        """[H * key width + H * vdim, rank + rot]: what turns a cached row into every head's key [up-projected | rotated part
+        (an identity block) | zeros to the kernel's width] and value. Made once from the two parameters."""
+        key = (self.w_uk._version, self.w_uv._version, self.w_uk.data_ptr(), self.w_uv.data_ptr())
+        if getattr(self, "_up_key", None) != key:
+            H, d, dr, dv, R, Kw = self.num_heads, self.dim, self.rot, self.vdim, self.rank, self._key_width()
+            up = torch.zeros(H * (Kw + dv), R + dr, dtype=self.w_uk.dtype, device=self.w_uk.device)
+            k = up[:H * Kw].view(H, Kw, R + dr)
+            k[:, :d, :R] = self.w_uk
+            k[:, d:d + dr, R:] = torch.eye(dr, dtype=up.dtype, device=up.device)
+            up[H * Kw:, :R] = self.w_uv.reshape(H * dv, R)
+            self._up, self._up_key = up, key
+        return self._up
+
+    def _prefill_up_projected(self, q_plain, q_rot_writer, kc, ctx):
+        """Prompt steps: the cached rows of the step's sequences (this step's own rows when no sequence has a past) times
+        _up_matrix give packed keys and values, and attention runs per head on the tcgen05 prompt kernel."""
+        T, H, d, dr, dv, Kw = q_plain.shape[0], self.num_heads, self.dim, self.rot, self.vdim, self._key_width()
+        D = self.rank + dr
+        rows = kc
+        if any(kl != ql for _, ql, kl in ctx.host_spans):
+            slots = ctx.scratch.get("packed key slots")
+            if slots is None:
+                slots = ctx.scratch["packed key slots"] = packed_key_slots(ctx, kc.device)
+            rows = ops.gather_rows_by_head(self.k_cache.view(-1, 1, D), slots, 1, slots.numel()).view(-1, D)
+        q = torch.empty(T, H, Kw, dtype=q_plain.dtype, device=q_plain.device)
+        q[:, :, :d].copy_(q_plain)
+        q_rot_writer(q[:, :, d:d + dr])
+        if d + dr < Kw:
+            q[:, :, d + dr:].zero_()
+        kv = torch.nn.functional.linear(rows, self._up_matrix())
+        k = kv[:, :H * Kw].unflatten(1, (H, Kw))
+        v = kv[:, H * Kw:].unflatten(1, (H, dv))
+        return ops.prefill_varlen_attn(q, k, v, ctx.cu_seqlens_q, ctx.cu_seqlens_k, ctx.max_seqlen_q, ctx.max_seqlen_k,
+                                       self.scale, H, vdim=dv, window=self.window)
+
+    OWN_KERNEL = True             # csrc/latent_attn.cu where it takes the sizes
     DECODE_WINDOW_MAX = 4096      # decode steps gather a window of at most this many rows per sequence
 
     def _decode_window_by_products(self, qx, ctx):

@@ -1215,6 +1215,56 @@ def latent_kv_prep(dq, dkv, wq, wc, positions, rank, rot, dims, base, interleave
     return cq, kc
 
 
+LATENT_MAX_DIM, LATENT_MAX_RANK = 576, 512
+
+
+def latent_attn_fits(q, rank):
+    """Does latent_attn serve these query rows [T, H, D] (16-bit, sizes in multiples of 8 inside its limits)?"""
+    D = q.shape[-1]
+    return q.dtype != torch.float32 and D % 8 == 0 and rank % 8 == 0 and D <= LATENT_MAX_DIM and rank <= LATENT_MAX_RANK
+
+
+def latent_attn(q, k, spans: StepSpans, scale, rank, block_tables=None, window=0, max_keys=None, splits=None):
+    """Causal softmax attention over latent rows (csrc/latent_attn.cu), 16-bit: q [T, H, D] contiguous; every head of a
+    token reads the same row of D columns per key, as key and (its first `rank` columns) as value. k: this step's rows
+    [Tk, D] (packed, row-strided view allowed), or with block_tables the cache [nb, bs, D]. Returns [T, H*rank]. window as
+    in attn_generic. max_keys: an upper bound of the keys per sequence (default: what the table holds, or Tk); splits: CTAs
+    that share one row tile's keys (default: chosen from the launch's size)."""
+    _need_cuda(q, k, block_tables)
+    T, H, D = q.shape
+    if not q.is_contiguous() or k.dtype != q.dtype or k.stride(-1) != 1:
+        raise ValueError("q contiguous [T, H, D]; key rows of q's dtype with unit inner stride")
+    lib = _C.load()
+    if block_tables is not None:
+        if block_tables.dtype != torch.int32 or block_tables.stride(1) != 1:
+            raise TypeError("block_tables must be row-major int32")
+        _, bs = _cache_dims(k, D)
+        ks, bt_ptr, bt_stride = D, block_tables.data_ptr(), block_tables.stride(0)
+        most = block_tables.shape[1] * bs
+    else:
+        if k.shape[-1] != D:
+            raise ValueError("key rows must have q's width")
+        bs, bt_ptr, bt_stride = 0, None, 0
+        ks = k.stride(0) if k.shape[0] > 1 else D
+        most = k.shape[0]
+    keys = min(most, int(max_keys)) if max_keys is not None else most
+    if window:
+        keys = min(keys, window + 64)
+    if splits is None:
+        rows = spans.max_q * H
+        splits = lib.b200_latent_attn_splits((-(-rows // 32) if rows > 16 else 1) * spans.num_seqs, keys)
+    out = torch.empty(T, H * rank, dtype=q.dtype, device=q.device)
+    part_o = part_ml = None
+    if splits > 1:
+        part_o = torch.empty(T * H * splits * rank, dtype=torch.float32, device=q.device)
+        part_ml = torch.empty(T * H * splits * 2, dtype=torch.float32, device=q.device)
+    cu_q, cu_k, ctx = spans.ptrs()
+    _C.check(lib.b200_latent_attn(out.data_ptr(), q.data_ptr(), k.data_ptr(), ks, bt_ptr, bt_stride, bs, cu_q, cu_k, ctx,
+                                  spans.num_seqs, spans.max_q, T, H, D, int(rank), float(scale), int(window), int(splits),
+                                  _ptr(part_o), _ptr(part_ml), _dt(q), _stream()), "b200_latent_attn")
+    return out
+
+
 def masked_softmax(scores, heads, first_pos, key_lo, scale, window, dtype, ctx_lens=None, chunks=None):
     """scores fp32 [rows, nk] of `heads` query heads per token -> softmax(scale * scores) over the visible keys in
     `dtype`, hidden keys 0. Without ctx_lens / chunks the rows are consecutive tokens of one sequence (row r at position
