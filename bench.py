@@ -27,7 +27,8 @@ the all-reduce form and its latency, and the same workload at TP=1 (rank 0) for 
 `--hybrid --design nirelix` does the same for the Nirelix decoder beside the Zegopel decoder of the same width, and
 `--hybrid --design fitevik` for the Fitevik decoder beside the Nirelix decoder of the same width, and
 `--hybrid --design nurilorn` for the Nurilorn decoder beside the Zegopel decoder of the same width, and
-`--hybrid --design pofazen` for the Pofazen decoder beside the Nirelix decoder of the same width.
+`--hybrid --design pofazen` for the Pofazen decoder beside the Nirelix decoder of the same width, and
+`--hybrid --design ragilorn` for the Ragilorn decoder beside the Nurilorn decoder of the same width.
 """
 from __future__ import annotations
 
@@ -116,8 +117,9 @@ def parse_args():
                          "nirelix: nirelix-1k:zegopel-1k,nirelix-2k:zegopel-2k; with --design fitevik: "
                          "fitevik-1k:nirelix-1k,fitevik-2k:nirelix-2k; with --design nurilorn: "
                          "nurilorn-1k:zegopel-1k,nurilorn-2k:zegopel-2k; with --design pofazen: "
-                         "pofazen-1k:nirelix-1k,pofazen-2k:nirelix-2k)")
-    ap.add_argument("--design", default="zegopel", choices=["zegopel", "nirelix", "fitevik", "nurilorn", "pofazen"],
+                         "pofazen-1k:nirelix-1k,pofazen-2k:nirelix-2k; with --design ragilorn: "
+                         "ragilorn-1k:nurilorn-1k,ragilorn-2k:nurilorn-2k)")
+    ap.add_argument("--design", default="zegopel", choices=["zegopel", "nirelix", "fitevik", "nurilorn", "pofazen", "ragilorn"],
                     help="with --hybrid: whose presets and kernel table are measured")
     ap.add_argument("--kv-cache-dtype", default="auto", choices=["auto", "fp8"],
                     help="fp8: e4m3 KV cache (an extra line; the contract line is the default bf16 cache)")
@@ -1336,6 +1338,182 @@ def pofazen_kernel_table(width, head_dim, tokens, seqs, peak_gbs):
     return rows
 
 
+def ragilorn_kernel_table(width, head_dim, tokens, seqs, peak_gbs):
+    """The kernels that the Ragilorn decoder adds or extends, alone, at the layer sizes of a `width`-wide model, as a
+    prompt step (`seqs` x tokens/seqs) and as a decode step (`seqs` rows at that context), each beside the like kernel of
+    the Nurilorn, Nirelix or Pofazen decoder. frac = algorithmic bytes / time / measured copy bandwidth."""
+    from nanovllm import ops
+    from nanovllm.layers.moe import GroupedSigmoidMoe
+    from nanovllm.layers.seq_mixers import BandScaledRotary, LatentAttention
+    from nanovllm.utils.context import get_context, reset_context, set_context
+    dev, bf = "cuda", torch.bfloat16
+    g = torch.Generator(device=dev).manual_seed(0)
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    rnd = lambda *shape: torch.randn(*shape, device=dev, generator=g)
+    H = width // head_dim
+    G = max(1, H // 4)
+    rows = []
+
+    def add(name, step, fn, nbytes, like=None, like_fn=None, like_bytes=None, flops=None, like_flops=None):
+        t = _timed(fn, flush)
+        row = {"kernel": name, "step": step, "us": round(t * 1e6, 1), "GB/s": round(nbytes / t / 1e9),
+               "frac_of_measured_copy": round(nbytes / t / 1e9 / peak_gbs, 3)}
+        if flops:
+            row["TFLOP/s"] = round(flops / t / 1e12, 2)
+        if like_fn is not None:
+            tl = _timed(like_fn, flush)
+            row["like"] = {"kernel": like, "us": round(tl * 1e6, 1),
+                           "frac_of_measured_copy": round(like_bytes / tl / 1e9 / peak_gbs, 3)}
+            if like_flops:
+                row["like"]["TFLOP/s"] = round(like_flops / tl / 1e12, 2)
+            row["times_as_far_from_roofline_as_like"] = round((like_bytes / tl) / (nbytes / t), 2)
+            if flops and like_flops:
+                row["times_as_far_from_flop_roofline_as_like"] = round((like_flops / tl) / (flops / t), 2)
+        rows.append(row)
+
+    stretch = {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}
+    rot = BandScaledRotary(head_dim // 2, 1e6, True, stretch)
+    chunk = window = 512
+    for step, T in (("prompt", tokens), ("decode", seqs)):
+        per = T // seqs if step == "prompt" else 1
+        ctx = tokens // seqs
+        if step == "prompt":
+            cu = torch.arange(0, T + 1, per, dtype=torch.int32, device=dev)
+            spans = ops.StepSpans(cu, cu, None, per)
+        else:
+            spans = ops.StepSpans(None, None, torch.full((T,), ctx, dtype=torch.int32, device=dev))
+        # residual path: gated branch + norm, and with the average over the depth (like: scaled branch + grouped norm)
+        y, res, gate = rnd(T, width).to(bf), rnd(T, width), rnd(T, 2 * width).to(bf)[:, width:]
+        ls, w1 = rnd(width), rnd(width) * 0.1
+        like = ("residual_scale_groupnorm", lambda: ops.residual_scale_groupnorm_(res, y, ls, 0.5, w1, 1e-6, 4, bf),
+                T * width * 12)
+        add("residual_gate_average, inside a layer", step,
+            lambda: ops.residual_gate_average(res, y, gate, w1, 1e-6, bf, x_out=res), T * width * 14, *like)
+        n = 14                                                       # half-way down a 28-layer stack
+        hist, avg = rnd(n + 1, T, width), rnd(n + 1) * 0.1
+        add(f"residual_gate_average, average over {n} earlier entries", step,
+            lambda: ops.residual_gate_average(res, y, gate, w1, 1e-6, bf, x_out=res, keep=hist[n], hist=hist, n=n, avg=avg),
+            T * width * (18 + 4 * n), *like)
+        del hist
+        emb = rnd(32768, width).to(bf)
+        ids = torch.randint(0, 32768, (T,), device=dev, generator=g)
+        add("residual_gate_average, embedding looked up", step,
+            lambda: ops.residual_gate_average(None, emb, None, w1, 1e-6, bf, c=32.0, y_index=ids, keep=res), T * width * 8,
+            "residual_scale_groupnorm, embedding looked up",
+            lambda: ops.residual_scale_groupnorm_(res, emb, None, 32.0, w1, 1e-6, 4, bf, accumulate=False, y_index=ids),
+            T * width * 8)
+        ff = 3 * width
+        gu = rnd(T, 2 * ff + width).to(bf)
+        add("act_and_mul(silu), inside a wider row", step, lambda: ops.act_and_mul(gu[:, :2 * ff], "silu"), T * ff * 6,
+            "glu_clamped", lambda: ops.glu_clamped(gu.view(-1)[:T * 2 * ff].view(T, 2 * ff), 1.702, 7.0), T * ff * 6)
+        # mixer preparation
+        nq, nk = H * head_dim, G * head_dim
+        pos = torch.arange(T, device=dev) % max(per, 1) + (0 if step == "prompt" else ctx - 1)
+        tab = ops.rotary_table(pos, rot.freq.to(dev), rot.magnitude)
+        nb = (T + 15) // 16 + 1
+        kc = torch.zeros(nb, 16, nk, dtype=bf, device=dev)
+        vc = torch.zeros(nb, 16, nk, dtype=bf, device=dev)
+        sl = torch.arange(T, dtype=torch.int32, device=dev)
+        qkv, other, lam = rnd(T, nq + 2 * nk).to(bf), rnd(T, nk).to(bf), torch.full((1,), 0.4, device=dev)
+        prep_bytes = T * (2 * (nq // 2 + nk) * 2 + nk * 2 + 2 * nk * 2 + rot.dims * 4)
+        add("rope_mix_cache, values as they are", step,
+            lambda: ops.rope_mix_cache(qkv, tab, H, G, head_dim, head_dim, rot.dims, True, None, None, kc, vc, sl), prep_bytes,
+            "rope_mix_cache, values blended",
+            lambda: ops.rope_mix_cache(qkv, tab, H, G, head_dim, head_dim, rot.dims, True, other, lam, kc, vc, sl),
+            prep_bytes + T * nk * 4)
+        R, dr, Q = 4 * head_dim, head_dim // 2, 3 * width // 4
+        lat, wq, wc = rnd(T, Q + R + dr).to(bf), rnd(Q), rnd(R)
+        cache_new = torch.zeros(nb, 16, R + dr, dtype=bf, device=dev)
+        add("latent_kv_prep, no query latent, rotation by table", step,
+            lambda: ops.latent_kv_prep(None, lat[:, Q:], None, wc, pos, R, dr, dr, 1.0, True, 1e-6, cache_new, sl, table=tab),
+            T * ((R + dr) * 6 + dr * 4), "latent_kv_prep",
+            lambda: ops.latent_kv_prep(lat[:, :Q], lat[:, Q:], wq, wc, pos, R, dr, dr, 1e4, True, 1e-6, cache_new, sl),
+            T * (Q * 4 + (R + dr) * 6))
+        qp = rnd(T, H, head_dim + dr).to(bf)
+        qo = torch.empty(T, H, R + dr, dtype=bf, device=dev)
+        add("rotary_heads by table", step,
+            lambda: ops.rotary_heads(qp[:, :, head_dim:], pos, H, dr, dr, 1.0, True, out=qo[:, :, R:], table=tab),
+            T * (H * dr * 4 + dr * 4), "rotary_heads",
+            lambda: ops.rotary_heads(qp[:, :, head_dim:], pos, H, dr, dr, 1e4, True, out=qo[:, :, R:]), T * H * dr * 4)
+        # attention inside chunks (like: inside a window of the same size)
+        bs = 64
+        per_seq = -(-ctx // bs)
+        nblk = seqs * per_seq
+        kcache, vcache = rnd(nblk + 1, bs, nk).to(bf), rnd(nblk + 1, bs, nk).to(bf)
+        tables = torch.randperm(nblk, device=dev, generator=g).to(torch.int32).view(seqs, per_seq)
+        qh = (rnd(T, H, head_dim) * 0.5).to(bf)
+        scale = head_dim ** -0.5
+        if step == "prompt":
+            seen = {"chunk": sum(i % chunk + 1 for i in range(per)) * seqs, "window": sum(min(window, i + 1) for i in range(per)) * seqs}
+            fast = lambda **kw: ops.prefill_varlen_attn(qh, kcache, vcache, spans.cu_q, spans.cu_k, per, per, scale, G,
+                                                        block_tables=tables, **kw)
+            name, keys = "prefill_varlen_attn (tcgen05)", ctx
+        else:
+            seen = {"chunk": T * ((ctx - 1) % chunk + 1), "window": T * min(window, ctx)}
+            fast = lambda **kw: ops.paged_decode_attn(qh, kcache, vcache, tables, spans.ctx_lens, scale, G, **kw)
+            name, keys = "paged_decode_attn", min(window, ctx)
+        att_bytes = T * 2 * nq * 2 + seqs * keys * 2 * nk * 2
+        add(name + f", chunks of {chunk}", step, lambda: fast(chunk=chunk), att_bytes, name + f", window {window}",
+            lambda: fast(window=window), att_bytes, flops=4.0 * seen["chunk"] * nq, like_flops=4.0 * seen["window"] * nq)
+        add(name + ", plain", step, lambda: fast(), T * 2 * nq * 2 + seqs * ctx * 2 * nk * 2,
+            flops=4.0 * (seqs * per * (per + 1) / 2 if step == "prompt" else T * ctx) * nq)
+        # latent attention without a window (like: the windowed form of the Nirelix decoder as composed products)
+        cache = (rnd(nblk + 1, bs, R + dr) * 0.3).to(bf)
+        ours = LatentAttention(H, head_dim, dr, head_dim, R, 0.07)
+        theirs = LatentAttention(H, head_dim, dr, head_dim, R, 0.07, window=window)
+        for m_ in (ours, theirs):
+            m_.w_uk.data, m_.w_uv.data = (rnd(H, head_dim, R) * 0.05).to(bf), (rnd(H, head_dim, R) * 0.05).to(bf)
+            m_.k_cache = cache
+        qx = (rnd(T, H, R + dr) * 0.3).to(bf)
+        new = (rnd(T, R + dr) * 0.3).to(bf)
+        if step == "prompt":
+            set_context(True, cu_seqlens_q=spans.cu_q, cu_seqlens_k=spans.cu_k, max_seqlen_q=per, max_seqlen_k=per,
+                        block_tables=tables, block_size=bs, host_spans=[(i * per, per, per) for i in range(seqs)])
+            pairs = seqs * per * (per + 1) / 2
+            mine = lambda: ours._prefill_up_projected(qp[:, :, :head_dim], lambda out: out.copy_(qp[:, :, head_dim:]), new,
+                                                      get_context())
+            products = lambda: theirs._prefill_by_products(qx, None, get_context(), True)
+            mine_name = "latent attention, up-projected (product + tcgen05)"
+        else:
+            set_context(False, context_lens=spans.ctx_lens, block_tables=tables, block_size=bs)
+            pairs = T * ctx
+            mine = lambda: ops.latent_attn(qx, cache, spans, 0.07, R, block_tables=tables)
+            products = lambda: theirs._decode_window_by_products(qx, get_context())
+            mine_name = "latent_attn, all keys"
+        lat_bytes = lambda keys: T * H * (R + dr + R) * 2 + seqs * keys * (R + dr) * 2
+        per_pair = 2.0 * H * (2 * R + dr)                            # as absorbed: what a (query, key) pair costs either form
+        with torch.inference_mode():
+            add(mine_name, step, mine, lat_bytes(ctx), "latent attention by products (window 512)", products,
+                lat_bytes(ctx if step == "prompt" else min(window, ctx)), flops=pairs * per_pair, like_flops=seen["window"] * per_pair)
+            if step == "prompt":
+                add("latent_attn, all keys (short portions)", step,
+                    lambda: ops.latent_attn(qx, cache, spans, 0.07, R, block_tables=tables, max_keys=per), lat_bytes(ctx),
+                    flops=pairs * per_pair)
+        reset_context()
+        # mixture of experts: scores as they are, weighted at the input (like: normalised, weighted at the output)
+        E, top, ffe = 16, 2, width // 2
+        x, logits, corr = rnd(T, width).to(bf), rnd(T, E), rnd(E) * 0.1
+        add("moe_route_grouped, scores as they are", step, lambda: ops.moe_route_grouped(logits, None, top, normalize=False),
+            T * (E * 4 + top * 8), "moe_route_grouped", lambda: ops.moe_route_grouped(logits, corr, top, 4, 2, 1.5),
+            T * (E * 4 + top * 8))
+        with torch.device(dev):
+            ours_moe = GroupedSigmoidMoe(width, ffe, E, top, correction=False, normalize=False, weigh="input").to(bf)
+            theirs_moe = GroupedSigmoidMoe(width, ffe, E, top, 4, 2, 1.5).to(bf)
+        for m_ in (ours_moe, theirs_moe):
+            for p_ in m_.parameters():
+                p_.data.copy_((torch.randn(p_.shape, device=dev, generator=g) * 0.03).to(p_.dtype))
+            m_.router.data = m_.router.data.float()
+        theirs_moe.correction.data = theirs_moe.correction.data.float()
+        moe_bytes = 3 * E * ffe * width * 2 + T * width * 4
+        with torch.inference_mode():
+            add("mixture weighted at the experts' input", step, lambda: ours_moe(x), moe_bytes,
+                "mixture weighted at the experts' output", lambda: theirs_moe(x), moe_bytes,
+                flops=6.0 * T * top * ffe * width, like_flops=6.0 * T * top * ffe * width)
+        z = rnd(seqs, 131072)
+        add("logit_cap (131072 columns per sequence)", step, lambda: ops.logit_cap_(z, 0.25, 30.0), z.numel() * 8)
+    return rows
+
+
 def hybrid_compare(args):
     """--hybrid: the Zegopel presets beside the dense presets of the same width and depth, each through the engine
     (LLM.add_request / LLM.step; prompt steps, then CUDA-graph decode steps), plus the kernel table."""
@@ -1352,7 +1530,8 @@ def hybrid_compare(args):
     pairs = args.hybrid_pairs or {"nirelix": "nirelix-1k:zegopel-1k,nirelix-2k:zegopel-2k",
                                   "fitevik": "fitevik-1k:nirelix-1k,fitevik-2k:nirelix-2k",
                                   "nurilorn": "nurilorn-1k:zegopel-1k,nurilorn-2k:zegopel-2k",
-                                  "pofazen": "pofazen-1k:nirelix-1k,pofazen-2k:nirelix-2k"}.get(
+                                  "pofazen": "pofazen-1k:nirelix-1k,pofazen-2k:nirelix-2k",
+                                  "ragilorn": "ragilorn-1k:nurilorn-1k,ragilorn-2k:nurilorn-2k"}.get(
         args.design, "zegopel-1k:qwen3-0.6b,zegopel-2k:llama-3.2-1b")
     out["design"] = args.design
     for pair in pairs.split(","):
@@ -1375,7 +1554,8 @@ def hybrid_compare(args):
             del llm
             torch.cuda.empty_cache()
     table = {"nirelix": nirelix_kernel_table, "fitevik": fitevik_kernel_table,
-             "nurilorn": nurilorn_kernel_table, "pofazen": pofazen_kernel_table}.get(args.design, hybrid_kernel_table)
+             "nurilorn": nurilorn_kernel_table, "pofazen": pofazen_kernel_table,
+             "ragilorn": ragilorn_kernel_table}.get(args.design, hybrid_kernel_table)
     out["kernels"] = {"width_1024_head_128": table(1024, 128, 16384, 16, peak),
                       "width_2048_head_64": table(2048, 64, 16384, 16, peak)}
     out["clocks"] = clocks.stop()
