@@ -221,9 +221,10 @@ int b200_prefill_varlen_attn_capped(void* out, const void* q, const void* k, con
                                     int32_t block_size, float scale, float softcap, const float* sink, int32_t dtype,
                                     void* workspace, int64_t workspace_bytes, b200_stream_t stream);
 
-/* The general form: keys of head_dim (64, 128 or 192) and values of value_dim (64 or 128; out [total_q, num_heads*value_dim], v rows and
- * caches value_dim wide per head); window > 0: the query at position i sees keys j <= i with i - j < window or
- * j < keep_first (window 0: every earlier key); chunk > 0 (without a window): those with j / chunk == i / chunk. Served by the tcgen05 kernel only, like the capped form. */
+/* The general form: keys of head_dim (64, 128 or 192) and values of value_dim (64 or 128; out [total_q,
+ * num_heads*value_dim], v rows and caches value_dim wide per head); window > 0: the query at position i sees keys j
+ * <= i with i - j < window or j < keep_first (window 0: every earlier key); chunk > 0 (without a window): those with
+ * j / chunk == i / chunk. Served by the tcgen05 kernel only, like the capped form. */
 int b200_prefill_varlen_attn_windowed(void* out, const void* q, const void* k, const void* v,
                                       const int32_t* cu_seqlens_q, const int32_t* cu_seqlens_k, int32_t num_seqs,
                                       int32_t total_q, int32_t total_k, int32_t max_seqlen_q, int32_t max_seqlen_k,
@@ -378,8 +379,8 @@ int b200_moe_gather_rows(void* xs, const void* x, const int32_t* offsets, const 
                          int32_t pairs, int32_t num_local, int32_t top_k, int32_t hidden,
                          int64_t x_stride, int32_t dtype, b200_stream_t stream);
 int b200_moe_gemm_gate_up_umma(void* h, const void* xs, const void* w13, const int32_t* offsets,
-                               const int32_t* sorted_pair, const float* in_scale, int32_t pairs, int32_t hidden, int32_t inter, int32_t num_local,
-                               int32_t dtype, b200_stream_t stream);
+                               const int32_t* sorted_pair, const float* in_scale, int32_t pairs, int32_t hidden, int32_t inter,
+                               int32_t num_local, int32_t dtype, b200_stream_t stream);
 int b200_moe_gemm_down_umma(void* y, const void* h, const void* w2, const int32_t* offsets,
                             const int32_t* sorted_pair, const void* topk_weights, int32_t pairs,
                             int32_t inter, int32_t hidden, int32_t num_local, int32_t dtype,
@@ -660,9 +661,10 @@ int b200_wkv_prep(float* r_out, float* k_out, float* decay, float* bonus, const 
                   const void* k, int64_t k_stride, const float* z, const float* w0, const float* u, int32_t tokens,
                   int32_t num_heads, int32_t dim, int32_t dtype, b200_stream_t stream);
 
-/* Latent attention, per token: cq [T, q_rank] = rms(dq) * wq (dq NULL: no query latent); row = [rms(dkv[:rank]) * wc | rotary(dkv[rank:])]
- * (rot columns, the first `dims` rotated) written to kc [T, rank + rot] (optional) and to the paged cache
- * [nb, bs, rank + rot] at `slots` (flat, or (block, offset) pairs; optional). table as in b200_rotary_heads. */
+/* Latent attention, per token: cq [T, q_rank] = rms(dq) * wq (dq NULL: no query latent); row = [rms(dkv[:rank]) * wc
+ * | rotary(dkv[rank:])] (rot columns, the first `dims` rotated) written to kc [T, rank + rot] (optional) and to the
+ * paged cache [nb, bs, rank + rot] at `slots` (flat, or (block, offset) pairs; optional). table as in
+ * b200_rotary_heads. */
 int b200_latent_kv_prep(void* cq, void* kc, void* cache, const int32_t* slots, int32_t slot_pairs,
                         int32_t block_size, const void* dq, int64_t dq_stride, const void* dkv,
                         int64_t dkv_stride, const float* wq, const float* wc, const int64_t* positions,

@@ -22,7 +22,8 @@
 //    the whole group shares a single read of the KV bytes. fp32 online softmax in the exp2
 //    domain; running max/sum per thread, reduced with warp shuffles.
 //  * Optional sliding window with kept first tokens, or chunks (a row sees its own chunk, a window of its own length): the
-//    work list of a row holds only the tiles that have a visible key (tile_list), borders are masked element by element. Keys and values may have different head sizes (DK, DV).
+//    work list of a row holds only the tiles that have a visible key (tile_list), borders are masked element by
+//    element. Keys and values may have different head sizes (DK, DV).
 //  Algorithmic bytes per launch: sum_b ctx_b * 2 * Hkv * D * 2 B (+ q, out: negligible).
 #include "decode_common.cuh"
 

@@ -5,8 +5,8 @@
 //                       h = norm(u): the "residual add + next pre-norm" of a multi-stream residual in ONE launch.
 //                       norm is a layer norm with weight and bias, or an RMS norm with a (offset + w) weight.
 //   rotary_heads        rotary positions on the first `dims` columns of every head (pairs (2i, 2i+1) or
-//                       (i, i + dims/2); angles from a base, or a table of cos and sin), a scale per head range, output in fp32 or the element type, with free
-//                       input/output head strides (so that a rotated part can be written into a wider head).
+//                       (i, i + dims/2); angles from a base, or a table of cos and sin), a scale per head range, output
+//                       in fp32 or the element type, with free input/output head strides (so that a rotated part can be written into a wider head).
 //   delta_prep          what a gated delta rule reads besides v: q and k as fp32 unit vectors (q scaled), the decay
 //                       exp(-exp(A) softplus(a + bias)) per key channel or per head, and beta = sigmoid(b), all fp32.
 //   wkv_prep            what a wkv recurrence reads besides v: the receptance and k in fp32, the decay exp(-exp(z + w0))
@@ -353,15 +353,16 @@ wkv_prep_kernel(float* __restrict__ r_out, float* __restrict__ k_out, float* __r
 }
 
 // ------------------------------------------------------------------ latents of a latent attention
-// One CTA per token. cq = rms(dq) * wq (element type; skipped without dq); row = [rms(c) * wc | rotate(kr)] (element type) into `kc`
-// (packed, [tokens, rank + rot]) and, when slots are given, into the paged cache row of the token.
+// One CTA per token. cq = rms(dq) * wq (element type; skipped without dq); row = [rms(c) * wc | rotate(kr)] (element
+// type) into `kc` (packed, [tokens, rank + rot]) and, when slots are given, into the paged cache row of the token.
 template <typename T>
 __global__ void __launch_bounds__(128)
 latent_kv_prep_kernel(T* __restrict__ cq, T* __restrict__ kc, T* __restrict__ cache, const int* __restrict__ slots,
                       int slot_pairs, int block_size, const T* __restrict__ dq, int64_t dq_stride,
                       const T* __restrict__ dkv, int64_t dkv_stride, const float* __restrict__ wq,
                       const float* __restrict__ wc, const int64_t* __restrict__ positions,
-                      const float2* __restrict__ table, int q_rank, int rank, int rot, int dims, int interleaved, double log2_base, float eps) {
+                      const float2* __restrict__ table, int q_rank, int rank, int rot, int dims, int interleaved,
+                      double log2_base, float eps) {
   __shared__ float red[32];
   pdl_wait();
   const int64_t t = blockIdx.x;
@@ -768,7 +769,8 @@ extern "C" int b200_latent_kv_prep(void* cq, void* kc, void* cache, const int32_
   B200_DISPATCH_3(dtype, T, launch_pdl(latent_kv_prep_kernel<T>, dim3(tokens), dim3(128), 0, (cudaStream_t)stream,
                                        (T*)cq, (T*)kc, (T*)cache, slots, slot_pairs, block_size, (const T*)dq,
                                        dq_stride, (const T*)dkv, dkv_stride, wq, wc, positions,
-                                       reinterpret_cast<const float2*>(table), q_rank, rank, rot, dims, interleaved, log2(base), eps));
+                                       reinterpret_cast<const float2*>(table), q_rank, rank, rot, dims, interleaved,
+                                       log2(base), eps));
   return finish_launch();
 }
 

@@ -5,7 +5,8 @@ for the current token), the mixes of a token with the token before that the wkv 
 rotary positions on part of a head (plain, or with frequencies stretched by a ramp between a fast and a slow band or
 between a short and a long wavelength), causal softmax attention whose key and value sizes may differ (optionally inside
 a sliding window with first tokens that stay visible or inside chunks, with capped scores, a sink in the denominator and a gate per
-head), attention whose heads are mixed before the softmax (with a distance bias, a sink, and keys and values that may be another layer's), attention over a cached latent, and the mixing weights of a residual that is
+head), attention whose heads are mixed before the softmax (with a distance bias, a sink, and keys and values that may
+be another layer's), attention over a cached latent, and the mixing weights of a residual that is
 kept in several streams.
 
 Every block reads the step's ``Context`` (which tokens belong to which sequence, their cache slots and

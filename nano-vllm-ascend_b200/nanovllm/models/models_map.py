@@ -9,7 +9,9 @@ with the norm on each sublayer's output) and Nurilorn (gated attention with capp
 stretched band by band and values blended across layers, on a residual with scaled branches and grouped norms) and
 Pofazen (windowed gated attention beside a gated delta rule in one mixer, and wkv recurrences with a token shift, on a
 residual whose norm is taken of the sum) and Ragilorn (attention inside chunks and latent attention, branches gated element
-by element, each layer handing on a weighted sum of all layers before it) are additions; their config.json names them with an ``"architecture"`` string (config.NativeConfig). Qwen2 checkpoints are served by the Qwen3 class, as in the reference:
+by element, each layer handing on a weighted sum of all layers before it) are additions; their config.json names them
+with an ``"architecture"`` string (config.NativeConfig). Qwen2 checkpoints are served by the Qwen3 class, as in the
+reference:
 the config's ``attention_bias`` decides between QKV bias (Qwen2) and QK-norm (Qwen3).
 """
 from __future__ import annotations

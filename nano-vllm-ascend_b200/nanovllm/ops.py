@@ -858,7 +858,8 @@ def act_and_mul(x, act="silu"):
         raise ValueError("act_and_mul input must be a matrix with unit inner stride")
     rows, inter = x.shape[0], x.shape[1] // 2
     out = torch.empty(rows, inter, dtype=x.dtype, device=x.device)
-    _C.check(_C.load().b200_act_and_mul(out.data_ptr(), x.data_ptr(), x.stride(0) if rows > 1 else x.shape[1], rows, inter, _ACTS[act], _dt3(x), _stream()),
+    _C.check(_C.load().b200_act_and_mul(out.data_ptr(), x.data_ptr(), x.stride(0) if rows > 1 else x.shape[1],
+                                        rows, inter, _ACTS[act], _dt3(x), _stream()),
              "b200_act_and_mul")
     return out
 
@@ -988,7 +989,8 @@ def attn_generic(q, k, v, spans: StepSpans, scale, num_kv_heads, vdim, block_tab
     v [Tk, G, vdim] (token-strided views allowed) in the order of spans.cu_k; paged mode (block_tables given):
     k, v are the caches [nb, bs, G*dim], [nb, bs, G*vdim]. Returns [T, H*vdim]. window > 0: position i sees the
     keys j <= i with i - j < window or j < keep_first; chunk > 0 (without a window): those with j // chunk == i // chunk. v
-    None: the values are the first vdim columns of the key rows. softcap > 0: scores become softcap * tanh(score / softcap). sink fp32 [H]: exp(sink[h]) joins the softmax denominator (no key,
+    None: the values are the first vdim columns of the key rows. softcap > 0: scores become softcap * tanh(score /
+    softcap). sink fp32 [H]: exp(sink[h]) joins the softmax denominator (no key,
     no value). gate [T, H] (q's dtype, row-strided view allowed): head h of token t is multiplied by sigmoid(gate[t, h])."""
     _need_cuda(q, k, v, block_tables, sink, gate)
     _f32(sink)
@@ -1441,7 +1443,8 @@ def moe_experts_generic(x, w13, w2, topk_weights, plan: MoePlan, act=None, glu=N
 
 
 # ---------------------------------------------------------------------------------------------------
-# Scaled residual with a grouped norm, gated residual with a depth average, capped logits, rotary positions from a frequency table fused with value blending and the K/V
+# Scaled residual with a grouped norm, gated residual with a depth average, capped logits, rotary positions from a
+# frequency table fused with value blending and the K/V
 # scatter, and the per-head output gate (csrc/seq_ops.cu).
 def wkv_prep(r, k, z, w0, u, num_heads, dim):
     """r, k [T, H*dim] (row-strided views allowed), z fp32 [T, H*dim]; w0, u fp32 [H*dim] -> (r fp32, k fp32, decay =
@@ -1525,7 +1528,8 @@ def residual_gate_average(x, y, gate, w, eps, dtype, c=1.0, y_index=None, x_out=
         raise ValueError("gate [rows, hidden] of the model dtype with unit inner stride")
     if any(t is not None and t.shape != (rows, hidden) for t in (x, x_out, keep)):
         raise ValueError("x, x_out, keep are [rows, hidden]")
-    if avg is not None and (avg.numel() != n + 1 or (n and (hist is None or hist.shape[0] < n or hist.shape[1:] != (rows, hidden)))):
+    if avg is not None and (avg.numel() != n + 1 or
+                            (n and (hist is None or hist.shape[0] < n or hist.shape[1:] != (rows, hidden)))):
         raise ValueError("avg [n + 1] over hist [>= n, rows, hidden]")
     h = torch.empty(rows, hidden, dtype=dtype, device=y.device) if w is not None else None
     _C.check(_C.load().b200_residual_gate_average(
